@@ -62,9 +62,12 @@ class ScheduleEntry:
     """One execution of a layer.  Every execution has cache storage of its own (a layer
     that is named twice runs with the same weights but keeps two caches), unless
     ``cache_of`` names an EARLIER position of the schedule: then this execution uses the
-    storage of that one (a layer that reads another layer's keys and values)."""
+    storage of that one (a layer that reads another layer's keys and values).
+    ``add_embedding``: the embedding's output is added to the stream right before this execution
+    (a further pass over layers that run several times starts so)."""
     layer: int
     cache_of: Optional[int] = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)

@@ -10,15 +10,19 @@
 //   cache write    src/l5_model.c:232-247      K after norm and rotation, V raw
 //   SiLU gate      src/l3_math.c:57-62, src/l5_model.c:594-595
 #include "common.cuh"
+#include "glu.cuh"
 
 G2B_DEFINE_LAST_ERROR
 
 // ---------------------------------------------------------------------------
-// embedding: out[t, :] = table[ids[t], :] * scale   (out is the 32-bit residual stream)
+// embedding: out[t, :] = table[ids[t], :] * scale   (out is the 32-bit residual stream); with a position
+// table also + positions[tok_pos[t], :], and a second copy of the rows into `again` when it is given
 // ---------------------------------------------------------------------------
 template <typename TW>
 __global__ void embed_rows_kernel(const TW *__restrict__ table, const int *__restrict__ ids,
-                                  float *__restrict__ out, int H, int V, float scale) {
+                                  float *__restrict__ out, int H, int V, float scale,
+                                  const TW *__restrict__ positions, const int *__restrict__ tok_pos, int n_pos,
+                                  float *__restrict__ again) {
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.x;
@@ -27,18 +31,29 @@ __global__ void embed_rows_kernel(const TW *__restrict__ table, const int *__res
   if (!ok) id = 0;                                   // host validates ids; never read outside
   const TW *row = table + (size_t)id * H;
   float *o = out + (size_t)t * H;
-  for (int j = threadIdx.x; j < H; j += blockDim.x) o[j] = ok ? to_f32(row[j]) * scale : 0.f;
+  // rows that only fill a step up may count past the table: their results are never used
+  const TW *prow = positions ? positions + (size_t)min(max(tok_pos[t], 0), n_pos - 1) * H : nullptr;
+  for (int j = threadIdx.x; j < H; j += blockDim.x) {
+    float v = ok ? to_f32(row[j]) * scale : 0.f;
+    if (prow) v += to_f32(prow[j]);
+    o[j] = v;
+    if (again) again[(size_t)t * H + j] = v;
+  }
 }
 
 extern "C" int g2b_embed_rows(const void *table, int table_dtype, const int *ids, float *out,
-                              int T, int H, int V, float scale, cudaStream_t stream) {
+                              int T, int H, int V, float scale, const void *positions, const int *tok_pos,
+                              int n_pos, float *again, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (positions && (!tok_pos || n_pos <= 0)) G2B_REFUSE("embed_rows: a position table needs its length and the tokens' positions");
   if (H <= 0 || V <= 0) G2B_REFUSE("embed_rows: bad sizes H=%d V=%d", H, V);
   const int threads = H >= 256 ? 256 : 64;
   if (table_dtype == G2B_F32)
-    g2b_launch(embed_rows_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float *)table, ids, out, H, V, scale);
+    g2b_launch(embed_rows_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float *)table, ids, out, H, V, scale,
+               (const float *)positions, tok_pos, n_pos, again);
   else if (table_dtype == G2B_BF16)
-    g2b_launch(embed_rows_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16 *)table, ids, out, H, V, scale);
+    g2b_launch(embed_rows_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16 *)table, ids, out, H, V, scale,
+               (const bf16 *)positions, tok_pos, n_pos, again);
   else
     G2B_REFUSE("embed_rows: unknown table dtype %d", table_dtype);
   return g2b_check_launch("embed_rows");
@@ -647,13 +662,11 @@ extern "C" int g2b_norm_shift(const float *x, const float *w, const float *mu, f
 // SiLU gate on a fused gate/up projection.  Rows of the fused matrix alternate in
 // blocks of `blk`: columns [2*blk*b, 2*blk*b+blk) are gate_{blk*b ..}, the next blk are
 // up_{blk*b ..}; blk == I means "all gates, then all ups".
-//   out[t, i] = (g / (1 + exp(-g))) * u
-// With `limit` > 0 the capped form: g = min(g, limit), u = clamp(u, -limit, limit),
-//   out[t, i] = g / (1 + exp(-alpha g)) * (u + 1)
+//   out[t, i] = (g / (1 + exp(-g))) * u, or another gate of the form in glu.cuh
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void swiglu_kernel(const T *__restrict__ gu, T *__restrict__ out, long long total,
-                              int I, int blk, float limit, float alpha) {
+                              int I, int blk, GluForm glu) {
   pdl_launch();
   pdl_wait();
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -662,22 +675,15 @@ __global__ void swiglu_kernel(const T *__restrict__ gu, T *__restrict__ out, lon
   const int i = (int)(idx % I);
   const int b = i / blk, r = i % blk;
   const T *row = gu + (size_t)t * 2 * I;
-  float g = to_f32(row[(size_t)2 * blk * b + r]);
-  float u = to_f32(row[(size_t)2 * blk * b + blk + r]);
-  if (limit > 0.f) {
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    out[idx] = from_f32<T>((g / (1.f + expf(-alpha * g))) * (u + 1.f));
-    return;
-  }
-  out[idx] = from_f32<T>((g / (1.f + expf(-g))) * u);
+  const float g = to_f32(row[(size_t)2 * blk * b + r]);
+  const float u = to_f32(row[(size_t)2 * blk * b + blk + r]);
+  out[idx] = from_f32<T>(glu_value(g, u, glu));
 }
 
 // The same in bfloat16 for blocks of a multiple of eight: a thread takes eight neighbouring outputs,
 // their gates and their ups as one 16-byte load each.
 __global__ void __launch_bounds__(256)
-swiglu8_kernel(const bf16 *__restrict__ gu, bf16 *__restrict__ out, long long total8, int I, int blk, float limit,
-               float alpha) {
+swiglu8_kernel(const bf16 *__restrict__ gu, bf16 *__restrict__ out, long long total8, int I, int blk, GluForm glu) {
   pdl_launch();
   pdl_wait();
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -693,40 +699,31 @@ swiglu8_kernel(const bf16 *__restrict__ gu, bf16 *__restrict__ out, long long to
   unsigned int ow[4];
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
-    float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&gw[e]));
-    float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&uw[e]));
-    float2 o;
-    if (limit > 0.f) {
-      g.x = fminf(g.x, limit), g.y = fminf(g.y, limit);
-      u.x = fminf(fmaxf(u.x, -limit), limit), u.y = fminf(fmaxf(u.y, -limit), limit);
-      o.x = (g.x / (1.f + expf(-alpha * g.x))) * (u.x + 1.f);
-      o.y = (g.y / (1.f + expf(-alpha * g.y))) * (u.y + 1.f);
-    } else {
-      o.x = (g.x / (1.f + expf(-g.x))) * u.x;
-      o.y = (g.y / (1.f + expf(-g.y))) * u.y;
-    }
-    const __nv_bfloat162 ob = __floats2bfloat162_rn(o.x, o.y);
+    const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&gw[e]));
+    const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&uw[e]));
+    const __nv_bfloat162 ob = __floats2bfloat162_rn(glu_value(g.x, u.x, glu), glu_value(g.y, u.y, glu));
     ow[e] = *reinterpret_cast<const unsigned int *>(&ob);
   }
   *reinterpret_cast<uint4 *>(out + (size_t)t * I + i) = make_uint4(ow[0], ow[1], ow[2], ow[3]);
 }
 
 extern "C" int g2b_swiglu(const void *gu, int dtype, int T_tokens, int I, int blk, void *out,
-                          float limit, float alpha, cudaStream_t stream) {
+                          float glu_limit, float glu_offset, float glu_c1, float glu_c3, cudaStream_t stream) {
+  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
   if (T_tokens <= 0) return 0;
   if (I <= 0 || blk <= 0 || I % blk) G2B_REFUSE("swiglu: block %d does not divide width %d", blk, I);
   const long long total = (long long)T_tokens * I;
   if (dtype == G2B_BF16 && blk % 8 == 0 && !(((uintptr_t)gu | (uintptr_t)out) & 15)) {
     const long long total8 = total / 8;
     g2b_launch(swiglu8_kernel, dim3((unsigned)((total8 + 255) / 256)), dim3(256), 0, stream, (const bf16 *)gu, (bf16 *)out,
-               total8, I, blk, limit, alpha);
+               total8, I, blk, glu);
     return g2b_check_launch("swiglu");
   }
   const unsigned blocks = (unsigned)((total + 255) / 256);
   if (dtype == G2B_F32)
-    g2b_launch(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float *)gu, (float *)out, total, I, blk, limit, alpha);
+    g2b_launch(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float *)gu, (float *)out, total, I, blk, glu);
   else if (dtype == G2B_BF16)
-    g2b_launch(swiglu_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16 *)gu, (bf16 *)out, total, I, blk, limit, alpha);
+    g2b_launch(swiglu_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16 *)gu, (bf16 *)out, total, I, blk, glu);
   else
     G2B_REFUSE("swiglu: unknown dtype %d", dtype);
   return g2b_check_launch("swiglu");

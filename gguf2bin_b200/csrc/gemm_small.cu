@@ -25,6 +25,7 @@
 // out[m, 8b + r] = silu(row r of block b) * (row 8 + r)   (src/l3_math.c:57-62,
 // src/l5_model.c:594-595 of AnonymoDGH/gguf2bin).
 #include "common.cuh"
+#include "glu.cuh"
 #include "mma.cuh"
 
 #include <cooperative_groups.h>
@@ -37,6 +38,14 @@ constexpr int XPAD = 32;                // elements of padding per staged row (6
 constexpr int XROW = KB + XPAD;
 constexpr int DEPTH = 4;                // K blocks of W in flight per thread
 
+// As in gemm_tc.cu: a build with -DG2B_GLU holds the gated epilogue alone, in its general form.
+#ifdef G2B_GLU
+__device__ __forceinline__ float glu_out(float gate, float up, const GluForm &f) { return glu_value(gate, up, f); }
+#define G2B_IF_UNGATED(...)
+#else
+__device__ __forceinline__ float glu_out(float gate, float up, const GluForm &) { return (gate / (1.f + expf(-gate))) * up; }
+#define G2B_IF_UNGATED(...) __VA_ARGS__
+#endif
 enum { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ACCUM_F32 = 2, EPI_SWIGLU_BF16 = 3 };
 
 __device__ __forceinline__ uint4 ld_stream(const void *p) {
@@ -50,7 +59,7 @@ __device__ __forceinline__ uint4 ld_stream(const void *p) {
 template <int MT, int EPI>
 __global__ void __launch_bounds__(WARPS * 32)
 gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *__restrict__ Cv,
-                  int M, int N, int K, int lda, int ldw, int ldc) {
+                  int M, int N, int K, int lda, int ldw, int ldc, GluForm glu) {
   pdl_launch();
   constexpr int MROWS = MT * 8;
   extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -144,7 +153,7 @@ gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *
       }
       const int col = (n0 >> 1) + r;
       if (m < M && n0 + 8 + r < N)
-        ((bf16 *)Cv)[(size_t)m * ldc + col] = __float2bfloat16_rn((gate / (1.f + expf(-gate))) * up);
+        ((bf16 *)Cv)[(size_t)m * ldc + col] = __float2bfloat16_rn(glu_out(gate, up, glu));
     }
   } else {
     for (int i = threadIdx.x; i < 16 * MROWS; i += WARPS * 32) {
@@ -184,7 +193,7 @@ gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *
 template <int MT, int EPI, int DEPTH_WHOLE, int SPLIT, bool NORMED = false>
 __global__ void __launch_bounds__(WARPS * 32, DEPTH_WHOLE == 4 ? 3 : 2)
 gemm_small_whole_kernel(const void *__restrict__ Av, const bf16 *__restrict__ W,
-                        void *__restrict__ Cv, int M, int N, int K, int lda, int ldw, int ldc, float eps) {
+                        void *__restrict__ Cv, int M, int N, int K, int lda, int ldw, int ldc, float eps, GluForm glu) {
   static_assert(!NORMED || SPLIT == 1, "the normalised product is not split over a cluster");
   pdl_launch();
   const bf16 *A = reinterpret_cast<const bf16 *>(Av);
@@ -325,7 +334,7 @@ gemm_small_whole_kernel(const void *__restrict__ Av, const bf16 *__restrict__ W,
       if (NORMED) { gate *= row_scale[m]; up *= row_scale[m]; }
       const int col = (n0 >> 1) + r;
       if (m < M && n0 + 8 + r < N)
-        ((bf16 *)Cv)[(size_t)m * ldc + col] = __float2bfloat16_rn((gate / (1.f + expf(-gate))) * up);
+        ((bf16 *)Cv)[(size_t)m * ldc + col] = __float2bfloat16_rn(glu_out(gate, up, glu));
     }
   } else {
     for (int i = threadIdx.x; i < 16 * MROWS; i += WARPS * 32) {
@@ -374,7 +383,7 @@ template <int MT>
 __global__ void __launch_bounds__(WARPS * 32, 1)
 gemm_small_stream_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *__restrict__ Cv,
                          int M, int N, int K, int lda, int ldw, int ldc, int epi, int n_chunks, int kbc,
-                         int tiles_per_cta) {
+                         int tiles_per_cta, GluForm glu) {
   pdl_launch();
   using C = StreamCfg<MT>;
   constexpr int MROWS = C::MROWS, XROWS = C::XROWS, RING = C::RING, G = STREAM_BATCH;
@@ -509,7 +518,7 @@ gemm_small_stream_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W,
             up += red[((size_t)w * 16 + 8 + r) * MROWS + m];
           }
           if (m < M && n0 + 8 + r < N)
-            ((bf16 *)Cv)[(size_t)m * ldc + (n0 >> 1) + r] = __float2bfloat16_rn((gate / (1.f + expf(-gate))) * up);
+            ((bf16 *)Cv)[(size_t)m * ldc + (n0 >> 1) + r] = __float2bfloat16_rn(glu_out(gate, up, glu));
         }
       } else {
         for (int i = threadIdx.x; i < 16 * MROWS; i += WARPS * 32) {
@@ -559,7 +568,7 @@ static int final_split(int N, int K) {
 
 template <int MT, int DEPTH_WHOLE, int SPLIT>
 static int launch_whole_depth(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw,
-                              int ldc, int epi, cudaStream_t stream) {
+                              int ldc, int epi, GluForm glu, cudaStream_t stream) {
   const int smem = (int)whole_smem(MT * 8, K, SPLIT);
   const int n_tiles = (N + 15) / 16;
   const unsigned grid = (unsigned)(n_tiles * SPLIT);
@@ -575,12 +584,12 @@ static int launch_whole_depth(const void *A, const void *W, void *C, int M, int 
     }                                                                                            \
     g2b_launch_cluster(gemm_small_whole_kernel<MT, E, DEPTH_WHOLE, SPLIT>, dim3(grid),           \
                        dim3(WARPS * 32), smem, stream, (unsigned)SPLIT, (const void *)A,         \
-                       (const bf16 *)W, C, M, N, K, lda, ldw, ldc, 0.f);                         \
+                       (const bf16 *)W, C, M, N, K, lda, ldw, ldc, 0.f, glu);                         \
   } while (0)
   switch (epi) {
-    case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;
-    case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;
-    case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;
+    G2B_IF_UNGATED(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
+    G2B_IF_UNGATED(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
+    G2B_IF_UNGATED(case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;)
     case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;
     default: G2B_REFUSE("gemm_small: unknown epilogue %d", epi);
   }
@@ -590,18 +599,18 @@ static int launch_whole_depth(const void *A, const void *W, void *C, int M, int 
 
 template <int MT>
 static int launch_whole(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw, int ldc,
-                        int epi, cudaStream_t stream) {
+                        int epi, GluForm glu, cudaStream_t stream) {
   const int nkb = (K + KB - 1) / KB;
   const int split = final_split(N, K);
-  if (split == 4) return launch_whole_depth<MT, 4, 4>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-  if (split == 2) return launch_whole_depth<MT, 4, 2>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-  if (nkb <= 4) return launch_whole_depth<MT, 4, 1>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-  return launch_whole_depth<MT, 8, 1>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
+  if (split == 4) return launch_whole_depth<MT, 4, 4>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+  if (split == 2) return launch_whole_depth<MT, 4, 2>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+  if (nkb <= 4) return launch_whole_depth<MT, 4, 1>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+  return launch_whole_depth<MT, 8, 1>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
 }
 
 template <int MT>
 static int launch_mt(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw,
-                     int ldc, int epi, cudaStream_t stream) {
+                     int ldc, int epi, GluForm glu, cudaStream_t stream) {
   constexpr int MROWS = MT * 8;
   const size_t stage = (size_t)2 * MROWS * XROW * sizeof(bf16);
   const size_t red = (size_t)WARPS * 16 * MROWS * sizeof(float);
@@ -618,12 +627,12 @@ static int launch_mt(const void *A, const void *W, void *C, int M, int N, int K,
       if (cfg_dev >= 0) configured.value[cfg_dev] = 1;                                           \
     }                                                                                            \
     g2b_launch(gemm_small_kernel<MT, E>, dim3(grid), dim3(WARPS * 32), smem, stream,                                 \
-        (const bf16 *)A, (const bf16 *)W, C, M, N, K, lda, ldw, ldc);                            \
+        (const bf16 *)A, (const bf16 *)W, C, M, N, K, lda, ldw, ldc, glu);                       \
   } while (0)
   switch (epi) {
-    case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;
-    case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;
-    case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;
+    G2B_IF_UNGATED(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
+    G2B_IF_UNGATED(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
+    G2B_IF_UNGATED(case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;)
     case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;
     default: G2B_REFUSE("gemm_small: unknown epilogue %d", epi);
   }
@@ -636,6 +645,7 @@ static int launch_mt(const void *A, const void *W, void *C, int M, int N, int K,
 template <int MT, int DEPTH_WHOLE>
 static int launch_normed(const float *X, const void *W, void *C, int M, int N, int K, int ldx, int ldw,
                          int ldc, int epi, float eps, cudaStream_t stream) {
+  const GluForm glu = {INFINITY, 0.f, 1.f, 0.f};             // SiLU
   const int smem = (int)whole_smem(MT * 8, K, 1);
   const unsigned grid = (unsigned)((N + 15) / 16);
 #define G2B_LAUNCH(E)                                                                            \
@@ -649,11 +659,11 @@ static int launch_normed(const float *X, const void *W, void *C, int M, int N, i
       if (cfg_dev >= 0) configured.value[cfg_dev] = smem;                                        \
     }                                                                                            \
     g2b_launch(gemm_small_whole_kernel<MT, E, DEPTH_WHOLE, 1, true>, dim3(grid), dim3(WARPS * 32), smem, \
-               stream, (const void *)X, (const bf16 *)W, C, M, N, K, ldx, ldw, ldc, eps);        \
+               stream, (const void *)X, (const bf16 *)W, C, M, N, K, ldx, ldw, ldc, eps, glu);   \
   } while (0)
   switch (epi) {
-    case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;
-    case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;
+    G2B_IF_UNGATED(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
+    G2B_IF_UNGATED(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
     case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;
     default: G2B_REFUSE("gemm_small_normed: epilogue %d (store or SiLU gate only)", epi);
   }
@@ -683,7 +693,7 @@ static bool stream_case(int M, int N, int K) {
 
 template <int MT>
 static int launch_stream(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw, int ldc,
-                         int epi, cudaStream_t stream) {
+                         int epi, GluForm glu, cudaStream_t stream) {
   if (epi < EPI_STORE_BF16 || epi > EPI_SWIGLU_BF16) G2B_REFUSE("gemm_small: unknown epilogue %d", epi);
   constexpr int CB = StreamCfg<MT>::CB;
   const int smem = (int)StreamCfg<MT>::TOTAL;
@@ -700,33 +710,35 @@ static int launch_stream(const void *A, const void *W, void *C, int M, int N, in
   const int per = (n_tiles + sm_count() - 1) / sm_count();          // tiles per CTA: the same for (almost) all
   const unsigned grid = (unsigned)((n_tiles + per - 1) / per);
   g2b_launch(gemm_small_stream_kernel<MT>, dim3(grid), dim3(WARPS * 32), smem, stream, (const bf16 *)A,
-             (const bf16 *)W, C, M, N, K, lda, ldw, ldc, epi, n_chunks, kbc, per);
+             (const bf16 *)W, C, M, N, K, lda, ldw, ldc, epi, n_chunks, kbc, per, glu);
   return g2b_check_launch("gemm_small_stream");
 }
 
 // A [M,K] and W [N,K] bfloat16 with unit inner stride; rows 16-byte aligned.
-// epi: 0 store bfloat16, 1 store float, 2 add into float, 3 SiLU gate (C is [M, N/2] bfloat16;
-// N must be a multiple of 16).
+// epi: 0 store bfloat16, 1 store float, 2 add into float, 3 gate (C is [M, N/2] bfloat16; N must be a
+// multiple of 16): SiLU, or in a build with -DG2B_GLU (that epilogue alone) the form of the glu_ numbers.
 extern "C" int g2b_gemm_small(const void *A, const void *W, void *C, int M, int N, int K, int lda,
-                              int ldw, int ldc, int epi, cudaStream_t stream) {
+                              int ldw, int ldc, int epi, float glu_limit, float glu_offset, float glu_c1,
+                              float glu_c3, cudaStream_t stream) {
+  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
   if (M <= 0 || N <= 0) return 0;
   if (M > 64) G2B_REFUSE("gemm_small: M=%d (at most 64 rows)", M);
   if (K <= 0 || K % 8 || lda % 8 || ldw % 8)
     G2B_REFUSE("gemm_small: K=%d and the row strides (%d, %d) must be multiples of 8", K, lda, ldw);
   if (((uintptr_t)A | (uintptr_t)W) & 15) G2B_REFUSE("gemm_small: operands must be 16-byte aligned");
   if (epi == EPI_SWIGLU_BF16 && N % 16) G2B_REFUSE("gemm_small: gated output needs N %% 16 == 0, N=%d", N);
-  if (stream_case(M, N, K)) return launch_stream<1>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
+  if (stream_case(M, N, K)) return launch_stream<1>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
   const int mrows = M <= 8 ? 8 : (M <= 16 ? 16 : (M <= 32 ? 32 : 64));
   if (whole_smem(mrows, K, final_split(N, K))) {
-    if (M <= 8) return launch_whole<1>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-    if (M <= 16) return launch_whole<2>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-    if (M <= 32) return launch_whole<4>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-    return launch_whole<8>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
+    if (M <= 8) return launch_whole<1>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+    if (M <= 16) return launch_whole<2>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+    if (M <= 32) return launch_whole<4>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+    return launch_whole<8>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
   }
-  if (M <= 8) return launch_mt<1>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-  if (M <= 16) return launch_mt<2>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-  if (M <= 32) return launch_mt<4>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
-  return launch_mt<8>(A, W, C, M, N, K, lda, ldw, ldc, epi, stream);
+  if (M <= 8) return launch_mt<1>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+  if (M <= 16) return launch_mt<2>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+  if (M <= 32) return launch_mt<4>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
+  return launch_mt<8>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
 }
 
 // Whether g2b_gemm_small_normed takes the case: up to 16 rows, the whole of A in shared memory,

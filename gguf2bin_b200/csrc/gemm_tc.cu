@@ -24,6 +24,7 @@
 // code in `*status`, all roles fall through to the common exit, the tensor memory is freed
 // and the kernel returns; the host reads `*status` (0 = fine).
 #include "common.cuh"
+#include "glu.cuh"
 #include "tc_common.cuh"
 
 G2B_DEFINE_LAST_ERROR
@@ -35,6 +36,17 @@ constexpr int BK = 64;                      // 64 bf16 = 128 bytes = one swizzle
 constexpr int THREADS = 192;
 
 enum { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ACCUM_F32 = 2, EPI_SWIGLU_BF16 = 3 };
+// The gate of the gated epilogue: SiLU; in a build with -DG2B_GLU, which holds that epilogue alone, the
+// general form that the launch gives (glu.cuh).
+#ifdef G2B_GLU
+__device__ __forceinline__ float glu_out(float gate, float up, const GluForm &f) { return glu_value_fast(gate, up, f); }
+#define G2B_CASE_UNGATED(...)
+#else
+__device__ __forceinline__ float glu_out(float gate, float up, const GluForm &) {
+  return __fdividef(gate, 1.f + __expf(-gate)) * up;
+}
+#define G2B_CASE_UNGATED(...) G2B_CASE(__VA_ARGS__)
+#endif
 enum { ST_OK = 0, ST_PRODUCER_TIMEOUT = 1, ST_MMA_TIMEOUT = 2, ST_EPILOGUE_TIMEOUT = 3 };
 
 __device__ __forceinline__ uint32_t pack2(uint32_t lo, uint32_t hi) {
@@ -63,7 +75,7 @@ template <int BN, int STAGES> struct Smem {
 // shared memory of this warp (used by the float outputs to turn rows into coalesced stores).
 template <int BN, int EPI>
 __device__ __forceinline__ void epilogue_tile(uint32_t tmem, float *scr, void *__restrict__ Cv, int m0, int n0,
-                                              int M, int N, int ldc, int warp, int lane) {
+                                              int M, int N, int ldc, int warp, int lane, const GluForm &glu) {
       const int row = m0 + warp * 32 + lane;
 #pragma unroll 1
       for (int c0 = 0; c0 < BN; c0 += 32) {
@@ -105,7 +117,7 @@ __device__ __forceinline__ void epilogue_tile(uint32_t tmem, float *scr, void *_
             for (int j = 0; j < 8; ++j) {
               const float gate = __uint_as_float(r[16 * blk + j]);
               const float up = __uint_as_float(r[16 * blk + 8 + j]);
-              h[8 * blk + j] = __fdividef(gate, 1.f + __expf(-gate)) * up;
+              h[8 * blk + j] = glu_out(gate, up, glu);
             }
           if (n + 32 <= N && ((((uintptr_t)dst) & 15) == 0)) {
 #pragma unroll
@@ -142,7 +154,7 @@ __device__ __forceinline__ void epilogue_tile(uint32_t tmem, float *scr, void *_
 template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-               void *__restrict__ Cv, int M, int N, int K, int ldc, int *__restrict__ status) {
+               void *__restrict__ Cv, int M, int N, int K, int ldc, int *__restrict__ status, GluForm glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = Smem<BN, STAGES>;
@@ -218,7 +230,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
       if (lane == 0) atomicExch(status, ST_EPILOGUE_TIMEOUT);
     } else {
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-      epilogue_tile<BN, EPI>(tmem, reinterpret_cast<float *>(smem) + warp * (32 * 33), Cv, m0, n0, M, N, ldc, warp, lane);
+      epilogue_tile<BN, EPI>(tmem, reinterpret_cast<float *>(smem) + warp * (32 * 33), Cv, m0, n0, M, N, ldc, warp, lane, glu);
     }
   }
   asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -243,7 +255,7 @@ template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                        void *__restrict__ Cv, const int *__restrict__ plan, int n_groups, int Nw, int K, int ldc,
-                       int *__restrict__ status) {
+                       int *__restrict__ status, GluForm glu) {
   pdl_launch();
   pdl_wait();                  // the plan is an earlier kernel's output
   const int tile = blockIdx.y;
@@ -322,7 +334,7 @@ gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_c
       if (lane == 0) atomicExch(status, ST_EPILOGUE_TIMEOUT);
     } else {
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-      epilogue_tile<BN, EPI>(tmem, reinterpret_cast<float *>(smem) + warp * (32 * 33), Cv, m0, n0, m_end, Nw, ldc, warp, lane);
+      epilogue_tile<BN, EPI>(tmem, reinterpret_cast<float *>(smem) + warp * (32 * 33), Cv, m0, n0, m_end, Nw, ldc, warp, lane, glu);
     }
   }
   asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -346,7 +358,7 @@ gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_c
 template <int EPI>
 __device__ __forceinline__ void epilogue_chunk(const uint32_t (&v)[32], int c, unsigned char *stage,
                                                const CUtensorMap *map_c, int y, int n0, int M, int N, int lane,
-                                               uint32_t &box) {
+                                               uint32_t &box, const GluForm &glu) {
   // which 16-byte chunks of the row this accumulator chunk fills, and whether it completes a box
   constexpr int PER_BOX = EPI == EPI_SWIGLU_BF16 ? 4 : (EPI == EPI_STORE_BF16 ? 2 : 1);
   const int part = c % PER_BOX;
@@ -378,7 +390,7 @@ __device__ __forceinline__ void epilogue_chunk(const uint32_t (&v)[32], int c, u
       for (int j = 0; j < 8; ++j) {
         const float gate = __uint_as_float(v[16 * blk + j]);
         const float up = __uint_as_float(v[16 * blk + 8 + j]);
-        h[8 * blk + j] = __fdividef(gate, 1.f + __expf(-gate)) * up;
+        h[8 * blk + j] = glu_out(gate, up, glu);
       }
 #pragma unroll
     for (int j = 0; j < 2; ++j)
@@ -404,7 +416,7 @@ __device__ __forceinline__ void epilogue_chunk(const uint32_t (&v)[32], int c, u
 template <int BN, int EPI>
 __device__ __forceinline__ void epilogue_tile_bulk(uint32_t tmem, unsigned char *stage, const CUtensorMap *map_c,
                                                    int m0, int n0, int M, int N, int warp, int lane,
-                                                   uint32_t &box) {
+                                                   uint32_t &box, const GluForm &glu) {
   constexpr int CHUNKS = BN / 32;
   const uint32_t lane_addr = tmem + ((uint32_t)(warp * 32) << 16);
   const int y = m0 + warp * 32;
@@ -414,7 +426,7 @@ __device__ __forceinline__ void epilogue_tile_bulk(uint32_t tmem, unsigned char 
   for (int c = 0; c < CHUNKS; ++c) {
     asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
     if (c + 1 < CHUNKS) tmem_ld32(lane_addr + 32 * (c + 1), r[(c + 1) & 1]);
-    epilogue_chunk<EPI>(r[c & 1], c, stage, map_c, y, n0, M, N, lane, box);
+    epilogue_chunk<EPI>(r[c & 1], c, stage, map_c, y, n0, M, N, lane, box, glu);
   }
 }
 
@@ -489,7 +501,7 @@ __device__ __forceinline__ void parts_send(unsigned char *ring, uint32_t part_ba
 template <int BN, int EPI>
 __device__ __forceinline__ void parts_finish(uint32_t tmem, const unsigned char *ring, unsigned char *stage,
                                              const CUtensorMap *map_c, int m0, int n0, int M, int N, int warp,
-                                             int lane, uint32_t &box, int rank, int S) {
+                                             int lane, uint32_t &box, int rank, int S, const GluForm &glu) {
   constexpr int CHUNKS = BN / 32;
   const int own_lo = part_chunk_lo<BN, EPI>(rank, S), own_n = part_chunk_lo<BN, EPI>(rank + 1, S) - own_lo;
   const uint32_t lane_addr = tmem + ((uint32_t)(warp * 32) << 16);
@@ -520,7 +532,7 @@ __device__ __forceinline__ void parts_finish(uint32_t tmem, const unsigned char 
         }
       }
     }
-    epilogue_chunk<EPI>(v, own_lo + i, stage, map_c, y, n0, M, N, lane, box);
+    epilogue_chunk<EPI>(v, own_lo + i, stage, map_c, y, n0, M, N, lane, box, glu);
   }
 }
 
@@ -576,7 +588,7 @@ template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                           const __grid_constant__ CUtensorMap map_c, int M, int N, int K, int group_m,
-                          int k_parts, int *__restrict__ status) {
+                          int k_parts, int *__restrict__ status, GluForm glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = SmemP<BN, STAGES>;
@@ -727,7 +739,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
       int tm, tn;
       tile_of(t, tiles_m, tiles_n, group_m, tm, tn);
       const int m0 = tm * BM, n0 = tn * BN;
-      epilogue_tile_bulk<BN, EPI>(tmem + buf * BN, stage, &map_c, m0, n0, M, N, warp, lane, box);
+      epilogue_tile_bulk<BN, EPI>(tmem + buf * BN, stage, &map_c, m0, n0, M, N, warp, lane, box, glu);
       // every load of this warp from the accumulator has completed (each is waited for)
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
       __syncwarp();
@@ -763,7 +775,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
         uint32_t box = 0;
         int tm, tn;
         tile_of(walker, tiles_m, tiles_n, group_m, tm, tn);
-        parts_finish<BN, EPI>(tmem, smem, stage, &map_c, tm * BM, tn * BN, M, N, warp, lane, box, rank, k_parts);
+        parts_finish<BN, EPI>(tmem, smem, stage, &map_c, tm * BM, tn * BN, M, N, warp, lane, box, rank, k_parts, glu);
       }
       if (lane == 0) bulk_wait<0>();
     }
@@ -810,7 +822,7 @@ template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     const __grid_constant__ CUtensorMap map_c, int M, int N, int K, int group_m,
-                    int *__restrict__ status) {
+                    int *__restrict__ status, GluForm glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = SmemPair<BN, STAGES>;
@@ -918,7 +930,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       int tm, tn;
       tile_of(t, tiles_m, tiles_n, group_m, tm, tn);
       const int m0 = tm * (2 * BM) + (int)rank * BM, n0 = tn * BN;
-      epilogue_tile_bulk<BN, EPI>(tmem + buf * BN, stage, &map_c, m0, n0, M, N, warp, lane, box);
+      epilogue_tile_bulk<BN, EPI>(tmem + buf * BN, stage, &map_c, m0, n0, M, N, warp, lane, box, glu);
       // every load of this warp from the accumulator has completed (each is waited for)
       tc_fence_before();
       __syncwarp();
@@ -969,7 +981,7 @@ template <int BNB, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_wstream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
                        void *__restrict__ Cv, int M, int N, int K, int ldc, int splits,
-                       int *__restrict__ status) {
+                       int *__restrict__ status, GluForm glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = SmemWS<BNB, STAGES>;
@@ -1160,8 +1172,8 @@ gemm_tc_wstream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
         if ((lane & 2) == 0) {
           const int col = ((n >> 4) << 3) + (n & 7);          // output column of v.x
           bf16 *dst = (bf16 *)Cv + (size_t)m * ldc + col;
-          const float h0 = __fdividef(v.x, 1.f + __expf(-v.x)) * up.x, h1 = __fdividef(v.y, 1.f + __expf(-v.y)) * up.y;
-          const float h2 = __fdividef(v.z, 1.f + __expf(-v.z)) * up.z, h3 = __fdividef(v.w, 1.f + __expf(-v.w)) * up.w;
+          const float h0 = glu_out(v.x, up.x, glu), h1 = glu_out(v.y, up.y, glu);
+          const float h2 = glu_out(v.z, up.z, glu), h3 = glu_out(v.w, up.w, glu);
           if (n + 16 <= N && ((((uintptr_t)dst) & 7) == 0)) {
             *reinterpret_cast<uint2 *>(dst) = make_uint2(pack2f(h0, h1), pack2f(h2, h3));
           } else {
@@ -1229,7 +1241,7 @@ static int make_map_c(CUtensorMap *map, const void *base, int rows, int cols, in
 
 template <int BN, int STAGES, int EPI>
 static int launch(const CUtensorMap &ma, const CUtensorMap &mw, void *C, int M, int N, int K, int ldc,
-                  int *status, cudaStream_t stream) {
+                  int *status, GluForm glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = Smem<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1241,7 +1253,7 @@ static int launch(const CUtensorMap &ma, const CUtensorMap &mw, void *C, int M, 
   }
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
   if (grid.y > 65535) G2B_REFUSE("gemm_tc: M=%d is too large for one launch", M);
-  g2b_launch(gemm_tc_kernel<BN, STAGES, EPI>, dim3(grid), dim3(THREADS), smem, stream, ma, mw, C, M, N, K, ldc, status);
+  g2b_launch(gemm_tc_kernel<BN, STAGES, EPI>, dim3(grid), dim3(THREADS), smem, stream, ma, mw, C, M, N, K, ldc, status, glu);
   return g2b_check_launch("gemm_tc");
 }
 
@@ -1342,7 +1354,7 @@ static_assert(SmemP<128, 6>::RING_BYTES == 196608 && SmemP<256, 4>::RING_BYTES =
 // want_parts: 1 to 4 parts of K
 template <int BN, int STAGES, int EPI>
 static int launch_persistent(const CUtensorMap &ma, const CUtensorMap &mw, void *C, int M, int N, int K, int ldc,
-                             int want_parts, int *status, cudaStream_t stream) {
+                             int want_parts, int *status, GluForm glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = SmemP<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1375,13 +1387,13 @@ static int launch_persistent(const CUtensorMap &ma, const CUtensorMap &mw, void 
   const unsigned grid = parts > 1 ? (unsigned)(tiles * parts) : (unsigned)(tiles < sm_count() ? tiles : sm_count());
   g2b_launch_cluster(gemm_tc_persistent_kernel<BN, STAGES, EPI>, dim3(grid), dim3(THREADS), smem, stream,
                      (unsigned)parts, ma, mw, mc, M, N, K, rows_of_tiles_per_group((M + BM - 1) / BM, BM, K), parts,
-                     status);
+                     status, glu);
   return g2b_check_launch("gemm_tc (persistent)");
 }
 
 template <int BN, int STAGES, int EPI>
 static int launch_pair(const CUtensorMap &ma, const CUtensorMap &mw, void *C, int M, int N, int K, int ldc,
-                       int *status, cudaStream_t stream) {
+                       int *status, GluForm glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = SmemPair<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1405,13 +1417,13 @@ static int launch_pair(const CUtensorMap &ma, const CUtensorMap &mw, void *C, in
   if (max_pairs < 1) G2B_REFUSE("gemm_tc: the paired kernel needs two SMs");
   const unsigned pairs = (unsigned)(tiles < max_pairs ? tiles : max_pairs);
   g2b_launch_cluster(gemm_tc_pair_kernel<BN, STAGES, EPI>, dim3(2 * pairs), dim3(THREADS), smem, stream, 2u, ma, mw,
-                     mc, M, N, K, rows_of_tiles_per_group((M + 2 * BM - 1) / (2 * BM), 2 * BM, K), status);
+                     mc, M, N, K, rows_of_tiles_per_group((M + 2 * BM - 1) / (2 * BM), 2 * BM, K), status, glu);
   return g2b_check_launch("gemm_tc (pairs)");
 }
 
 template <int BNB, int STAGES, int EPI>
 static int launch_wstream(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw, int ldc,
-                          int want_splits, int *status, cudaStream_t stream) {
+                          int want_splits, int *status, GluForm glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   using S = SmemWS<BNB, STAGES>;
   const int cfg_dev = g2b_current_device();
@@ -1459,13 +1471,14 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
   while (splits > 1 && (splits - 1) * ((nkb + splits - 1) / splits) >= nkb) --splits;      // no empty part
   static_assert((2 * BNB + 8) * BM * 4 <= S::RING_BYTES, "the tile and the received ranges must fit the ring");
   g2b_launch_cluster(gemm_tc_wstream_kernel<BNB, STAGES, EPI>, dim3((unsigned)(tiles * splits)), dim3(THREADS),
-                     S::TOTAL, stream, (unsigned)splits, mw, ma, C, M, N, K, ldc, splits, status);
+                     S::TOTAL, stream, (unsigned)splits, mw, ma, C, M, N, K, ldc, splits, status, glu);
   return g2b_check_launch("gemm_tc (weight streaming)");
 }
 
 // A [M,K], W [N,K] bfloat16, inner stride 1, row strides multiples of 8 elements, base
 // addresses 16-byte aligned.  epi: 0 store bfloat16, 1 store float, 2 add into float,
-// 3 SiLU gate (C is [M, N/2] bfloat16; N a multiple of 16).  `status` is a device int the
+// 3 gate (C is [M, N/2] bfloat16; N a multiple of 16): SiLU, or in a build with -DG2B_GLU (which
+// has no other epilogue) the form of the four glu_ numbers (glu.cuh).  `status` is a device int the
 // kernel sets non-zero if one of its bounded waits gave up.  Tile shapes (bn, stages):
 // (64,4) (64,8) (128,3) (128,6) (256,4); bn = 0 picks one from the sizes: wide tiles when
 // there are plenty of them, narrow tiles with a deeper ring when the grid would not fill
@@ -1478,7 +1491,8 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
 // the launcher choose): the weight-streaming kernel with K split over a cluster.
 extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, int K, int lda,
                            int ldw, int ldc, int epi, int bn, int stages, int persistent, int *status,
-                           cudaStream_t stream) {
+                           float glu_limit, float glu_offset, float glu_c1, float glu_c3, cudaStream_t stream) {
+  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8 || ldw % 8)
     G2B_REFUSE("gemm_tc: K=%d and the row strides (%d, %d) must be multiples of 8", K, lda, ldw);
@@ -1497,13 +1511,13 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
     if (epi == E) {                                                                                        \
       /* more tiles than SMs (K is not split then): half the ring, so that two CTAs share an SM and */ \
       /* the tiles of the second round stream beside those of the first instead of after them       */ \
-      if (M <= 32 && crowded) return launch_wstream<32, 4, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, stream); \
-      if (M <= 32) return launch_wstream<32, 9, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, stream);   \
-      if (M <= 64 && crowded) return launch_wstream<64, 4, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, stream); \
-      if (M <= 64) return launch_wstream<64, 8, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, stream);   \
-      return launch_wstream<128, 6, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, stream);               \
+      if (M <= 32 && crowded) return launch_wstream<32, 4, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, glu, stream); \
+      if (M <= 32) return launch_wstream<32, 9, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, glu, stream);   \
+      if (M <= 64 && crowded) return launch_wstream<64, 4, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, glu, stream); \
+      if (M <= 64) return launch_wstream<64, 8, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, glu, stream);   \
+      return launch_wstream<128, 6, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, glu, stream);               \
     }
-    G2B_CASE(EPI_STORE_BF16) G2B_CASE(EPI_STORE_F32) G2B_CASE(EPI_ACCUM_F32) G2B_CASE(EPI_SWIGLU_BF16)
+    G2B_CASE_UNGATED(EPI_STORE_BF16) G2B_CASE_UNGATED(EPI_STORE_F32) G2B_CASE_UNGATED(EPI_ACCUM_F32) G2B_CASE(EPI_SWIGLU_BF16)
 #undef G2B_CASE
     G2B_REFUSE("gemm_tc: unknown epilogue %d", epi);
   }
@@ -1527,9 +1541,9 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
     if (rc) return rc;
 #define G2B_CASE(BN_, ST_, E) \
     if (bn == BN_ && stages == ST_ && epi == E)                                                      \
-      return launch_pair<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, status, stream);
+      return launch_pair<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, status, glu, stream);
 #define G2B_SHAPE(BN_, ST_) \
-    G2B_CASE(BN_, ST_, EPI_STORE_BF16) G2B_CASE(BN_, ST_, EPI_STORE_F32) G2B_CASE(BN_, ST_, EPI_ACCUM_F32) \
+    G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_BF16) G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_F32) G2B_CASE_UNGATED(BN_, ST_, EPI_ACCUM_F32) \
     G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
     G2B_SHAPE(256, 6) G2B_SHAPE(256, 4)
 #undef G2B_SHAPE
@@ -1540,20 +1554,20 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
   if (rc) return rc;
 #define G2B_CASE(BN_, ST_, E) \
   if (persistent && bn == BN_ && stages == ST_ && epi == E)                                        \
-    return launch_persistent<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, parts, status, stream);
+    return launch_persistent<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, parts, status, glu, stream);
 #define G2B_SHAPE(BN_, ST_) \
-  G2B_CASE(BN_, ST_, EPI_STORE_BF16) G2B_CASE(BN_, ST_, EPI_STORE_F32) \
-  G2B_CASE(BN_, ST_, EPI_ACCUM_F32) G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
+  G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_BF16) G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_F32) \
+  G2B_CASE_UNGATED(BN_, ST_, EPI_ACCUM_F32) G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
   G2B_SHAPE(128, 6) G2B_SHAPE(256, 4)
 #undef G2B_SHAPE
 #undef G2B_CASE
   if (persistent)
     G2B_REFUSE("gemm_tc: no persistent kernel for tile width %d with %d stages and epilogue %d", bn, stages, epi);
 #define G2B_CASE(BN_, ST_, E) \
-  if (bn == BN_ && stages == ST_ && epi == E) return launch<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, status, stream);
+  if (bn == BN_ && stages == ST_ && epi == E) return launch<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, status, glu, stream);
 #define G2B_SHAPE(BN_, ST_) \
-  G2B_CASE(BN_, ST_, EPI_STORE_BF16) G2B_CASE(BN_, ST_, EPI_STORE_F32) \
-  G2B_CASE(BN_, ST_, EPI_ACCUM_F32) G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
+  G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_BF16) G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_F32) \
+  G2B_CASE_UNGATED(BN_, ST_, EPI_ACCUM_F32) G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
   G2B_SHAPE(64, 4) G2B_SHAPE(64, 8) G2B_SHAPE(128, 3) G2B_SHAPE(128, 6) G2B_SHAPE(256, 4)
 #undef G2B_SHAPE
 #undef G2B_CASE
@@ -1562,7 +1576,7 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
 
 template <int BN, int STAGES, int EPI>
 static int launch_grouped(const CUtensorMap &ma, const CUtensorMap &mw, void *C, const int *plan, int n_groups, int Nw,
-                          int K, int ldc, int max_tiles, int *status, cudaStream_t stream) {
+                          int K, int ldc, int max_tiles, int *status, GluForm glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = Smem<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1574,7 +1588,7 @@ static int launch_grouped(const CUtensorMap &ma, const CUtensorMap &mw, void *C,
   }
   dim3 grid((Nw + BN - 1) / BN, max_tiles);
   g2b_launch(gemm_tc_grouped_kernel<BN, STAGES, EPI>, grid, dim3(THREADS), smem, stream, ma, mw, C, plan, n_groups, Nw, K,
-             ldc, status);
+             ldc, status, glu);
   return g2b_check_launch("gemm_tc (grouped)");
 }
 
@@ -1583,7 +1597,8 @@ static int launch_grouped(const CUtensorMap &ma, const CUtensorMap &mw, void *C,
 // gates and eight ups).
 extern "C" int g2b_gemm_tc_grouped(const void *A, const void *W, void *C, int rows, int n_groups, int Nw, int K,
                                    int lda, int ldc, int epi, const int *plan, int max_tiles, int *status,
-                                   cudaStream_t stream) {
+                                   float glu_limit, float glu_offset, float glu_c1, float glu_c3, cudaStream_t stream) {
+  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
   if (rows <= 0 || Nw <= 0 || n_groups <= 0 || max_tiles <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8) G2B_REFUSE("gemm_tc: K=%d and the row stride %d must be multiples of 8", K, lda);
   if (((uintptr_t)A | (uintptr_t)W) & 15) G2B_REFUSE("gemm_tc: operands must be 16-byte aligned");
@@ -1597,9 +1612,11 @@ extern "C" int g2b_gemm_tc_grouped(const void *A, const void *W, void *C, int ro
   rc = make_map(&mw, W, n_groups * Nw, K, K, 128);
   if (rc) return rc;
   if (epi == EPI_SWIGLU_BF16)
-    return launch_grouped<128, 6, EPI_SWIGLU_BF16>(ma, mw, C, plan, n_groups, Nw, K, ldc, max_tiles, status, stream);
+    return launch_grouped<128, 6, EPI_SWIGLU_BF16>(ma, mw, C, plan, n_groups, Nw, K, ldc, max_tiles, status, glu, stream);
+#ifndef G2B_GLU
   if (epi == EPI_STORE_F32)
-    return launch_grouped<128, 6, EPI_STORE_F32>(ma, mw, C, plan, n_groups, Nw, K, ldc, max_tiles, status, stream);
+    return launch_grouped<128, 6, EPI_STORE_F32>(ma, mw, C, plan, n_groups, Nw, K, ldc, max_tiles, status, glu, stream);
+#endif
   G2B_REFUSE("gemm_tc: the grouped kernel stores float or gated bfloat16, not epilogue %d", epi);
 }
 

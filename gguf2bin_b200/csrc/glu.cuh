@@ -1,0 +1,23 @@
+// The gate of a feed-forward with two input matrices, in one form with four numbers:
+//   out = g * sigmoid(g (c1 + c3 g^2)) * (u + offset),  g = min(gate, limit),  u = clamp(up, -limit, limit)
+// SiLU: limit infinite, offset 0, c1 1, c3 0.  The tanh form of GELU, 0.5 z (1 + tanh(k (z + 0.044715 z^3)))
+// with k = sqrt(2/pi), is z * sigmoid(2 k (z + 0.044715 z^3)): c1 = 2 k, c3 = 0.044715 c1.  The capped gate:
+// its limit, offset 1, c1 its slope.
+#pragma once
+
+struct GluForm {
+  float limit, offset, c1, c3;
+};
+
+__device__ __forceinline__ float glu_value(float gate, float up, const GluForm &f) {
+  const float g = fminf(gate, f.limit);
+  const float u = fminf(fmaxf(up, -f.limit), f.limit) + f.offset;
+  return g / (1.f + expf(-(g * fmaf(f.c3 * g, g, f.c1)))) * u;
+}
+
+// The same from the fast exponential and division, for epilogues that round to bfloat16.
+__device__ __forceinline__ float glu_value_fast(float gate, float up, const GluForm &f) {
+  const float g = fminf(gate, f.limit);
+  const float u = fminf(fmaxf(up, -f.limit), f.limit) + f.offset;
+  return __fdividef(g, 1.f + __expf(-(g * fmaf(f.c3 * g, g, f.c1)))) * u;
+}

@@ -1,6 +1,6 @@
 // A routed feed-forward: every token goes through `top` of a layer's small feed-forwards.
 //
-//   moe_route    scores s = softmax(z) over all experts (or sigmoid(z), each by itself) in 32-bit;
+//   moe_route    logits z (+ a bias per expert); scores s = softmax(z) over all experts (or sigmoid(z), each by itself) in 32-bit;
 //                optionally only the experts of the best groups of neighbours stay eligible; the `top` largest of s + c
 //                (c: a stored correction that steers the choice only) are chosen, ties to the
 //                lower index; the weights are the chosen experts' s as they are, or divided by
@@ -11,7 +11,8 @@
 //                output is their input); their pairs get no row.
 //   moe_gemm     one product per expert over its rows: out = A_rows . W_e^T, the rows of A
 //                gathered by the plan; with `swiglu` W_e holds gate rows then up rows and the
-//                output is silu(gate) * up.  32-bit accumulation; a row's sum runs over k in
+//                output is the gate of glu.cuh (silu(gate) * up, the
+//                capped gate, ...).  32-bit accumulation; a row's sum runs over k in
 //                ascending order whatever else is in the tile.
 //   moe_combine  y_t = sum_j weight_tj * (row of pair (t, j), or the token's own input for an
 //                expert without matrices), added in the order of j; stored, or added to what is there.
@@ -20,11 +21,11 @@
 // with atomic counters); what is computed for the pair does not: a row of a product depends on
 // that row alone, and the combination adds a token's choices in the order of the choice.
 #include "common.cuh"
+#include "glu.cuh"
+#include "join.cuh"
 #include "mma.cuh"
 
 G2B_DEFINE_LAST_ERROR
-
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 
 // Row of a gate/up matrix [2N, K] that holds gate (s = 0) or up (s = 1) row n: all gates and then all ups
 // (`blocked` = 0), or eight gates and the eight ups of the same outputs in turn (`blocked` = 1, the
@@ -76,7 +77,7 @@ extern "C" int g2b_moe_gather(const void *A, int dtype, int a_stride, const int 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float *__restrict__ z, const float *__restrict__ correction, int T, int N, int top,
                  int renormalise, int *__restrict__ idx, float *__restrict__ weight, float scale, int sigmoid,
-                 int groups, int keep) {
+                 int groups, int keep, const float *__restrict__ bias) {
   pdl_launch();
   pdl_wait();
   extern __shared__ float sm[];                 // per warp: s [N], pick [N], group scores [groups]
@@ -87,16 +88,19 @@ moe_route_kernel(const float *__restrict__ z, const float *__restrict__ correcti
   const float *zr = z + (size_t)t * N;
   if (sigmoid) {
     for (int j = lane; j < N; j += 32) {
-      s[j] = 1.f / (1.f + expf(-zr[j]));
+      s[j] = 1.f / (1.f + expf(-(zr[j] + (bias ? bias[j] : 0.f))));
       pick[j] = s[j] + (correction ? correction[j] : 0.f);
     }
   } else {
     float m = -INFINITY;
-    for (int j = lane; j < N; j += 32) m = fmaxf(m, zr[j]);
+    for (int j = lane; j < N; j += 32) {
+      s[j] = zr[j] + (bias ? bias[j] : 0.f);
+      m = fmaxf(m, s[j]);
+    }
     m = warp_max(m);
     float sum = 0.f;
     for (int j = lane; j < N; j += 32) {
-      const float e = expf(zr[j] - m);
+      const float e = expf(s[j] - m);
       s[j] = e;
       sum += e;
     }
@@ -164,7 +168,7 @@ moe_route_kernel(const float *__restrict__ z, const float *__restrict__ correcti
 
 extern "C" int g2b_moe_route(const float *z, const float *correction, int T, int N, int top, int renormalise,
                              int *idx, float *weight, float scale, int sigmoid, int groups, int keep,
-                             cudaStream_t stream) {
+                             const float *bias, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (top < 1 || top > N) G2B_REFUSE("moe_route: %d choices among %d experts", top, N);
   if (groups < 1) groups = 1;
@@ -173,7 +177,7 @@ extern "C" int g2b_moe_route(const float *z, const float *correction, int T, int
   const size_t smem = (size_t)ROUTE_WARPS * (2 * N + groups) * sizeof(float);
   if (smem > 48 * 1024) G2B_REFUSE("moe_route: %d experts are more than a block's shared memory holds", N);
   g2b_launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream, z,
-             correction, T, N, top, renormalise, idx, weight, scale, sigmoid, groups, keep);
+             correction, T, N, top, renormalise, idx, weight, scale, sigmoid, groups, keep, bias);
   return g2b_check_launch("moe_route");
 }
 
@@ -249,7 +253,7 @@ template <typename T, bool SWIGLU>
 __global__ void __launch_bounds__(128)
 moe_gemm_kernel(const T *__restrict__ A, int a_stride, const int *__restrict__ row_pair, int pairs_per_token,
                 const T *__restrict__ W, int N, int K, const int *__restrict__ plan, int n_real,
-                void *__restrict__ out, int out_f32, int blocked) {
+                void *__restrict__ out, int out_f32, int blocked, GluForm glu) {
   pdl_launch();
   pdl_wait();
   const int tile = blockIdx.y;
@@ -316,7 +320,7 @@ moe_gemm_kernel(const T *__restrict__ A, int a_stride, const int *__restrict__ r
     for (int j = 0; j < 4; ++j) {
       const int c = n0 + tx + 16 * j;
       if (c >= N) continue;
-      const float v = SWIGLU ? silu_f(acc[0][i][j]) * acc[SWIGLU ? 1 : 0][i][j] : acc[0][i][j];
+      const float v = SWIGLU ? glu_value(acc[0][i][j], acc[SWIGLU ? 1 : 0][i][j], glu) : acc[0][i][j];
       const size_t at = (size_t)(row0 + r) * N + c;
       if (out_f32) ((float *)out)[at] = v;
       else ((T *)out)[at] = from_f32<T>(v);
@@ -334,7 +338,7 @@ template <bool SWIGLU>
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(const bf16 *__restrict__ A, int a_stride, const int *__restrict__ row_pair, int pairs_per_token,
                     const bf16 *__restrict__ W, int N, int K, const int *__restrict__ plan, int n_real,
-                    void *__restrict__ out, int out_f32, int blocked) {
+                    void *__restrict__ out, int out_f32, int blocked, GluForm glu) {
   pdl_launch();
   pdl_wait();
   const int tile = blockIdx.y;
@@ -414,7 +418,7 @@ moe_gemm_mma_kernel(const bf16 *__restrict__ A, int a_stride, const int *__restr
         const int r = 16 * i + g + (f >> 1) * 8;
         const int c = n0 + warp * 16 + 8 * j + 2 * q + (f & 1);
         if (r >= rows || c >= N) continue;
-        const float v = SWIGLU ? silu_f(acc[0][i][j][f]) * acc[S - 1][i][j][f] : acc[0][i][j][f];
+        const float v = SWIGLU ? glu_value(acc[0][i][j][f], acc[S - 1][i][j][f], glu) : acc[0][i][j][f];
         const size_t at = (size_t)(row0 + r) * N + c;
         if (out_f32) ((float *)out)[at] = v;
         else ((bf16 *)out)[at] = __float2bfloat16_rn(v);
@@ -432,7 +436,7 @@ template <bool SWIGLU>
 __global__ void __launch_bounds__(256)
 moe_gemm_wide_kernel(const bf16 *__restrict__ A, int a_stride, const int *__restrict__ row_pair, int pairs_per_token,
                      const bf16 *__restrict__ W, int N, int K, const int *__restrict__ plan, int n_real,
-                     void *__restrict__ out, int out_f32, int blocked) {
+                     void *__restrict__ out, int out_f32, int blocked, GluForm glu) {
   pdl_launch();
   pdl_wait();
   constexpr int S = SWIGLU ? 2 : 1;
@@ -530,7 +534,7 @@ moe_gemm_wide_kernel(const bf16 *__restrict__ A, int a_stride, const int *__rest
         const int r = wm * 32 + 16 * i + g + (f >> 1) * 8;
         const int c = n0 + wn * 32 + 8 * j + 2 * q + (f & 1);
         if (r >= rows || c >= N) continue;
-        const float v = SWIGLU ? silu_f(acc[0][i][j][f]) * acc[S - 1][i][j][f] : acc[0][i][j][f];
+        const float v = SWIGLU ? glu_value(acc[0][i][j][f], acc[S - 1][i][j][f], glu) : acc[0][i][j][f];
         const size_t at = (size_t)(row0 + r) * N + c;
         if (out_f32) ((float *)out)[at] = v;
         else ((bf16 *)out)[at] = __float2bfloat16_rn(v);
@@ -562,7 +566,7 @@ template <typename T, bool SWIGLU>
 __global__ void __launch_bounds__(128)
 moe_gemv_kernel(const T *__restrict__ A, int a_stride, const int *__restrict__ row_pair, int pairs_per_token, int gather,
                 const int *__restrict__ idx, const T *__restrict__ W, int N, int K, const int *__restrict__ plan,
-                int n_real, void *__restrict__ out, int out_f32, int blocked) {
+                int n_real, void *__restrict__ out, int out_f32, int blocked, GluForm glu) {
   pdl_launch();
   pdl_wait();
   const int r = blockIdx.y;
@@ -600,7 +604,7 @@ moe_gemv_kernel(const T *__restrict__ A, int a_stride, const int *__restrict__ r
 #pragma unroll
   for (int j = 0; j < MV_COLS; ++j) {
     float v = warp_sum(acc[0][j]);
-    if (SWIGLU) v = silu_f(v) * warp_sum(acc[SWIGLU ? 1 : 0][j]);
+    if (SWIGLU) v = glu_value(v, warp_sum(acc[SWIGLU ? 1 : 0][j]), glu);
     if (lane == 0 && n0 + j < N) {
       const size_t at = (size_t)r * N + n0 + j;
       if (out_f32) ((float *)out)[at] = v;
@@ -614,65 +618,69 @@ extern "C" int g2b_moe_tile_rows() { return MG_BM; }
 template <typename T>
 static void launch_gemv(const void *A, int a_stride, const int *row_pair, int pairs_per_token, int gather, const int *idx,
                         const void *W, int N, int K, const int *plan, int n_real, int n_rows, int swiglu, void *out,
-                        int out_f32, int blocked, cudaStream_t stream) {
+                        int out_f32, int blocked, GluForm glu, cudaStream_t stream) {
   const dim3 grid((N + 4 * MV_COLS - 1) / (4 * MV_COLS), n_rows);
   if (swiglu)
     g2b_launch(moe_gemv_kernel<T, true>, grid, dim3(128), 0, stream, (const T *)A, a_stride, row_pair, pairs_per_token,
-               gather, idx, (const T *)W, N, K, plan, n_real, out, out_f32, blocked);
+               gather, idx, (const T *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
   else
     g2b_launch(moe_gemv_kernel<T, false>, grid, dim3(128), 0, stream, (const T *)A, a_stride, row_pair, pairs_per_token,
-               gather, idx, (const T *)W, N, K, plan, n_real, out, out_f32, blocked);
+               gather, idx, (const T *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
 }
 
 // Few rows: `row_pair` (row -> pair) and `idx` (pair -> expert) are both needed; `gather` says whether
 // row r reads A[pair / pairs_per_token] or A[r].
 extern "C" int g2b_moe_gemv(const void *A, int dtype, int a_stride, const int *row_pair, int pairs_per_token, int gather,
                             const int *idx, const void *W, int N, int K, const int *plan, int n_real, int n_rows,
-                            int swiglu, void *out, int out_f32, int blocked, cudaStream_t stream) {
+                            int swiglu, void *out, int out_f32, int blocked, float glu_limit, float glu_offset, float glu_c1,
+                            float glu_c3, cudaStream_t stream) {
+  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
   if (n_rows <= 0 || N <= 0) return 0;
   const int epl = dtype == G2B_BF16 ? 8 : 4;
   if (K % epl || a_stride % epl || (((uintptr_t)A | (uintptr_t)W) & 15))
     G2B_REFUSE("moe_gemv: K = %d or the rows' distance %d is no multiple of %d, or a pointer is off 16 bytes", K, a_stride, epl);
-  if (dtype == G2B_F32) launch_gemv<float>(A, a_stride, row_pair, pairs_per_token, gather, idx, W, N, K, plan, n_real, n_rows, swiglu, out, out_f32, blocked, stream);
-  else if (dtype == G2B_BF16) launch_gemv<bf16>(A, a_stride, row_pair, pairs_per_token, gather, idx, W, N, K, plan, n_real, n_rows, swiglu, out, out_f32, blocked, stream);
+  if (dtype == G2B_F32) launch_gemv<float>(A, a_stride, row_pair, pairs_per_token, gather, idx, W, N, K, plan, n_real, n_rows, swiglu, out, out_f32, blocked, glu, stream);
+  else if (dtype == G2B_BF16) launch_gemv<bf16>(A, a_stride, row_pair, pairs_per_token, gather, idx, W, N, K, plan, n_real, n_rows, swiglu, out, out_f32, blocked, glu, stream);
   else G2B_REFUSE("moe_gemv: unknown dtype %d", dtype);
   return g2b_check_launch("moe_gemv");
 }
 
 extern "C" int g2b_moe_gemm(const void *A, int dtype, int a_stride, const int *row_pair, int pairs_per_token,
                             const void *W, int N, int K, const int *plan, int n_real, int max_tiles, int swiglu,
-                            void *out, int out_f32, int blocked, cudaStream_t stream) {
+                            void *out, int out_f32, int blocked, float glu_limit, float glu_offset, float glu_c1,
+                            float glu_c3, cudaStream_t stream) {
+  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
   if (max_tiles <= 0 || N <= 0) return 0;
   const dim3 grid((N + MG_BN - 1) / MG_BN, max_tiles);
   if (dtype == G2B_F32) {
     if (swiglu)
       g2b_launch(moe_gemm_kernel<float, true>, grid, dim3(128), 0, stream, (const float *)A, a_stride, row_pair,
-                 pairs_per_token, (const float *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const float *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
     else
       g2b_launch(moe_gemm_kernel<float, false>, grid, dim3(128), 0, stream, (const float *)A, a_stride, row_pair,
-                 pairs_per_token, (const float *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const float *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
   } else if (dtype == G2B_BF16) {
     const bool mma = K % 8 == 0 && a_stride % 8 == 0 && (((uintptr_t)A | (uintptr_t)W) & 15) == 0;
     // many rows an expert (a prompt step): the wide tiles
     const bool wide = mma && max_tiles > 3 * n_real + 8;
     if (wide && swiglu)
       g2b_launch(moe_gemm_wide_kernel<true>, grid, dim3(256), 0, stream, (const bf16 *)A, a_stride, row_pair,
-                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
     else if (wide)
       g2b_launch(moe_gemm_wide_kernel<false>, grid, dim3(256), 0, stream, (const bf16 *)A, a_stride, row_pair,
-                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
     else if (mma && swiglu)
       g2b_launch(moe_gemm_mma_kernel<true>, grid, dim3(128), 0, stream, (const bf16 *)A, a_stride, row_pair,
-                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
     else if (mma)
       g2b_launch(moe_gemm_mma_kernel<false>, grid, dim3(128), 0, stream, (const bf16 *)A, a_stride, row_pair,
-                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
     else if (swiglu)
       g2b_launch(moe_gemm_kernel<bf16, true>, grid, dim3(128), 0, stream, (const bf16 *)A, a_stride, row_pair,
-                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
     else
       g2b_launch(moe_gemm_kernel<bf16, false>, grid, dim3(128), 0, stream, (const bf16 *)A, a_stride, row_pair,
-                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked);
+                 pairs_per_token, (const bf16 *)W, N, K, plan, n_real, out, out_f32, blocked, glu);
   } else {
     G2B_REFUSE("moe_gemm: unknown dtype %d", dtype);
   }
@@ -764,4 +772,20 @@ extern "C" int g2b_moe_combine(const float *rows, const int *pair_row, const flo
   if (T <= 0) return 0;
   g2b_launch(moe_combine_kernel, dim3(T), dim3(256), 0, stream, rows, pair_row, weight, x_self, T, top, Hw, out, accumulate);
   return g2b_check_launch("moe_combine");
+}
+
+// The combination as the sublayer result of a layer that norms it on the way in and on the way out (join.cuh):
+// y = base + sum, x += norm(y) * w (+ add), and the next sublayer's normed input.
+extern "C" int g2b_moe_combine_join(const float *rows, const int *pair_row, const float *weight, const float *base, int top,
+                                    float *x, const float *w, float eps, const float *add, int n_rows, int H,
+                                    const float *next_w, float next_eps, void *next, int dtype, cudaStream_t stream) {
+  if (n_rows <= 0 || H <= 0) return 0;
+  const JoinTail a = {w, eps, add, next_w, next_eps, next};
+  const JoinExperts from = {rows, pair_row, weight, base, top};
+  const bool aligned = !(((uintptr_t)x | (uintptr_t)rows | (uintptr_t)base | (uintptr_t)w | (uintptr_t)add | (uintptr_t)next_w |
+                          (uintptr_t)next) & 15);
+  if (dtype == G2B_F32) launch_join<float>(x, from, a, n_rows, H, aligned, stream);
+  else if (dtype == G2B_BF16) launch_join<bf16>(x, from, a, n_rows, H, aligned, stream);
+  else G2B_REFUSE("moe_combine_join: unknown dtype %d", dtype);
+  return g2b_check_launch("moe_combine_join");
 }

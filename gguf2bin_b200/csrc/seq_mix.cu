@@ -31,6 +31,7 @@
 //                         staged: rotated (then k times a constant), or made unit vectors.
 //   head_norm_gate        o / sqrt(mean(o^2) + eps) per head (times a weight), times silu(gate)
 //   gate_mul              o * sigmoid(gate) element by element, heads unpadded
+//   norm_join             x += norm(y) (+ another buffer), and the next sublayer's normed input (join.cuh)
 //   norm_add              x += y / sqrt(mean(y^2) + eps) * w, and the sum again in the compute type
 //
 // A state column (all D entries that feed one output channel) never mixes with another, so a
@@ -38,6 +39,7 @@
 // order: what it computes for a token depends on the tokens before it in the sequence only,
 // not on how they were cut into steps or on the batch.
 #include "common.cuh"
+#include "join.cuh"
 
 G2B_DEFINE_LAST_ERROR
 
@@ -1121,6 +1123,21 @@ extern "C" int g2b_norm_add(float *x, const float *y, const float *w, float eps,
   else
     G2B_REFUSE("norm_add: unknown dtype %d", dtype);
   return g2b_check_launch("norm_add");
+}
+
+// ---------------------------------------------------------------------------
+// x += norm(y) * w (+ add); the new x normed for the next sublayer (join.cuh)
+// ---------------------------------------------------------------------------
+extern "C" int g2b_norm_join(float *x, const float *y, const float *w, float eps, const float *add, int n_rows, int H,
+                             const float *next_w, float next_eps, void *next, int dtype, cudaStream_t stream) {
+  if (n_rows <= 0 || H <= 0) return 0;
+  const JoinTail a = {w, eps, add, next_w, next_eps, next};
+  const JoinRow from = {y};
+  const bool aligned = !(((uintptr_t)x | (uintptr_t)y | (uintptr_t)w | (uintptr_t)add | (uintptr_t)next_w | (uintptr_t)next) & 15);
+  if (dtype == G2B_F32) launch_join<float>(x, from, a, n_rows, H, aligned, stream);
+  else if (dtype == G2B_BF16) launch_join<bf16>(x, from, a, n_rows, H, aligned, stream);
+  else G2B_REFUSE("norm_join: unknown dtype %d", dtype);
+  return g2b_check_launch("norm_join");
 }
 
 // ---------------------------------------------------------------------------

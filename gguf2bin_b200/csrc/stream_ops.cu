@@ -366,6 +366,69 @@ extern "C" int g2b_latent_keep(const void *d, int d_stride, int rank, const floa
 }
 
 // ---------------------------------------------------------------------------
+// the two latents of a layer whose queries come from a latent too, both normed, each by a warp: the token's key
+// latent d into the page of its position (rows of `width` >= rank entries, zeros behind the rank), the query
+// latent e into rows of their own.  Either may be absent.
+// ---------------------------------------------------------------------------
+#define LPAIR_WARPS 4
+template <typename TA>
+__global__ void __launch_bounds__(LPAIR_WARPS * 32)
+latent_pair_kernel(const TA *__restrict__ d, int rank, int width, const float *__restrict__ d_w,
+                   TA *__restrict__ pages, const int *__restrict__ page_table, int P, int page_size,
+                   const int *__restrict__ tok_pos, const int *__restrict__ tok_seq, const TA *__restrict__ e, int e_rank,
+                   const float *__restrict__ e_w, TA *__restrict__ e_out, int stride, float eps, int n_tokens, int parts) {
+  pdl_launch();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * LPAIR_WARPS + warp;
+  if (item >= (long long)n_tokens * parts) return;
+  const int t = (int)(item / parts);
+  const bool keys = d && item % parts == 0;
+  const TA *src = (keys ? d : e) + (size_t)t * stride;
+  const int n = keys ? rank : e_rank;
+  const float *w = keys ? d_w : e_w;
+  TA *dst;
+  int fill = n;
+  if (keys) {
+    const int pos = tok_pos[t];
+    const int page = page_table[(size_t)tok_seq[t] * P + pos / page_size];
+    dst = pages + ((size_t)page * page_size + pos % page_size) * width;
+    fill = width;
+  } else {
+    dst = e_out + (size_t)t * e_rank;
+  }
+  float ss = 0.f;
+  for (int j = lane; j < n; j += 32) {
+    const float v = to_f32(src[j]);
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)n + eps);
+  for (int j = lane; j < fill; j += 32) dst[j] = from_f32<TA>(j < n ? (to_f32(src[j]) * inv) * w[j] : 0.f);
+}
+
+extern "C" int g2b_latent_pair(const void *d, int rank, int width, const float *d_w, void *pages, const int *page_table,
+                               int P, int page_size, const int *tok_pos, const int *tok_seq, const void *e, int e_rank,
+                               const float *e_w, void *e_out, int stride, float eps, int n_tokens, int dtype,
+                               cudaStream_t stream) {
+  const int parts = (d ? 1 : 0) + (e ? 1 : 0);
+  if (n_tokens <= 0 || !parts) return 0;
+  if (d && (rank <= 0 || width < rank || page_size <= 0)) G2B_REFUSE("latent_pair: rank %d in rows of %d", rank, width);
+  if (e && e_rank <= 0) G2B_REFUSE("latent_pair: query rank %d", e_rank);
+  const unsigned blocks = (unsigned)(((long long)n_tokens * parts + LPAIR_WARPS - 1) / LPAIR_WARPS);
+  if (dtype == G2B_F32)
+    g2b_launch(latent_pair_kernel<float>, dim3(blocks), dim3(LPAIR_WARPS * 32), 0, stream, (const float *)d, rank, width, d_w,
+               (float *)pages, page_table, P, page_size, tok_pos, tok_seq, (const float *)e, e_rank, e_w, (float *)e_out,
+               stride, eps, n_tokens, parts);
+  else if (dtype == G2B_BF16)
+    g2b_launch(latent_pair_kernel<bf16>, dim3(blocks), dim3(LPAIR_WARPS * 32), 0, stream, (const bf16 *)d, rank, width, d_w,
+               (bf16 *)pages, page_table, P, page_size, tok_pos, tok_seq, (const bf16 *)e, e_rank, e_w, (bf16 *)e_out,
+               stride, eps, n_tokens, parts);
+  else
+    G2B_REFUSE("latent_pair: unknown dtype %d", dtype);
+  return g2b_check_launch("latent_pair");
+}
+
+// ---------------------------------------------------------------------------
 // products with one small matrix per head.  W [heads * n, r] (rows of head h: h*n .. h*n+n-1).
 //   absorb: out[t, h, 0..r)  = sum_i W[h*n + i, :] * in[t, h, i]        (W_h^T applied; in has n per head)
 //   expand: out[t, h, 0..n)  = W[h*n + i, :] . in[t, h, :], times sigmoid(gate[t, h]) when gate

@@ -5,7 +5,7 @@ from __future__ import annotations
 
 GENERIC_UNITS = [("elementwise.cu", ()), ("gemm_simt.cu", ()), ("attn_generic.cu", ()),
                  ("sampling.cu", ()), ("random_init.cu", ()), ("stream_ops.cu", ()),
-                 ("seq_mix.cu", ()), ("moe.cu", ())]
+                 ("seq_mix.cu", ()), ("moe.cu", ()), ("channel_scan.cu", ())]
 
 # head sizes built ahead of time (what the tests and the benchmark use)
 HEAD_SIZES = (64, 128)
@@ -16,7 +16,7 @@ BF16_UNITS: list = []                   # bfloat16 kernels that take every size 
 
 def all_units() -> list:
     from .. import kernels_bf16  # noqa: F401  (registers the bfloat16 kernels' sources)
-    units = list(GENERIC_UNITS) + [(s, ()) for s, _ in BF16_UNITS]
+    units = list(GENERIC_UNITS) + list(BF16_UNITS)
     for src, extra in SPECIALISED_SOURCES:
         for hd in HEAD_SIZES:
             units.append((src, (f"HD={hd}",) + tuple(extra)))

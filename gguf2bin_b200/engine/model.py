@@ -67,6 +67,7 @@ class Model:
         self.head = head_class(spec.head)(spec.head, spec.vocab_size, spec.hidden_size, self.dtype,
                                           self.device)
         self.n_params = 0
+        self.rejoins = any(e.add_embedding for e in spec.schedule)
 
     # ---- construction ---------------------------------------------------------
     @classmethod
@@ -181,17 +182,32 @@ class Model:
         ws = ctx.workspace
         ctx.step_cache.clear()                     # per-step tables are rebuilt from this step's tokens
         x = ws.buffer("stream", (ctx.n_tokens, self.hidden), torch.float32)
+        # the embedding's output, kept where a later position of the schedule adds it to the stream again
+        start = ws.buffer("stream.start", (ctx.n_tokens, self.hidden), torch.float32) if self.rejoins else None
         if hasattr(self.embedding, "cache_need"):
             # an embedding that keeps something per sequence (the previous token, say) has the
             # storage of one more position behind the schedule's
             self.embedding.forward(ctx.tok_ids[:ctx.n_tokens], x, ctx, cache.view(len(self.spec.schedule)))
+        elif start is not None and getattr(self.embedding, "writes_again", False):
+            self.embedding.forward(ctx.tok_ids[:ctx.n_tokens], x, ctx, again=start)
         else:
             self.embedding.forward(ctx.tok_ids[:ctx.n_tokens], x, ctx)
+        if start is not None and not getattr(self.embedding, "writes_again", False):
+            start.copy_(x)
         schedule = self.spec.schedule
+        if schedule[0].add_embedding:
+            kernels.stream_add(x, start)
         for position, entry in enumerate(schedule):
-            # a block may leave its last elementwise step to the next block's first launch
-            ctx.next_block = self.blocks[schedule[position + 1].layer] if position + 1 < len(schedule) else None
-            self.blocks[entry.layer].forward(x, ctx, cache.view_for(position, self.spec.cache_owner(position)))
+            block, follows = self.blocks[entry.layer], position + 1 < len(schedule)
+            # a block may leave its last elementwise step to the next block's first launch, and may take along what
+            # is added to the stream in between; one that does not leaves nothing to a block behind such an addition
+            adds = follows and schedule[position + 1].add_embedding
+            ctx.next_add = start if adds else None
+            ctx.next_block = self.blocks[schedule[position + 1].layer] if follows and (
+                not adds or getattr(block, "takes_stream_add", False)) else None
+            block.forward(x, ctx, cache.view_for(position, self.spec.cache_owner(position)))
+            if ctx.next_add is not None:
+                kernels.stream_add(x, start)
         if n_want == 0:
             return None
         logits = logits_out if logits_out is not None else \

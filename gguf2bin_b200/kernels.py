@@ -8,8 +8,9 @@ device raises ``KernelError``, and a missing or unbuildable extension raises
 from __future__ import annotations
 
 import ctypes
+import math
 from ctypes import c_float, c_int, c_ulonglong, c_void_p
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -20,7 +21,8 @@ __all__ = ["KernelError", "KernelBuildError", "embed_rows", "rmsnorm", "qknorm_r
            "attention", "sample_rows", "sample_filtered", "recent_set", "seed_slots", "embed_pair_norm",
            "canon_conv", "norm_canon_single", "latent_keep", "head_product", "head_gate", "gated_add", "xielu",
            "proj_norm_rope_cache", "rotate_heads", "short_conv", "state_scan", "head_norm_gate", "gate_mul",
-           "norm_add", "norm_shift", "scan_gates_step", "scan_gates_max", "state_readout", "pool_update", "moe_route", "moe_plan", "moe_gemm", "moe_gemv", "moe_gather", "moe_gemm_tc", "moe_combine", "moe_combine_norm_add", "moe_tile_rows", "tanh_norm", "scaled_join", "relu2", "selective_scan", "diff_combine"]
+           "norm_add", "norm_shift", "scan_gates_step", "scan_gates_max", "state_readout", "pool_update", "moe_route", "moe_plan", "moe_gemm", "moe_gemv", "moe_gather", "moe_gemm_tc", "moe_combine", "moe_combine_norm_add", "moe_tile_rows", "tanh_norm", "scaled_join", "relu2", "selective_scan", "diff_combine", "GluForm", "norm_join", "moe_combine_join", "latent_pair",
+           "channel_scan", "stream_add"]
 
 F32, BF16 = 0, 1
 EPI_STORE_F32, EPI_STORE_BF16, EPI_ACCUM_F32 = 0, 1, 2
@@ -125,14 +127,56 @@ def _call(f, *args) -> None:
 # ---------------------------------------------------------------------------
 # elementwise.cu
 # ---------------------------------------------------------------------------
-def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-    """out[t] = table[ids[t]] widened to float32, times ``scale``.  ids int32 [T], out float32 [T, H]."""
+class GluForm(NamedTuple):
+    """The gate of a two-input feed-forward: g sigmoid(g (c1 + c3 g^2)) (u + offset) with g = min(gate, limit) and
+    u = clamp(up, -limit, limit) (csrc/glu.cuh).  ``SILU`` is the form that every gated kernel has built in."""
+    limit: float = math.inf
+    offset: float = 0.0
+    c1: float = 1.0
+    c3: float = 0.0
+
+    @classmethod
+    def gelu_tanh(cls) -> "GluForm":
+        """0.5 z (1 + tanh(k (z + 0.044715 z^3))), k = sqrt(2 / pi), as z sigmoid(2 k (z + 0.044715 z^3))."""
+        c1 = 2.0 * math.sqrt(2.0 / math.pi)
+        return cls(c1=c1, c3=0.044715 * c1)
+
+    @classmethod
+    def capped(cls, limit: float, slope: float) -> "GluForm":
+        return cls(limit=float(limit), offset=1.0, c1=float(slope))
+
+
+SILU = GluForm()
+_GLU_TYPES = [c_float, c_float, c_float, c_float]
+
+
+def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0, positions=None,
+               tok_pos=None, again=None) -> None:
+    """out[t] = table[ids[t]] widened to float32, times ``scale``.  ids int32 [T], out float32 [T, H].
+    ``positions`` [n, H] (the table's dtype): row ``tok_pos[t]`` of it is added.  ``again``: a second copy of
+    the rows, float32 [T, H]."""
     _need(ids, torch.int32, "ids")
     _need(out, torch.float32, "out")
+    if again is not None:
+        _need(again, torch.float32, "second copy")
+    if positions is not None and (positions.dtype != table.dtype or positions.shape[1] != table.shape[1]
+                                  or not positions.is_contiguous()):
+        raise KernelError("embed_rows: the position table must have the token table's dtype and width")
     V, H = table.shape
     f = _fn("elementwise.cu", "g2b_embed_rows",
-            [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
-    _call(f, _ptr(table), _code(table.dtype), _ptr(ids), _ptr(out), out.shape[0], H, V, float(scale), _stream())
+            [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p,
+             c_void_p])
+    _call(f, _ptr(table), _code(table.dtype), _ptr(ids), _ptr(out), out.shape[0], H, V, float(scale), _ptr(positions),
+          _ptr(tok_pos) if positions is not None else None, positions.shape[0] if positions is not None else 0,
+          _ptr(again), _stream())
+
+
+def stream_add(x32: torch.Tensor, y32: torch.Tensor) -> None:
+    """x += y, both float32 of one shape: what a model adds to its stream between two layers where no kernel of
+    the layers takes it along."""
+    _need(x32, torch.float32, "stream")
+    _need(y32, torch.float32, "addend")
+    x32.add_(y32)
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor,
@@ -241,14 +285,17 @@ def cache_write(k, v, n_kv_heads, head_dim, tok_pos, tok_seq, page_table, cache_
           _ptr(cache_pages), page_size, _stream())
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int, limit: float = 0.0, alpha: float = 1.0) -> None:
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int, limit: float = 0.0, alpha: float = 1.0,
+           form: GluForm = SILU) -> None:
     """out[t, i] = silu(g_i) * u_i from a fused projection whose columns alternate
     ``block`` gates and ``block`` ups.  ``limit`` > 0: the capped form, g = min(g, limit),
-    u = clamp(u, -limit, limit), out = g * sigmoid(alpha * g) * (u + 1)."""
+    u = clamp(u, -limit, limit), out = g * sigmoid(alpha * g) * (u + 1).  ``form``: any other gate."""
     T, I = out.shape
+    if limit > 0:
+        form = GluForm.capped(limit, alpha)
     f = _fn("elementwise.cu", "g2b_swiglu",
-            [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_void_p])
-    _call(f, _ptr(gate_up), _code(gate_up.dtype), T, I, block, _ptr(out), float(limit), float(alpha), _stream())
+            [c_void_p, c_int, c_int, c_int, c_int, c_void_p, *_GLU_TYPES, c_void_p])
+    _call(f, _ptr(gate_up), _code(gate_up.dtype), T, I, block, _ptr(out), *form, _stream())
 
 
 def norm_shift(x32, w, mu, kept, ctx, eps: float, h_out, hs_out) -> None:
@@ -374,6 +421,23 @@ def latent_keep(d, norm_w, eps, pages, h, ring, taps, ctx) -> None:
           ctx.page_table.shape[1] if d is not None else 0, ctx.page_size, _ptr(h) if ring is not None else None, _ptr(ring),
           h.shape[1] if ring is not None else 0, int(taps), _code(ref.dtype), _ptr(ctx.tok_pos),
           _ptr(ctx.tok_seq), _ptr(ctx.seq_slots), ref.shape[0], _stream())
+
+
+def latent_pair(d, width: int, d_w, pages, e, e_w, e_out, eps: float, ctx) -> None:
+    """rmsnorm(d) * d_w (d [T, rank]) into the latent pages at the tokens' positions, rows of ``width`` entries with zeros
+    behind the rank; rmsnorm(e) * e_w (e [T, n]) into ``e_out`` [T, n].  d and e are columns of one buffer."""
+    if d.dtype != e.dtype or d.stride(0) != e.stride(0) or d.stride(1) != 1 or e.stride(1) != 1:
+        raise KernelError("latent_pair: both latents are columns of one buffer")
+    if pages.dtype != d.dtype or e_out.dtype != d.dtype or not e_out.is_contiguous() or pages.shape[-1] != width:
+        raise KernelError("latent_pair: pages and output must have the input's dtype, pages rows of the given width")
+    _need(d_w, torch.float32, "latent norm weight")
+    _need(e_w, torch.float32, "query latent norm weight")
+    f = _fn("stream_ops.cu", "g2b_latent_pair",
+            [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
+             c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_void_p])
+    _call(f, _ptr(d), d.shape[1], width, _ptr(d_w), _ptr(pages), _ptr(ctx.page_table), ctx.page_table.shape[1],
+          ctx.page_size, _ptr(ctx.tok_pos), _ptr(ctx.tok_seq), _ptr(e), e.shape[1], _ptr(e_w), _ptr(e_out), d.stride(0),
+          float(eps), d.shape[0], _code(d.dtype), _stream())
 
 
 def head_product(x, w, out, heads: int, expand: bool, gate=None) -> None:
@@ -504,6 +568,13 @@ def attention_notices(what: str, head_dim: int, page_size: int, compute_dtype: t
     return []
 
 
+def padded_head_size(head_dim: int) -> int:
+    """The smallest head size of the tensor-core attention kernels that holds ``head_dim`` entries; ``head_dim``
+    itself where none does."""
+    from . import kernels_bf16
+    return min((s for s in kernels_bf16.FAST_HEAD_SIZES if s >= head_dim), default=head_dim)
+
+
 # ---------------------------------------------------------------------------
 # attention
 # ---------------------------------------------------------------------------
@@ -573,11 +644,11 @@ def normed_product(x32, eps, w, out, gate_block=None) -> bool:
     return False
 
 
-def gate_up_fused(h, w_gate_up, mid, block) -> bool:
-    """silu(gate) * up computed inside the product's epilogue; False when no kernel takes
-    the case (the caller then runs the product and ``swiglu`` separately)."""
+def gate_up_fused(h, w_gate_up, mid, block, form: GluForm = SILU) -> bool:
+    """silu(gate) * up (or another gate of ``GluForm``'s kind) computed inside the product's epilogue; False when
+    no kernel takes the case (the caller then runs the product and ``swiglu`` separately)."""
     if h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16:
-        return (_bf16 or _bf16_mod()).gate_up_bf16(h, w_gate_up, mid, block)
+        return (_bf16 or _bf16_mod()).gate_up_bf16(h, w_gate_up, mid, block, form)
     return False
 
 
@@ -891,6 +962,35 @@ def norm_add(x32, y32, w, eps, cast_out=None) -> None:
           _code(cast_out.dtype) if cast_out is not None else F32, _stream())
 
 
+def _join_args(x32, norm_w, base32, add32, next_norm, next_out):
+    for t, what in ((norm_w, "norm weight"), (base32, "base"), (add32, "addend")):
+        if t is not None:
+            _need(t, torch.float32, what)
+    for t in (base32, add32, next_out):
+        if t is not None and (tuple(t.shape) != tuple(x32.shape) or not t.is_contiguous()):
+            raise KernelError("norm_join: every buffer must be contiguous and of the stream's shape")
+    if (next_norm is None) != (next_out is None):
+        raise KernelError("norm_join: the next norm and its output go together")
+    if next_norm is None:
+        return None, 0.0
+    next_w, next_eps = next_norm
+    if next_w is not None:
+        _need(next_w, torch.float32, "next norm weight")
+    return next_w, float(next_eps)
+
+
+def norm_join(x32, y32, norm_w, eps: float, next_norm=None, next_out=None, add32=None) -> None:
+    """x += y / sqrt(mean(y^2) + eps) * norm_w (+ ``add32``), float32; ``next_norm`` = (weight or None, eps) with
+    ``next_out`` [T, H] (compute type): the new rows also leave normed, the next sublayer's input."""
+    _need(x32, torch.float32, "stream")
+    _need(y32, torch.float32, "sublayer output")
+    next_w, next_eps = _join_args(x32, norm_w, y32, add32, next_norm, next_out)
+    f = _fn("seq_mix.cu", "g2b_norm_join",
+            [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p])
+    _call(f, _ptr(x32), _ptr(y32), _ptr(norm_w), float(eps), _ptr(add32), x32.shape[0], x32.shape[1], _ptr(next_w), next_eps,
+          _ptr(next_out), _code(next_out.dtype) if next_out is not None else F32, _stream())
+
+
 def selective_scan(x, dt32, dt_bias, bc, a, skip, z, state, ctx, out, out_scale: float = 1.0) -> None:
     """A state-space recurrence with a decay per state entry, over the step's tokens in order:
     dt = softplus(dt32 + dt_bias); S[c, n] = exp(dt_c a[c, n]) S[c, n] + dt_c x_c B_n; y_c = sum_n S[c, n] C_n;
@@ -935,8 +1035,8 @@ def moe_tile_rows() -> int:
 
 
 def moe_route(z32, correction, top: int, renormalise: bool, idx, weight, scale: float = 1.0, score: str = "softmax",
-              groups: int = 1, keep: int = 1) -> None:
-    """softmax over all experts of ``z32`` [T, N] (``score`` "sigmoid": every logit's sigmoid by itself);
+              groups: int = 1, keep: int = 1, bias=None) -> None:
+    """``bias`` (float32 [N], if given) is added to the logits ``z32``; then softmax over all experts of ``z32`` [T, N] (``score`` "sigmoid": every logit's sigmoid by itself);
     the ``top`` largest of score + correction chosen (``idx`` int32 [T, top]); ``weight`` float32 [T, top]
     their scores (divided by their sum + 1e-20 when ``renormalise``), times ``scale``.  ``groups`` > 1: the
     experts are that many equal groups of neighbours, a group counts as the sum of its two best scores,
@@ -947,9 +1047,9 @@ def moe_route(z32, correction, top: int, renormalise: bool, idx, weight, scale: 
     _need(idx, torch.int32, "idx")
     _need(weight, torch.float32, "weight")
     f = _fn("moe.cu", "g2b_moe_route", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
-                                        c_int, c_int, c_int, c_void_p])
+                                        c_int, c_int, c_int, c_void_p, c_void_p])
     _call(f, _ptr(z32), _ptr(correction), z32.shape[0], z32.shape[1], top, 1 if renormalise else 0, _ptr(idx),
-          _ptr(weight), float(scale), 1 if score == "sigmoid" else 0, int(groups), int(keep), _stream())
+          _ptr(weight), float(scale), 1 if score == "sigmoid" else 0, int(groups), int(keep), _ptr(bias), _stream())
 
 
 def moe_plan(idx, n_real: int, max_tiles: int, plan, row_pair, pair_row) -> None:
@@ -960,22 +1060,22 @@ def moe_plan(idx, n_real: int, max_tiles: int, plan, row_pair, pair_row) -> None
 
 
 def moe_gemm(a, row_pair, pairs_per_token: int, w, n_out: int, plan, n_real: int, max_tiles: int, swiglu: bool,
-             out, blocked: bool = False) -> None:
+             out, blocked: bool = False, form: GluForm = SILU) -> None:
     """Per expert e over its rows: out[row] = a[source of row] . w[e]^T; ``w`` [E, n_out (x2 with
     ``swiglu``: gate rows then up rows, or, ``blocked``, eight gates and eight ups in turn), K];
-    ``row_pair`` None: row r reads a[r]."""
+    ``row_pair`` None: row r reads a[r].  ``form``: the gate of ``swiglu`` (default SiLU)."""
     if w.dtype != a.dtype:
         raise KernelError("moe_gemm: activations and expert matrices must have one dtype")
     f = _fn("moe.cu", "g2b_moe_gemm",
             [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int,
-             c_void_p, c_int, c_int, c_void_p])
+             c_void_p, c_int, c_int, *_GLU_TYPES, c_void_p])
     _call(f, _ptr(a), _code(a.dtype), _dense_rows(a, "a"), _ptr(row_pair), pairs_per_token, _ptr(w), n_out,
           a.shape[1], _ptr(plan), n_real, max_tiles, 1 if swiglu else 0, _ptr(out),
-          1 if out.dtype == torch.float32 else 0, 1 if blocked else 0, _stream())
+          1 if out.dtype == torch.float32 else 0, 1 if blocked else 0, *form, _stream())
 
 
 def moe_gemv(a, row_pair, pairs_per_token: int, gather: bool, idx, w, n_out: int, plan, n_real: int, n_rows: int,
-             swiglu: bool, out, blocked: bool = False) -> bool:
+             swiglu: bool, out, blocked: bool = False, form: GluForm = SILU) -> bool:
     """``moe_gemm`` for a step of few rows: a warp per four output columns of one row, the weight rows
     streamed with 16-byte loads.  ``gather``: row r reads a[pair / pairs_per_token], else a[r].  False
     when the sizes do not allow 16-byte loads (the caller then takes ``moe_gemm``)."""
@@ -986,10 +1086,10 @@ def moe_gemv(a, row_pair, pairs_per_token: int, gather: bool, idx, w, n_out: int
         return False
     f = _fn("moe.cu", "g2b_moe_gemv",
             [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
-             c_int, c_void_p, c_int, c_int, c_void_p])
+             c_int, c_void_p, c_int, c_int, *_GLU_TYPES, c_void_p])
     _call(f, _ptr(a), _code(a.dtype), _dense_rows(a, "a"), _ptr(row_pair), pairs_per_token, 1 if gather else 0,
           _ptr(idx), _ptr(w), n_out, a.shape[1], _ptr(plan), n_real, n_rows, 1 if swiglu else 0, _ptr(out),
-          1 if out.dtype == torch.float32 else 0, 1 if blocked else 0, _stream())
+          1 if out.dtype == torch.float32 else 0, 1 if blocked else 0, *form, _stream())
     return True
 
 
@@ -1003,13 +1103,14 @@ def moe_gather(a, row_pair, pairs_per_token: int, plan, n_real: int, out) -> Non
           out.shape[0], a.shape[1], _ptr(out), _stream())
 
 
-def moe_gemm_tc(a_rows, w, n_out: int, plan, n_real: int, max_tiles: int, swiglu: bool, out) -> bool:
+def moe_gemm_tc(a_rows, w, n_out: int, plan, n_real: int, max_tiles: int, swiglu: bool, out,
+                form: GluForm = SILU) -> bool:
     """``moe_gemm`` on the tcgen05 kernel: ``a_rows`` [rows, K] bfloat16, gathered in the plan's order;
     ``w`` [E, n_out (x2, blocked, with ``swiglu``), K]; out float32 [rows, n_out], or bfloat16 with
     ``swiglu``.  False when the sizes do not fit the kernel."""
     if a_rows.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         return False
-    return (_bf16 or _bf16_mod()).gemm_tc_grouped(a_rows, w, n_out, plan, n_real, max_tiles, swiglu, out)
+    return (_bf16 or _bf16_mod()).gemm_tc_grouped(a_rows, w, n_out, plan, n_real, max_tiles, swiglu, out, form)
 
 
 def moe_combine(rows32, pair_row, weight, x_self32, top: int, out32, accumulate: bool = False) -> None:
@@ -1035,3 +1136,61 @@ def moe_combine_norm_add(rows32, pair_row, weight, x32, norm_w, eps: float, top:
     _call(f, _ptr(rows32), _ptr(pair_row), _ptr(weight), _ptr(x32), _ptr(norm_w), eps, x32.shape[0], top,
           x32.shape[1], _ptr(cast_out), _code(cast_out.dtype) if cast_out is not None else F32, _stream())
     return True
+
+
+def moe_combine_join(rows32, pair_row, weight, base32, top: int, x32, norm_w, eps: float, next_norm=None, next_out=None,
+                     add32=None) -> None:
+    """``norm_join`` with y = base + sum_j weight[t, j] * rows32[pair_row[t, j]] (the token's own x where a pair has no
+    row): a routed feed-forward's result, on top of ``base32`` (a shared expert's; None: nothing), joins the stream."""
+    for t, what in ((rows32, "experts' rows"), (x32, "stream"), (weight, "weights")):
+        _need(t, torch.float32, what)
+    next_w, next_eps = _join_args(x32, norm_w, base32, add32, next_norm, next_out)
+    f = _fn("moe.cu", "g2b_moe_combine_join",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p,
+             c_float, c_void_p, c_int, c_void_p])
+    _call(f, _ptr(rows32), _ptr(pair_row), _ptr(weight), _ptr(base32), top, _ptr(x32), _ptr(norm_w), float(eps), _ptr(add32),
+          x32.shape[0], x32.shape[1], _ptr(next_w), next_eps, _ptr(next_out),
+          _code(next_out.dtype) if next_out is not None else F32, _stream())
+
+
+# ---------------------------------------------------------------------------
+# channel_scan.cu: a matrix state per head with a decay per key channel
+# ---------------------------------------------------------------------------
+CHANNEL_TILES_WIDE_FROM = 4096      # tokens of a step from which its segments are the work list's 128-row tiles
+
+
+def channel_scan(q, k, v, low, w_low, bias32, state, ctx, out32, heads: int, qk_dim: int, v_dim: int, q_scale: float,
+                 tau: float) -> None:
+    """S <- diag(a_t) S + k_t v_t^T, o_t = S^T (q_t q_scale) per head, a_t = sigmoid(w_low low_t + bias)^(1/tau) per key
+    channel; over the step's tokens in order, 32-bit.  q, k [T, heads*qk_dim], v [T, heads*v_dim], low [T, R]: rows of
+    wider buffers in the compute type; ``w_low`` [heads*qk_dim, R] (R a multiple of 8), ``bias32`` float32; ``state``
+    float32 [slots, heads, v_dim, qk_dim] is read and left up to date; ``out32`` float32 [T, heads*v_dim].
+    A prompt step walks the segments of its sequences (the tiles of the attention's work list) side by side."""
+    T, R = q.shape[0], w_low.shape[1]
+    for t, what in ((state, "state"), (out32, "scan output"), (bias32, "decay bias")):
+        _need(t, torch.float32, what)
+    if tuple(state.shape[1:]) != (heads, v_dim, qk_dim) or tuple(out32.shape) != (T, heads * v_dim) \
+            or w_low.shape[0] != heads * qk_dim or low.shape[1] != R or not w_low.is_contiguous():
+        raise KernelError(f"channel_scan: state {tuple(state.shape)}, output {tuple(out32.shape)} or decay matrix "
+                          f"{tuple(w_low.shape)} do not fit {heads} heads of {v_dim} columns of {qk_dim}")
+    if any(t.dtype != q.dtype for t in (k, v, low, w_low)):
+        raise KernelError("channel_scan: q, k, v, low and the decay matrix must have one dtype")
+    f = _fn("channel_scan.cu", "g2b_channel_scan",
+            [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+             c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
+             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
+    tiles, n_tiles, rows, scratch = None, 0, 0, (None,) * 5
+    if T > ctx.n_seqs:
+        wide = T >= CHANNEL_TILES_WIDE_FROM
+        tiles, n_tiles, rows = (ctx.attn_tiles_wide, ctx.n_attn_tiles_wide, 128) if wide else \
+            (ctx.attn_tiles, ctx.n_attn_tiles, 64)
+        segments = T // rows + ctx.n_seqs + 1
+        ws, f32 = ctx.workspace, torch.float32
+        scratch = tuple(ws.buffer(f"channel.{n}", (T, heads * qk_dim), f32) for n in ("q", "k", "decay")) + (
+            ws.buffer("channel.states", (segments, heads, v_dim, qk_dim), f32),
+            ws.buffer("channel.decays", (segments, heads, qk_dim), f32))
+        count_launches(3 if n_tiles > ctx.n_seqs else 1)
+    _call(f, _code(q.dtype), _ptr(q), _dense_rows(q, "q"), _ptr(k), _dense_rows(k, "k"), _ptr(v), _dense_rows(v, "v"),
+          _ptr(low), _dense_rows(low, "low"), _ptr(w_low), _ptr(bias32), heads, qk_dim, v_dim, R, float(q_scale),
+          1.0 / float(tau), _ptr(state), _ptr(ctx.seq_slots), _ptr(ctx.seq_meta), T, ctx.n_seqs, _ptr(tiles), n_tiles, rows,
+          *(_ptr(t) for t in scratch), _ptr(out32), _stream())

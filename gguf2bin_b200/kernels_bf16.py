@@ -8,7 +8,7 @@ import torch
 
 from .csrc import units
 from . import kernels
-from .kernels import KernelError, _call, _fn, _ptr, _stream
+from .kernels import SILU, _GLU_TYPES, KernelError, _call, _fn, _ptr, _stream
 
 FAST_HEAD_SIZES = (64, 128)          # head sizes the tensor-core attention kernels are written for
 DECODE_CHUNK_KEYS = 256              # keys per CTA of the decode kernel (attn_decode.cu)
@@ -18,7 +18,9 @@ units.SPECIALISED_SOURCES[:] = [("attn_decode.cu", ()), ("attn_decode.cu", ("ATT
                                 ("attn_decode_noalloc.cu", ()),
                                 ("attn_prefill.cu", ()), ("attn_prefill_tc.cu", ()),
                                 ("attn_prefill_tc_split.cu", ()), ("attn_pool_decode.cu", ())]
-units.BF16_UNITS[:] = [("gemm_small.cu", ()), ("gemm_tc.cu", ())]
+# a build with G2B_GLU holds the gated epilogue alone, in the form that a launch gives (other gates than SiLU)
+GLU_DEFINES = ("G2B_GLU",)
+units.BF16_UNITS[:] = [("gemm_small.cu", ()), ("gemm_tc.cu", ()), ("gemm_small.cu", GLU_DEFINES), ("gemm_tc.cu", GLU_DEFINES)]
 
 
 SMALL_M = 64                         # rows the weight-streaming product takes
@@ -32,11 +34,12 @@ def _small_ok(a: torch.Tensor, w: torch.Tensor) -> bool:
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def _gemm_small(a, w, out, epi) -> None:
+def _gemm_small(a, w, out, epi, form=SILU) -> None:
     f = _fn("gemm_small.cu", "g2b_gemm_small",
-            [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+            [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, *_GLU_TYPES, c_void_p],
+            defines=GLU_DEFINES if form != SILU else ())
     _call(f, _ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
-          w.stride(0), out.stride(0), epi, _stream())
+          w.stride(0), out.stride(0), epi, *form, _stream())
 
 
 def normed_product(x32: torch.Tensor, eps: float, w: torch.Tensor, out: torch.Tensor, gated: bool) -> bool:
@@ -112,7 +115,7 @@ def _tc_ok(a: torch.Tensor, w: torch.Tensor) -> bool:
             and w.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def _gemm_tc(a, w, out, epi, bn: int = 0, stages: int = 0, persistent=False, defines=()) -> None:
+def _gemm_tc(a, w, out, epi, bn: int = 0, stages: int = 0, persistent=False, defines=(), form=SILU) -> None:
     """bn = 0 lets the launcher pick the tile shape from the sizes.  persistent: one CTA per SM
     walks over the tiles with two accumulators (shapes (128, 6) and (256, 4)); persistent = 2:
     pairs of CTAs on 256 x 256 tiles (shapes (256, 6) and (256, 4)); persistent = 3: at most 128
@@ -120,13 +123,14 @@ def _gemm_tc(a, w, out, epi, bn: int = 0, stages: int = 0, persistent=False, def
     ``defines``: another build of the source (the tests' build whose waits run out)."""
     f = _fn("gemm_tc.cu", "g2b_gemm_tc",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_int, c_int, c_void_p, c_void_p], defines=tuple(defines))
+             c_int, c_int, c_void_p, *_GLU_TYPES, c_void_p],
+            defines=tuple(defines) + (GLU_DEFINES if form != SILU else ()))
     _call(f, _ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
           w.stride(0), out.stride(0), epi, bn, stages, int(persistent),
-          _ptr(_status_word(a.device)), _stream())
+          _ptr(_status_word(a.device)), *form, _stream())
 
 
-def gemm_tc_grouped(a_rows, w, n_out: int, plan, n_groups: int, max_tiles: int, swiglu: bool, out) -> bool:
+def gemm_tc_grouped(a_rows, w, n_out: int, plan, n_groups: int, max_tiles: int, swiglu: bool, out, form=SILU) -> bool:
     """One product per group of rows on the tcgen05 kernel (see ``g2b_gemm_tc_grouped``); False when
     the sizes or alignments do not fit (the caller has other kernels)."""
     K = a_rows.shape[1]
@@ -141,10 +145,10 @@ def gemm_tc_grouped(a_rows, w, n_out: int, plan, n_groups: int, max_tiles: int, 
         return False
     f = _fn("gemm_tc.cu", "g2b_gemm_tc_grouped",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-             c_void_p, c_void_p])
+             c_void_p, *_GLU_TYPES, c_void_p], defines=GLU_DEFINES if swiglu and form != SILU else ())
     _call(f, _ptr(a_rows), _ptr(w), _ptr(out), a_rows.shape[0], n_groups, n_w, K, a_rows.stride(0), out.stride(0),
           EPI_SWIGLU_BF16 if swiglu else EPI_STORE_F32, _ptr(plan), max_tiles, _ptr(_status_word(a_rows.device)),
-          _stream())
+          *form, _stream())
     return True
 
 
@@ -289,17 +293,17 @@ def _sm_count(device) -> int:
     return _sm_counts[key]
 
 
-def gate_up_bf16(h: torch.Tensor, w_gate_up: torch.Tensor, mid: torch.Tensor, block: int) -> bool:
-    """mid = silu(gate) * up with the gate computed in the product's epilogue; takes fused
+def gate_up_bf16(h: torch.Tensor, w_gate_up: torch.Tensor, mid: torch.Tensor, block: int, form=SILU) -> bool:
+    """mid = silu(gate) * up (or the gate of ``form``) with the gate computed in the product's epilogue; takes fused
     matrices whose rows alternate 8 gates / 8 ups."""
     if block != 8 or mid.dtype != torch.bfloat16 or mid.stride(1) != 1 or w_gate_up.shape[0] % 16:
         return False
     choice, bn, stages, persistent = _route(h, w_gate_up, mid)
     if choice == "small":
-        _gemm_small(h, w_gate_up, mid, EPI_SWIGLU_BF16)
+        _gemm_small(h, w_gate_up, mid, EPI_SWIGLU_BF16, form)
         return True
     if choice == "tc":
-        _gemm_tc(h, w_gate_up, mid, EPI_SWIGLU_BF16, bn, stages, persistent)
+        _gemm_tc(h, w_gate_up, mid, EPI_SWIGLU_BF16, bn, stages, persistent, form=form)
         return True
     return False
 

@@ -61,6 +61,8 @@ class StepContext:
     n_attn_tiles_wide: int = 0
     step_cache: dict = field(default_factory=dict)   # tensors derived once per step (cleared by the model)
     next_block: Optional[object] = None              # the block that runs after the one running now (None: the last)
+    next_add: Optional[torch.Tensor] = None          # what is added to the stream before the next block; a block that
+                                                     # takes it along (``takes_stream_add``) sets this back to None
 
     def rope_table(self, inv_freq: torch.Tensor, mult: float = 1.0) -> torch.Tensor:
         """(cos, sin) of every token's position times ``inv_freq``, both times ``mult``, computed once

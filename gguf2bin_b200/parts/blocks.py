@@ -7,7 +7,9 @@ short convolution over time in front of the mixer, and an optional feed-forward.
 ``parallel_shift``: h = norm(x); x += mixer(shift(h)) + feed_forward(h): one norm, both sublayers read
 it, and the mixer's copy is mixed with the token before, channel by channel.
 ``parallel_scaled``: h = norm(x); x += s1 * mixer(h) + s2 * feed_forward(h): one norm of any registered kind,
-both sublayers read it, and each result is multiplied by a learned number per channel before the sum."""
+both sublayers read it, and each result is multiplied by a learned number per channel before the sum.
+``sandwich_norm``: x += norm(mixer(norm(x))); x += norm(feed_forward(norm(x))): an RMS norm on either side of every
+sublayer."""
 from __future__ import annotations
 
 import torch
@@ -538,7 +540,125 @@ class ParallelScaledBlock:
             kernels.scaled_join(x32, y1, self.mixer_scale, y2, self.ffn_scale)
 
 
+class SandwichNormBlock:
+    """``sandwich_norm``: x <- x + norm1b(mixer(norm1(x))), then x <- x + norm2b(feed_forward(norm2(x))); four RMS norms of
+    the layer's kind, statistics and the sum in 32-bit.  A layer may have no feed-forward.  Any mixer and feed-forward of
+    the library fit: a sublayer stores into a 32-bit buffer where it can (``forward_store``, ``forward_into``) and adds
+    into a cleared one where it cannot.
+
+    One launch a sublayer does everything between two products: the result's norm, the sum, what the model adds to the
+    stream in front of the next block (``StepContext.next_add``), and the next sublayer's norm, the next block's among
+    them (``StepContext.step_cache`` hands its rows over).  For routed experts that launch also sums the experts."""
+    takes_stream_add = True
+
+    def __init__(self, layer: LayerSpec, hidden_size: int, dtype: torch.dtype, device):
+        self.names = dict(layer.block["names"])
+        self.hidden, self.dtype = int(hidden_size), dtype
+
+        def norm(spec):
+            made = norm_class(spec)(spec, hidden_size, dtype, device)
+            if not isinstance(made, RMSNorm):
+                raise ConfigError("sandwich_norm: the norms around a sublayer are rmsnorms")
+            return made
+        ffn_norm = layer.ffn_norm or layer.norm
+        self.mixer_norm, self.mixer_out_norm = norm(layer.norm), norm(layer.norm)
+        self.mixer = mixer_class(layer.mixer)(layer.mixer, hidden_size, dtype, device)
+        self.feed_forward = self.ffn_norm = self.ffn_out_norm = None
+        if layer.feed_forward is not None:
+            self.ffn_norm, self.ffn_out_norm = norm(ffn_norm), norm(ffn_norm)
+            self.feed_forward = feed_forward_class(layer.feed_forward)(layer.feed_forward, hidden_size, dtype, device)
+
+    @classmethod
+    def expected(cls, layer: LayerSpec, hidden_size: int) -> dict:
+        names = dict(layer.block["names"])
+        ffn_norm = layer.ffn_norm or layer.norm
+        out = {}
+        for key in ("mixer_norm", "mixer_out_norm"):
+            out.update(norm_class(layer.norm).expected(layer.norm, hidden_size, names[key]))
+        out.update(mixer_class(layer.mixer).expected(layer.mixer, hidden_size))
+        second = {}
+        for key in ("ffn_norm", "ffn_out_norm"):
+            second.update(norm_class(ffn_norm).expected(ffn_norm, hidden_size, names[key]))
+        if layer.feed_forward is not None:
+            out.update(second)
+            out.update(feed_forward_class(layer.feed_forward).expected(layer.feed_forward, hidden_size))
+        else:        # a checkpoint may carry the second pair of norms all the same; they are unused
+            out.update({k: Expected(e.shape, e.init, optional=True) for k, e in second.items()})
+        return out
+
+    def bind(self, tensors: dict) -> None:
+        n = self.names
+        self.mixer_norm.bind(tensors[n["mixer_norm"]])
+        self.mixer_out_norm.bind(tensors[n["mixer_out_norm"]])
+        self.mixer.bind(tensors)
+        if self.feed_forward is not None:
+            self.ffn_norm.bind(tensors[n["ffn_norm"]])
+            self.ffn_out_norm.bind(tensors[n["ffn_out_norm"]])
+            self.feed_forward.bind(tensors)
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def parts(self) -> tuple:
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_out_norm, self.ffn_norm, self.feed_forward,
+                                 self.ffn_out_norm) if p is not None)
+
+    def weights(self):
+        for part in self.parts():
+            yield from getattr(part, "weights", tuple)()
+
+    def notices(self) -> list:
+        return [line for part in self.parts() for line in getattr(part, "notices", list)()]
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(part, "graph_safe", False) for part in self.parts())
+
+    def forward(self, x32: torch.Tensor, ctx, cache_view) -> None:
+        T, H, ws = x32.shape[0], self.hidden, ctx.workspace
+        key = ("sandwich_norm.normed", x32.data_ptr())
+        h = ctx.step_cache.pop(key, None)
+        if h is None:                              # the block in front left no normed rows
+            h = ws.buffer("sandwich.normed", (T, H), self.dtype)
+            self.mixer_norm.forward(x32, h)
+        # what the block's last launch takes along: the addition in front of the next block, and that block's norm
+        follower = ctx.next_block if isinstance(ctx.next_block, SandwichNormBlock) else None
+        after, add, ctx.next_add = (follower.mixer_norm if follower is not None else None), ctx.next_add, None
+        y = ws.buffer("sandwich.result", (T, H), torch.float32)
+        ff = self.feed_forward
+        if hasattr(self.mixer, "forward_store"):
+            self.mixer.forward_store(h, ctx, cache_view, y)
+        else:
+            y.zero_()
+            self.mixer.forward(h, ctx, cache_view, y)
+        # both sublayers have read h by the time the launch that overwrites it runs (stream order)
+        if ff is None:
+            self._join(x32, y, self.mixer_out_norm, after, h, add)
+        else:
+            self._join(x32, y, self.mixer_out_norm, self.ffn_norm, h, None)
+            norm, nxt = self.ffn_out_norm, self._next(after)
+            if not (isinstance(ff, RoutedExperts) and ff.forward_norm_join(
+                    h, ctx, y, x32, norm.weight, norm.eps, nxt, h if nxt is not None else None, add)):
+                if hasattr(ff, "forward_into"):
+                    ff.forward_into(h, ctx, y)
+                else:
+                    y.zero_()
+                    ff.forward(h, ctx, y)
+                self._join(x32, y, norm, after, h, add)
+        if follower is not None:
+            ctx.step_cache[key] = h
+
+    @staticmethod
+    def _next(norm):
+        return None if norm is None else (norm.weight, norm.eps)
+
+    def _join(self, x32, y, norm, after, h, add) -> None:
+        """x += norm(y) (+ add), and the rows that the norm ``after`` makes of the new x into h."""
+        kernels.norm_join(x32, y, norm.weight, norm.eps, self._next(after), h if after is not None else None, add)
+
+
 register_block("prenorm", PreNormBlock)
+register_block("sandwich_norm", SandwichNormBlock)
 register_block("parallel_scaled", ParallelScaledBlock)
 register_block("parallel_shift", ParallelShiftBlock)
 register_block("gated_prenorm", GatedPreNormBlock)

@@ -2,7 +2,8 @@
 into logits.
 
 ``token_embedding``: row ``id`` of the table, widened to float32
-(src/l5_model.c:488-492 of AnonymoDGH/gguf2bin), times ``scale`` when the spec has one.
+(src/l5_model.c:488-492 of AnonymoDGH/gguf2bin), times ``scale`` when the spec has one; with
+``positions`` (a name, and ``n_positions``) plus that table's row of the token's position.
 ``lm_head``: logits = h . W^T in float32, W a matrix of its own or, when ``tied``, the
 embedding's table (src/l5_model.c:600-605: without an output tensor the reference
 multiplies by the token-embedding matrix).
@@ -24,26 +25,39 @@ from .registry import register_embedding, register_head
 
 class TokenEmbedding:
     graph_safe = True          # its step only launches kernels: may be replayed from a CUDA graph
+    writes_again = True        # takes a second buffer for its rows
 
     def __init__(self, spec: PartSpec, vocab_size: int, hidden_size: int, dtype: torch.dtype, device):
         self.name = spec["name"]
         self.vocab, self.hidden = int(vocab_size), int(hidden_size)
         self.scale = float(spec.get("scale") if spec.get("scale") is not None else 1.0)
         self.table: Optional[torch.Tensor] = None      # [vocab, hidden]; a tied head multiplies by it
+        self.positions_name = spec.get("positions")
+        self.positions: Optional[torch.Tensor] = None  # [n_positions, hidden]
+        self._rows = None                              # what the kernel reads: the table in the positions' type
 
     @classmethod
     def expected(cls, spec: PartSpec, vocab_size: int, hidden_size: int) -> dict:
-        return {spec["name"]: Expected((int(vocab_size), int(hidden_size)))}
+        out = {spec["name"]: Expected((int(vocab_size), int(hidden_size)))}
+        if spec.get("positions"):
+            out[spec["positions"]] = Expected((int(spec["n_positions"]), int(hidden_size)))
+        return out
 
     def bind(self, tensors: dict) -> None:
-        self.table = tensors[self.name].contiguous()
+        self.table = self._rows = tensors[self.name].contiguous()
+        if self.positions_name:
+            self.positions = tensors[self.positions_name].contiguous()
+            if self.positions.dtype != self.table.dtype:          # one of them is kept in 32-bit: read both so
+                self.positions, self._rows = self.positions.float(), self.table.float()
 
     def weights(self):
-        return (self.table,)
+        return tuple(t for t in (self.table, self.positions, self._rows if self._rows is not self.table else None)
+                     if t is not None)
 
-    def forward(self, tok_ids: torch.Tensor, out32: torch.Tensor, ctx) -> None:
-        """out32[t] = table[tok_ids[t]] * scale as float32; out32 is [T, hidden]."""
-        kernels.embed_rows(self.table, tok_ids, out32, self.scale)
+    def forward(self, tok_ids: torch.Tensor, out32: torch.Tensor, ctx, again=None) -> None:
+        """out32[t] = table[tok_ids[t]] * scale (+ positions[its position]) as float32; out32 is [T, hidden].
+        ``again``: a second buffer that gets the same rows."""
+        kernels.embed_rows(self._rows, tok_ids, out32, self.scale, self.positions, ctx.tok_pos, again)
 
 
 class LMHead:

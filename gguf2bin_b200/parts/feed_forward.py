@@ -8,6 +8,9 @@ A width that is no multiple of eight keeps the plain order (all gates, then all 
 With ``limit`` the gate is capped from above and the up value from both sides, the gate's sigmoid
 takes a slope and the up value an offset of one: g = min(gate x, limit), u = clamp(up x, -limit,
 limit), down( g sigmoid(alpha g) (u + 1) ), ``alpha`` 1.702 unless the spec says otherwise.
+``activation`` = "gelu_tanh": the gate's activation is the tanh form of GELU, 0.5 z (1 + tanh(sqrt(2/pi) (z +
+0.044715 z^3))), instead of SiLU.  All of these are one form with four numbers (``kernels.GluForm``), which the
+products' epilogues take.
 """
 from __future__ import annotations
 
@@ -18,6 +21,17 @@ from ..config.specs import ConfigError, PartSpec
 from ..weights.loader import Expected
 from .fused import normed_linear
 from .registry import feed_forward_class, register_feed_forward
+
+
+def gate_form(what: str, activation, limit: float, alpha: float) -> kernels.GluForm:
+    """The gate of a two-input feed-forward as the kernels take it."""
+    if limit < 0:
+        raise ConfigError(f"{what}: limit must be positive (or absent)")
+    if activation not in (None, "silu", "gelu_tanh") or (limit and activation is not None):
+        raise ConfigError(f"{what}: the activation is 'silu' or 'gelu_tanh', or a limit makes it the capped gate")
+    if limit:
+        return kernels.GluForm.capped(limit, alpha)
+    return kernels.GluForm.gelu_tanh() if activation == "gelu_tanh" else kernels.SILU
 
 
 class SwiGLU:
@@ -32,8 +46,7 @@ class SwiGLU:
         self.w_gate_up = self.w_down = None
         self.limit = float(spec.get("limit") or 0.0)
         self.alpha = float(spec.get("alpha") if spec.get("alpha") is not None else 1.702)
-        if self.limit < 0:
-            raise ConfigError("swiglu: limit must be positive (or absent)")
+        self.form = gate_form("swiglu", spec.get("activation"), self.limit, self.alpha)
 
     @classmethod
     def expected(cls, spec: PartSpec, hidden_size: int) -> dict:
@@ -57,7 +70,7 @@ class SwiGLU:
     def absorb_norm_weight(self, norm) -> bool:
         """As ``GQAAttention.absorb_norm_weight``, into the columns of the gate/up matrix."""
         if self.dtype != torch.bfloat16 or self.w_gate_up.dtype != torch.bfloat16 or self.block != 8 \
-                or not hasattr(norm, "give_up_weight") or self.limit:
+                or not hasattr(norm, "give_up_weight") or self.form != kernels.SILU:
             return False
         w = norm.give_up_weight()
         self.w_gate_up = (self.w_gate_up.float() * w.to(self.w_gate_up.device)[None, :]).to(torch.bfloat16).contiguous()
@@ -68,18 +81,25 @@ class SwiGLU:
                 + kernels.product_notices("feed-forward down", self.w_down, self.dtype))
 
     def forward(self, h: torch.Tensor, ctx, residual32: torch.Tensor) -> None:
+        self._run(h, ctx, residual32, True)
+
+    def forward_into(self, h: torch.Tensor, ctx, out32: torch.Tensor) -> None:
+        """Stores the result instead of adding it."""
+        self._run(h, ctx, out32, False)
+
+    def _run(self, h, ctx, out32, accumulate: bool) -> None:
         T = h.shape[0]
         ws = ctx.workspace
         mid = ws.buffer("ffn.mid", (T, self.inter), self.dtype)
-        if self.limit or not kernels.gate_up_fused(h, self.w_gate_up, mid, self.block):
+        if not kernels.gate_up_fused(h, self.w_gate_up, mid, self.block, self.form):
             gu = ws.buffer("ffn.gate_up", (T, 2 * self.inter), self.dtype)
             kernels.linear(h, self.w_gate_up, gu)
-            kernels.swiglu(gu, mid, self.block, self.limit, self.alpha)
-        kernels.linear(mid, self.w_down, residual32, accumulate=True)
+            kernels.swiglu(gu, mid, self.block, form=self.form)
+        kernels.linear(mid, self.w_down, out32, accumulate=accumulate)
 
     def forward_from_stream(self, x32: torch.Tensor, norm, ctx, residual32: torch.Tensor) -> None:
         """The same with the block's norm folded into the gate/up product."""
-        if self.limit:                 # the fused epilogues know the plain SiLU gate only
+        if self.form != kernels.SILU:  # the products that norm their own input know the plain SiLU gate only
             h = ctx.workspace.buffer("fused.normed", tuple(x32.shape), self.dtype)
             norm.forward(x32, h)
             return self.forward(h, ctx, residual32)
@@ -177,7 +197,9 @@ class RoutedExperts:
     instead of a softmax.  ``groups`` with ``groups_kept``: the experts form that many equal groups of
     neighbours, a group counts as the sum of its two largest scores, and only experts of the best
     ``groups_kept`` groups can be chosen.  ``shared``: the spec of one more feed-forward (any registered kind)
-    that runs for every token and is added.
+    that runs for every token and is added.  ``router_bias``: a stored vector that is part of the logits (name
+    ``router_bias``).  ``limit`` (with ``alpha``, 1.702 unless the spec says otherwise): the experts' gate is the capped
+    one of ``swiglu``.
 
     A step groups its (token, choice) pairs by expert on the device (``moe_plan``) and runs one
     grouped product for gate and up with the activation in its epilogue and one for down; nothing
@@ -195,7 +217,10 @@ class RoutedExperts:
         if self.E < 0 or self.I < 0 or not (1 <= self.top <= self.E + self.I) or self.E > 1024:
             raise ConfigError(f"routed_experts: {self.top} choices among {self.E} + {self.I} experts")
         self.names = dict(spec["names"])
-        self.w_router = self.correction = self.w_gate_up = self.w_down = None
+        self.w_router = self.correction = self.router_bias = self.w_gate_up = self.w_down = None
+        self.has_bias = bool(spec.get("router_bias") or False)
+        self.form = gate_form("routed_experts", None, float(spec.get("limit") or 0.0),
+                              float(spec.get("alpha") if spec.get("alpha") is not None else 1.702))
         self.blocked = False
         self.scale = float(spec.get("scale") if spec.get("scale") is not None else 1.0)
         self.score = spec.get("score") or "softmax"
@@ -216,6 +241,8 @@ class RoutedExperts:
         out = {n["router"]: Expected((E + I, hidden_size))}
         if spec.get("correction"):
             out[n["correction"]] = Expected((E + I,))
+        if spec.get("router_bias"):
+            out[n["router_bias"]] = Expected((E + I,))
         for e in range(E):
             out[n["gate"].format(e)] = Expected((inter, hidden_size))
             out[n["up"].format(e)] = Expected((inter, hidden_size))
@@ -231,6 +258,8 @@ class RoutedExperts:
         self.w_router = tensors[n["router"]].contiguous()
         if self.has_correction:
             self.correction = tensors[n["correction"]].to(torch.float32).contiguous()
+        if self.has_bias:
+            self.router_bias = tensors[n["router_bias"]].to(torch.float32).contiguous()
         if self.E:
             mats = [tensors[n[k].format(e)] for e in range(self.E) for k in ("gate", "up", "down")]
             common = torch.float32 if any(m.dtype == torch.float32 for m in mats) else mats[0].dtype
@@ -248,7 +277,8 @@ class RoutedExperts:
             self.w_down = torch.stack([tensors[n["down"].format(e)].to(common) for e in range(self.E)]).contiguous()
 
     def weights(self):
-        own = tuple(t for t in (self.w_router, self.correction, self.w_gate_up, self.w_down) if t is not None)
+        own = tuple(t for t in (self.w_router, self.correction, self.router_bias, self.w_gate_up, self.w_down)
+                    if t is not None)
         return own + (tuple(self.shared.weights()) if self.shared is not None else ())
 
     def notices(self) -> list:
@@ -286,6 +316,23 @@ class RoutedExperts:
         rows32, pair_row, weight = self._experts(h, ctx)
         return kernels.moe_combine_norm_add(rows32, pair_row, weight, x32, norm_w, eps, self.top, cast_out)
 
+    def forward_norm_join(self, h: torch.Tensor, ctx, y32, x32, norm_w, eps: float, next_norm, next_out, add32) -> bool:
+        """For a block that norms on both sides of the feed-forward: the experts' sum, on top of the shared expert's
+        result (``y32`` is its buffer), is normed, joins the stream and leaves the next sublayer's input in one pass
+        (``kernels.norm_join``).  False (nothing done) where an expert's output is its input."""
+        if self.I:
+            return False
+        if self.shared is not None:
+            if hasattr(self.shared, "forward_into"):
+                self.shared.forward_into(h, ctx, y32)
+            else:
+                y32.zero_()
+                self.shared.forward(h, ctx, y32)
+        rows32, pair_row, weight = self._experts(h, ctx)
+        kernels.moe_combine_join(rows32, pair_row, weight, y32 if self.shared is not None else None, self.top, x32, norm_w,
+                                 eps, next_norm, next_out, add32)
+        return True
+
     def _experts(self, h: torch.Tensor, ctx):
         """Routing, plan and the experts' products: (rows, pair -> row, weights)."""
         T, ws, top, E = h.shape[0], ctx.workspace, self.top, self.E
@@ -294,7 +341,7 @@ class RoutedExperts:
         idx = ws.buffer("moe.idx", (T, top), torch.int32)
         weight = ws.buffer("moe.weight", (T, top), torch.float32)
         kernels.moe_route(z, self.correction, top, self.renormalise, idx, weight, self.scale, self.score, self.groups,
-                          self.groups_kept)
+                          self.groups_kept, self.router_bias)
         n_pairs = T * top
         tile = kernels.moe_tile_rows()
         max_tiles = -(-n_pairs // tile) + E               # every expert's last tile may be part full
@@ -315,14 +362,14 @@ class RoutedExperts:
             done = False
             if few:
                 done = kernels.moe_gemv(a, row_pair, top, True, idx, self.w_gate_up, self.inter, plan, E, n_pairs,
-                                        True, mid, self.blocked)
+                                        True, mid, self.blocked, self.form)
             elif many and self.hidden % 8 == 0:
                 rows = ws.buffer("moe.gathered", (n_pairs, self.hidden), wt)
                 kernels.moe_gather(a, row_pair, top, plan, E, rows)
-                done = kernels.moe_gemm_tc(rows, self.w_gate_up, self.inter, plan, E, max_tiles, True, mid)
+                done = kernels.moe_gemm_tc(rows, self.w_gate_up, self.inter, plan, E, max_tiles, True, mid, self.form)
             if not done:
                 kernels.moe_gemm(a, row_pair, top, self.w_gate_up, self.inter, plan, E, max_tiles, True, mid,
-                                 self.blocked)
+                                 self.blocked, self.form)
             done = False
             if few:
                 done = kernels.moe_gemv(mid, row_pair, top, False, idx, self.w_down, self.hidden, plan, E, n_pairs,

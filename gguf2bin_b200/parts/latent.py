@@ -10,7 +10,11 @@ panel per page: ``KVNeed(planes=1)``), and applies U_v to each head's weighted s
 Options, each a parameter of the spec: ``sink`` (a learned logit per head that joins the
 softmax's denominator and nothing else), ``out_gate`` (each head's output times the sigmoid of
 a linear function of u), ``shared_kv`` (no down-projection: the layer attends over the latents
-that the schedule entry's ``cache_of`` layer stored), ``scale``.
+that the schedule entry's ``cache_of`` layer stored), ``scale``, ``q_rank`` (queries come from a latent of their own
+of that many numbers, c_q = rmsnorm(W_dq u) * w_q, q = W_uq c_q; names ``q_down``, ``q_down_norm``, and ``q`` for W_uq),
+``window`` (a token sees the last ``window`` positions, its own among them), ``pad_rank`` (bfloat16: latents of a rank
+below a size that the tensor-core attention kernels take lie in rows of that size, zero-filled, as do the
+up-projections' columns; scores and sums are what they were).
 
 Scores, softmax and the latent's norm are 32-bit; products accumulate in 32-bit.
 
@@ -65,13 +69,23 @@ class LatentAttention:
             raise ConfigError("latent_attention: heads, sizes and rank must be positive")
         if self.rank > 512:
             raise ConfigError(f"latent_attention: kv_rank {self.rank} is more than the attention kernels' 512")
+        self.q_rank = int(spec.get("q_rank") or 0)
+        self.window = int(spec.get("window") or 0)
+        if spec.get("pad_rank") and not self.q_rank:
+            raise ConfigError("latent_attention: padded ranks go with a query latent")
+        if self.q_rank < 0 or self.window < 0 or (self.q_rank and (self.shared_kv or self.has_gate)):
+            raise ConfigError("latent_attention: q_rank and window are positive or absent; a query latent goes with "
+                              "neither shared latents nor a gate")
         self.dtype, self.device = dtype, device
         self.names = dict(spec["names"])
-        # columns of the fused input product: queries, then the latent (unless shared), then the gates
-        self.n_q = self.nh * self.dk
-        self.n_c = 0 if self.shared_kv else self.rank
+        self.own_rank = self.rank                 # what the down-projection makes; ``rank``: a row of the pages
+        if spec.get("pad_rank") and dtype == torch.bfloat16:
+            self.rank = kernels.padded_head_size(self.rank)
+        # columns of the fused input product: queries (or their latent), then the latent (unless shared), then the gates
+        self.n_q = self.q_rank or self.nh * self.dk
+        self.n_c = 0 if self.shared_kv else self.own_rank
         self.n_g = self.nh if self.has_gate else 0
-        self.w_in = self.w_o = self.w_uk = self.w_uv = self.c_norm = self.sink = None
+        self.w_in = self.w_o = self.w_uk = self.w_uv = self.c_norm = self.sink = self.w_uq = self.q_norm = None
         self.fold_k = self.fold_v = False
 
     # ---- weights -------------------------------------------------------------
@@ -79,8 +93,12 @@ class LatentAttention:
     def expected(cls, spec: PartSpec, hidden_size: int) -> dict:
         n = dict(spec["names"])
         nh, dk, dv, r = spec["n_heads"], spec["qk_dim"], spec["v_dim"], spec["kv_rank"]
-        out = {n["q"]: Expected((nh * dk, hidden_size)), n["up_k"]: Expected((nh * dk, r)),
+        qr = spec.get("q_rank")
+        out = {n["q"]: Expected((nh * dk, qr or hidden_size)), n["up_k"]: Expected((nh * dk, r)),
                n["up_v"]: Expected((nh * dv, r)), n["o"]: Expected((hidden_size, nh * dv))}
+        if qr:
+            out[n["q_down"]] = Expected((qr, hidden_size))
+            out[n["q_down_norm"]] = Expected((qr,), init="scale")
         if not (spec.get("shared_kv") or False):
             out[n["down"]] = Expected((r, hidden_size))
             out[n["down_norm"]] = Expected((r,), init="scale")
@@ -93,18 +111,27 @@ class LatentAttention:
     def bind(self, tensors: dict) -> None:
         n = self.names
         w_q, w_o = tensors[n["q"]], tensors[n["o"]]
+        up_k, up_v = tensors[n["up_k"]], tensors[n["up_v"]]
+        if self.rank != self.own_rank:             # columns of zeros behind the rank
+            up_k, up_v = (torch.nn.functional.pad(t, (0, self.rank - self.own_rank)) for t in (up_k, up_v))
+        q_in = self.q_rank or self.hidden          # what the queries are a product of
         folding = self.dtype == torch.bfloat16 and w_q.dtype == torch.bfloat16 and w_o.dtype == torch.bfloat16
-        self.fold_k = folding and folds(self.rank, self.dk, self.nh, self.hidden)
+        self.fold_k = folding and folds(self.rank, self.dk, self.nh, q_in)
         self.fold_v = folding and folds(self.rank, self.dv, self.nh, self.hidden)
         if self.fold_k:
             # W_q'[h] = U_k[h]^T W_q[h]: [rank, qk_dim] x [qk_dim, width] per head; the queries then
             # come out of the input product in latent coordinates, `rank` numbers per head
-            uk = tensors[n["up_k"]].double().view(self.nh, self.dk, self.rank)
-            wq = w_q.double().view(self.nh, self.dk, self.hidden)
-            w_q = torch.einsum("hdr,hdw->hrw", uk, wq).reshape(self.nh * self.rank, self.hidden) \
+            uk = up_k.double().view(self.nh, self.dk, self.rank)
+            wq = w_q.double().view(self.nh, self.dk, q_in)
+            w_q = torch.einsum("hdr,hdw->hrw", uk, wq).reshape(self.nh * self.rank, q_in) \
                 .to(torch.bfloat16).contiguous()
-            self.n_q = self.nh * self.rank
+            if not self.q_rank:
+                self.n_q = self.nh * self.rank
         parts = [w_q]
+        if self.q_rank:
+            self.w_uq = w_q.contiguous()
+            self.q_norm = tensors[n["q_down_norm"]].to(torch.float32).contiguous()
+            parts = [tensors[n["q_down"]]]
         if not self.shared_kv:
             parts.append(tensors[n["down"]])
             self.c_norm = tensors[n["down_norm"]].to(torch.float32).contiguous()
@@ -118,35 +145,40 @@ class LatentAttention:
         self.w_in = torch.cat([p.to(common) for p in parts], dim=0).contiguous()
         if self.fold_v:
             # W_o'[:, h] = W_o[:, h] U_v[h]: [width, v_dim] x [v_dim, rank] per head
-            uv = tensors[n["up_v"]].double().view(self.nh, self.dv, self.rank)
+            uv = up_v.double().view(self.nh, self.dv, self.rank)
             wo = w_o.double().view(self.hidden, self.nh, self.dv)
             self.w_o = torch.einsum("whv,hvr->whr", wo, uv).reshape(self.hidden, self.nh * self.rank) \
                 .to(torch.bfloat16).contiguous()
         else:
             self.w_o = w_o.contiguous()
-            self.w_uv = tensors[n["up_v"]].to(self.dtype).contiguous()
+            self.w_uv = up_v.to(self.dtype).contiguous()
         if not self.fold_k:
-            self.w_uk = tensors[n["up_k"]].to(self.dtype).contiguous()
+            self.w_uk = up_k.to(self.dtype).contiguous()
         if self.has_sink:
             self.sink = tensors[n["sink"]].to(torch.float32).contiguous()
 
     def weights(self):
-        return [t for t in (self.w_in, self.w_o, self.w_uk, self.w_uv, self.c_norm, self.sink)
+        return [t for t in (self.w_in, self.w_o, self.w_uk, self.w_uv, self.c_norm, self.sink, self.w_uq, self.q_norm)
                 if t is not None]
 
     def notices(self) -> list:
         from ..cache.storage import PAGE_SIZE
         return (kernels.product_notices("latent attention input", self.w_in, self.dtype)
+                + kernels.product_notices("latent attention queries", self.w_uq, self.dtype)
                 + kernels.product_notices("latent attention output", self.w_o, self.dtype)
                 + kernels.attention_notices("latent attention", self.rank, PAGE_SIZE, self.dtype))
 
     # ---- cache ---------------------------------------------------------------
     def cache_need(self):
-        return None if self.shared_kv else KVNeed(1, self.rank, 0, planes=1)
+        return None if self.shared_kv else KVNeed(1, self.rank, self.window, planes=1)
 
     # ---- step ----------------------------------------------------------------
     def forward(self, u: torch.Tensor, ctx, view: KVView, residual32: torch.Tensor) -> None:
         self._run(u, ctx, view, residual32, True, None)
+
+    def forward_store(self, u: torch.Tensor, ctx, view: KVView, out32: torch.Tensor) -> None:
+        """Stores the mixer's result instead of adding it."""
+        self._run(u, ctx, view, out32, False, None)
 
     def forward_into(self, u: torch.Tensor, ctx, view: KVView, out32: torch.Tensor, keep=None) -> None:
         """Stores the mixer's result instead of adding it.  ``keep`` = (rows, ring, taps): the
@@ -192,7 +224,14 @@ class LatentAttention:
         d = proj[:, self.n_q:self.n_q + self.n_c] if self.n_c else None
         gate = proj[:, self.n_q + self.n_c:self.n_q + self.n_c + self.n_g] if self.n_g else None
         rows, ring, taps = keep if keep is not None else (None, None, 0)
-        if d is not None or ring is not None:
+        if self.q_rank:
+            if ring is not None:
+                kernels.latent_keep(None, None, 0.0, None, rows, ring, taps, ctx)
+            cq = ws.buffer("latent.cq", (T, self.q_rank), self.dtype)
+            kernels.latent_pair(d, self.rank, self.c_norm, view.pages, q, self.q_norm, cq, self.eps, ctx)
+            q = ws.buffer("latent.uq", (T, self.w_uq.shape[0]), self.dtype)
+            kernels.linear(cq, self.w_uq, q)
+        elif d is not None or ring is not None:
             kernels.latent_keep(d, self.c_norm, self.eps, view.pages if d is not None else None,
                                 rows, ring, taps, ctx)
         if self.fold_k:
@@ -202,7 +241,7 @@ class LatentAttention:
             self._per_head(q, self.w_uk, qa, False, None)
         mix = ws.buffer("latent.mix", (T, self.nh * self.rank), self.dtype)
         # with U_v folded into the output matrix the heads' gate is the attention's last step
-        kernels.attention(qa, mix, view.pages, ctx, self.nh, 1, self.rank, view.page_size, 0, self.scale,
+        kernels.attention(qa, mix, view.pages, ctx, self.nh, 1, self.rank, view.page_size, self.window, self.scale,
                           sink=self.sink, planes=1, gate=gate if self.fold_v else None)
         if self.fold_v:
             o = mix

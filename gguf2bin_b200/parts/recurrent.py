@@ -37,6 +37,11 @@ entry n: S[c, n] = exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n, y_c = sum_n S[c, n]
 output product.  The state [inner, state_dim] is 32-bit and starts at zero; the convolution's last
 inputs are a ring by position.  Step sizes, decays and the recurrence are 32-bit.
 
+``gla``: linear attention with a decay per key channel that depends on the token.  q = W_q h * qk_dim^-1/2, k = W_k h,
+v = W_v h; a = sigmoid(z)^(1/tau) with z = W_a2 (W_a1 h) + b, one number per head and key channel (W_a1's rows, the
+rank of the decay, come from the checkpoint); per head S_t = diag(a_t) S_{t-1} + k_t v_t^T, o_t = S_t^T q_t; each head's
+o divided by its root mean square, times a weight over v_dim shared by the heads, times silu(W_g h); output product.
+
 ``parallel``: several mixers that read the same input; the result is the sum of theirs, each times
 its ``out_scale``.  A branch is any registered mixer that takes ``out_scale``.
 
@@ -52,7 +57,8 @@ import torch
 from .. import kernels
 from ..cache.storage import StateNeed
 from ..config.specs import ConfigError, PartSpec
-from ..weights.loader import Expected
+from ..weights.loader import Expected, FreeSize
+from ..weights.safetensors_io import WeightsError
 from .registry import mixer_class, position_class, register_mixer
 
 
@@ -463,6 +469,85 @@ class MLSTMMixer:
         kernels.linear(og, self.w_o, residual32, accumulate=accumulate)
 
 
+class GatedLinearAttention:
+    graph_safe = True
+    LOW_RANK = 16             # rank of the decay's matrices where random weights are made (a checkpoint brings its own)
+
+    def __init__(self, spec: PartSpec, hidden_size: int, dtype: torch.dtype, device):
+        self.H, self.D, self.V = int(spec["n_heads"]), int(spec["qk_dim"]), int(spec["v_dim"])
+        self.hidden, self.dtype, self.device = int(hidden_size), dtype, device
+        if min(self.H, self.D, self.V) <= 0 or self.D > 512:
+            raise ConfigError("gla: heads, qk_dim (at most 512) and v_dim must be positive")
+        self.tau, self.eps = float(spec["tau"]), float(spec["eps"])
+        if not self.tau > 0:
+            raise ConfigError("gla: tau must be positive")
+        self.out_scale = float(spec.get("out_scale") if spec.get("out_scale") is not None else 1.0)
+        self.names = dict(spec["names"])
+        self.w_in = self.w_low = self.b_low = self.norm_w = self.w_o = None
+        self.low_at = 0
+
+    @classmethod
+    def expected(cls, spec: PartSpec, hidden_size: int) -> dict:
+        n = dict(spec["names"])
+        H, D, V = int(spec["n_heads"]), int(spec["qk_dim"]), int(spec["v_dim"])
+        rank = FreeSize(cls.LOW_RANK)
+        return {n["q"]: Expected((H * D, hidden_size)), n["k"]: Expected((H * D, hidden_size)),
+                n["v"]: Expected((H * V, hidden_size)), n["gate"]: Expected((H * V, hidden_size)),
+                n["a1"]: Expected((rank, hidden_size)), n["a2"]: Expected((H * D, rank)), n["a_bias"]: Expected((H * D,)),
+                n["norm"]: Expected((V,), init="scale"), n["o"]: Expected((hidden_size, H * V))}
+
+    def bind(self, tensors: dict) -> None:
+        n = self.names
+        a1, a2 = tensors[n["a1"]], tensors[n["a2"]]
+        rank = a1.shape[0]
+        if a2.shape[1] != rank:
+            raise WeightsError(f"{n['a1']} has {rank} rows, {n['a2']} {a2.shape[1]} columns: they must be equal")
+        if rank > 1024:
+            raise WeightsError(f"{n['a1']}: a decay rank of {rank} (at most 1024)")
+        # one product: q | k | v | gate | (zeros) | a1 | (zeros): the decay's columns start on 16 bytes and are a multiple
+        # of eight, as are a2's
+        w = _padded_rows([tensors[n[k]] for k in ("q", "k", "v", "gate")])
+        low = _padded_rows([a1])
+        self.low_at, self.rank = w.shape[0], low.shape[0]
+        common = _common_dtype([w, low])
+        self.w_in = torch.cat([w.to(common), low.to(common)], dim=0).contiguous()
+        self.w_low = torch.nn.functional.pad(a2, (0, self.rank - rank)).to(self.dtype).contiguous()
+        self.b_low = tensors[n["a_bias"]].to(torch.float32).contiguous()
+        self.norm_w = tensors[n["norm"]].to(torch.float32).contiguous()
+        self.w_o = tensors[n["o"]].contiguous()
+
+    def weights(self):
+        return (self.w_in, self.w_low, self.b_low, self.norm_w, self.w_o)
+
+    def notices(self) -> list:
+        return (kernels.product_notices("gated linear attention input", self.w_in, self.dtype)
+                + kernels.product_notices("gated linear attention output", self.w_o, self.dtype))
+
+    def cache_need(self):
+        return StateNeed((self.H, self.V, self.D), torch.float32)
+
+    def forward(self, h: torch.Tensor, ctx, view, residual32: torch.Tensor) -> None:
+        self._run(h, ctx, view, residual32, True)
+
+    def forward_store(self, h: torch.Tensor, ctx, view, out32: torch.Tensor) -> None:
+        """Stores the result instead of adding it."""
+        self._run(h, ctx, view, out32, False)
+
+    def _run(self, h, ctx, view, residual32, accumulate: bool) -> None:
+        T, ws = h.shape[0], ctx.workspace
+        nq, nv = self.H * self.D, self.H * self.V
+        proj = ws.buffer("gla.in", (T, self.w_in.shape[0]), self.dtype)
+        kernels.linear(h, self.w_in, proj)
+        o32 = ws.buffer("gla.o", (T, nv), torch.float32)
+        kernels.channel_scan(proj[:, :nq], proj[:, nq:2 * nq], proj[:, 2 * nq:2 * nq + nv],
+                             proj[:, self.low_at:self.low_at + self.rank], self.w_low, self.b_low, view.states, ctx, o32,
+                             self.H, self.D, self.V, self.D ** -0.5, self.tau)
+        og = ws.buffer("gla.gated", (T, nv), self.dtype)
+        kernels.head_norm_gate(o32, self.H, self.V, self.norm_w, self.eps, proj[:, 2 * nq + nv:2 * nq + 2 * nv],
+                               self.out_scale, og)
+        kernels.linear(og, self.w_o, residual32, accumulate=accumulate)
+
+
 class ParallelMixer:
     """Branches side by side on one input; what each stores is kept under ``<branch>.<name>``."""
 
@@ -527,6 +612,7 @@ class ParallelMixer:
 
 register_mixer("retention", RetentionMixer)
 register_mixer("gated_delta", GatedDeltaMixer)
+register_mixer("gla", GatedLinearAttention)
 register_mixer("parallel", ParallelMixer)
 register_mixer("ssd", SSDMixer)
 register_mixer("mlstm", MLSTMMixer)

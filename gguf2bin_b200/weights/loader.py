@@ -22,6 +22,11 @@ import torch
 from .safetensors_io import SafetensorsFile, WeightsError, open_model_files
 
 
+class FreeSize(int):
+    """A size that the configuration does not give: a checkpoint's tensor may have any positive one there, and
+    the part that binds it takes it from the tensor.  The number itself is what random weights are made with."""
+
+
 @dataclass(frozen=True)
 class Expected:
     """A tensor the model needs.  ``init`` tells the random-weights writer how to fill
@@ -42,13 +47,18 @@ def runtime_dtype(stored: torch.dtype, compute: torch.dtype) -> torch.dtype:
     return torch.bfloat16
 
 
+def shape_fits(found: tuple, expected: tuple) -> bool:
+    return len(found) == len(expected) and all(
+        f > 0 if isinstance(e, FreeSize) else f == e for f, e in zip(found, expected))
+
+
 def check_names_and_shapes(expected: Mapping[str, Expected],
                            found: Mapping[str, tuple]) -> None:
     """Raises one ``WeightsError`` listing all missing, unexpected and misshapen tensors."""
     missing = [n for n, e in expected.items() if n not in found and not e.optional]
     unexpected = [n for n in found if n not in expected]
     wrong = [(n, tuple(found[n]), tuple(e.shape)) for n, e in expected.items()
-             if n in found and tuple(found[n]) != tuple(e.shape)]
+             if n in found and not shape_fits(tuple(found[n]), tuple(e.shape))]
     if not (missing or unexpected or wrong):
         return
     lines = ["weights do not match the model:"]
