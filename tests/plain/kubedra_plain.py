@@ -214,6 +214,71 @@ def forward(cfg, t, tokens, layers_out=None, watch=None):
     return centred_norm(x, t["final.norm"], eps) @ t["embed"].T
 
 
+def routing_margin(z, top):
+    """How far one token's last chosen logit stands above the best one left out (inf: nothing is left out)."""
+    ranked = -np.sort(-z)
+    return ranked[top - 1] - ranked[top] if top < len(ranked) else np.inf
+
+
+class Stepper:
+    """The same model a token at a time: what every layer run keeps of the tokens before is a list of latents or a
+    state.  ``step(token)`` gives the token's logits; a snapshot can be returned to."""
+
+    def __init__(self, cfg, t):
+        self.cfg, self.t, self.n = cfg, t, 0
+        self.runs = layer_runs(cfg)
+        self.kept = [[] if cfg["layers"][i]["type"] == "latent_attention" else None for i, _ in self.runs]
+
+    def snapshot(self):
+        return self.n, [list(k) if isinstance(k, list) else k for k in self.kept]
+
+    def restore(self, snap):
+        self.n, self.kept = snap[0], [list(k) if isinstance(k, list) else k for k in snap[1]]
+
+    def _latent(self, r, h, m, pre):
+        t, eps, H = self.t, float(self.cfg["norm"]["eps"]), int(m["heads"])
+        q = ((rms_divide(h @ t[pre + "dq"].T, eps) * t[pre + "dq.norm"]) @ t[pre + "uq"].T).reshape(H, -1)
+        self.kept[r].append(latents(h, t, pre, eps)[0])
+        window = int((m.get("mask") or {}).get("size") or 0)
+        c = np.array(self.kept[r][-window:] if window else self.kept[r])
+        k = (c @ t[pre + "uk"].T).reshape(len(c), H, -1)
+        v = (c @ t[pre + "uv"].T).reshape(len(c), H, -1)
+        s = np.einsum("nhd,hd->hn", k, q) * float(m["scale"])
+        e = np.exp(s - s.max(axis=1, keepdims=True))
+        o = np.einsum("hn,nhv->hv", e / e.sum(axis=1, keepdims=True), v)
+        return o.reshape(1, -1) @ t[pre + "o"].T
+
+    def _gla(self, r, h, m, pre):
+        t, eps = self.t, float(self.cfg["norm"]["eps"])
+        H, D, V = int(m["heads"]), int(m["dim"]), int(m["vdim"])
+        S = self.kept[r] if self.kept[r] is not None else np.zeros((H, D, V))
+        k, v = (h @ t[pre + "k"].T).reshape(H, D), (h @ t[pre + "v"].T).reshape(H, V)
+        S = key_decays(h, m, t, pre)[0][:, :, None] * S + k[:, :, None] * v[:, None, :]
+        self.kept[r] = S
+        o = np.einsum("hdv,hd->hv", S, (h @ t[pre + "q"].T).reshape(H, D) * D ** -0.5)
+        o = rms_divide(o, eps) * t[pre + "norm"]
+        return (o.reshape(1, -1) * silu(h @ t[pre + "g"].T)) @ t[pre + "o"].T
+
+    def step(self, token, watch=None):
+        cfg, t, eps = self.cfg, self.t, float(self.cfg["norm"]["eps"])
+        start = embed(t, [token], self.n)
+        x = start.copy()
+        for r, (i, again) in enumerate(self.runs):
+            layer, pre = cfg["layers"][i], f"l{i}."
+            if again:
+                x = x + start
+            h = centred_norm(x, t[pre + "norm1"], eps)
+            one = self._latent if layer["type"] == "latent_attention" else self._gla
+            x = x + centred_norm(one(r, h, layer["mixer"], pre + "mix."), t[pre + "norm1b"], eps)
+            if layer.get("mlp") is not None:
+                h = centred_norm(x, t[pre + "norm2"], eps)
+                if watch is not None:
+                    watch(i, h)
+                x = x + centred_norm(feed_forward(h, layer["mlp"], t, pre + "mlp."), t[pre + "norm2b"], eps)
+        self.n += 1
+        return (centred_norm(x, t["final.norm"], eps) @ t["embed"].T)[0]
+
+
 def load(folder):
     folder = Path(folder)
     return json.loads((folder / "config.json").read_text()), read_safetensors(folder / "model.safetensors")
