@@ -2,7 +2,7 @@
 """Decode and prefill throughput of gguf2bin_b200 on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-                    [--workload decode|ragged8|b64|senotar|levolix|sominex|mopitar] [--batch B] [--layers L] [--context C]
+                    [--workload decode|ragged8|b64|senotar|levolix|sominex|mopitar|kubedra] [--batch B] [--layers L] [--context C]
                     [--no-points] [--sizes 0.6b|8b|14b]
 
 The default run has the layer sizes of Qwen3-0.6B (28 layers, width 1024, 16/8 heads of
@@ -52,6 +52,11 @@ attention with a sink beside a selective state-space branch, layers that borrow 
 experts in groups) beside Sominex, the library's closest design (one norm in front of both sublayers,
 windowed attention, a state-space mixer, routed experts with a shared one), at equal width, layer count,
 vocabulary and, within a few per cent, active parameters.
+
+``--workload kubedra`` sets Kubedra (norms on both sides of a sublayer, latent attention behind a window with
+queries from a latent, gated linear attention with a decay per key channel, capped routed experts with a shared
+one) beside Levolix, the library's closest design (a matrix state per head, normed sublayer outputs, routed
+experts, a tied head), in the same way.
 
 Peaks come from MEASURED_PEAKS.json beside this file when present, else from the
 fallback figures 6.65 TB/s and 1.59 PFLOP/s.  Inputs are synthetic.  Between timed steps
@@ -704,6 +709,102 @@ def mopitar_comparison(a, pk) -> int:
     return 0
 
 
+# ---- Kubedra beside Levolix at equal sizes ----------------------------------------------------------
+def kubedra_config(width, layers, vocab, positions) -> dict:
+    """Latent attention behind a window of 512, then two layers of gated linear attention with Levolix's head sizes, and
+    so on; the first feed-forward dense, the others routed with a shared expert."""
+    out = []
+    moe = dict(kind="moe", expert=dict(ff=3 * width // 4, limit=7.0), router=dict(experts=16, top=3),
+               shared=dict(ff=width, limit=7.0))
+    for i in range(layers):
+        if i % 3:
+            kind, mixer = "gla", dict(heads=width // 256, dim=128, vdim=256, tau=16.0)
+        else:
+            kind = "latent_attention"
+            mixer = dict(heads=width // 128, dim=128, vdim=128, q_rank=width // 2, kv_rank=128, scale=128 ** -0.5,
+                         mask=dict(size=512))
+        out.append(dict(type=kind, mixer=mixer, mlp=moe if i else dict(kind="dense", ff=3 * width)))
+    return dict(architecture="Kubedra", width=width, vocab=vocab, max_positions=positions, norm=dict(eps=1e-6), layers=out)
+
+
+def kubedra_bytes_and_flops(cfg: dict) -> dict:
+    """As ``levolix_bytes_and_flops``; ``kv_bytes_per_token``: of a layer's latents, read once for keys and values."""
+    W, V = cfg["width"], cfg["vocab"]
+    active = total = state_bytes = kv_per_token = attn = 0
+    for layer in cfg["layers"]:
+        m, mlp = layer["mixer"], layer["mlp"]
+        H, D, Vd = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "gla":
+            mix = W * H * (2 * D + 3 * Vd) + 16 * (W + H * D)
+            state_bytes += 2 * 4 * H * D * Vd                                   # read and written
+        else:
+            qr, r = m["q_rank"], m["kv_rank"]
+            mix = W * (qr + r + H * Vd) + H * D * (qr + r) + H * Vd * r
+            kv_per_token += 2 * r
+            attn += 4 * H * r
+        if mlp["kind"] == "dense":
+            a = t = 3 * W * mlp["ff"]
+        else:
+            e, one = mlp["router"], 3 * W * mlp["expert"]["ff"]
+            rest = W * e["experts"] + 3 * W * mlp["shared"]["ff"]
+            a, t = rest + one * e["top"], rest + one * e["experts"]
+        active += mix + a
+        total += mix + t
+    return dict(layer_params=active, total_params=total, weight_bytes=2 * (total + V * W), state_bytes=state_bytes,
+                kv_bytes_per_token=kv_per_token, attn_flops_per_pair=attn)
+
+
+def kubedra_comparison(a, pk) -> int:
+    import torch
+    from gguf2bin_b200.api import LLM
+    layers, vocab, batch, T = a.layers or 6, 151936, a.batch or 8, a.prefill_tokens
+    steps, warmup = a.steps or 128, max(a.warmup, 8)
+    max_tokens = batch * (T + warmup + steps + 128)
+    rows = {}
+    clocks = ClockSampler()
+    clocks.start()
+    for name, (width, ret, att, delta, moe, *_rest) in LEVOLIX_SIZES.items():
+        if a.sizes_only and name not in a.sizes_only.split(","):
+            continue
+        row = {}
+        for arch in ("kubedra", "levolix"):
+            if arch == "kubedra":
+                cfg = kubedra_config(width, layers, vocab, T + warmup + steps + 128)
+                sizes = kubedra_bytes_and_flops(cfg)
+                seen = cfg["layers"][0]["mixer"]["mask"]["size"]
+                pairs = sum(min(t + 1, seen) for t in range(T))
+            else:
+                cfg = levolix_config(width, ret, att, delta, moe, layers, vocab)
+                sizes = levolix_bytes_and_flops(cfg)
+                chunk = att[3]
+                pairs = sum(t % chunk + 1 for t in range(T))
+                seen = chunk / 2.0
+            flops = 2.0 * T * sizes["layer_params"] + sizes["attn_flops_per_pair"] * pairs + 2.0 * vocab * width
+            llm = LLM.random(cfg, seed=0, dtype="bfloat16", max_tokens=max_tokens, max_seqs=batch + 1)
+            first, ms, plain = timed_prompt_step(llm, random_prompts(1, T, vocab, 1), repeats=3)
+            sec, per_step, mean_ctx = decode_device_timed(llm, random_prompts(batch, T, vocab, 100), steps, warmup,
+                                                          vocab, whole_batch_prefill=False)
+            step_bytes = sizes["weight_bytes"] + batch * (sizes["state_bytes"] + min(mean_ctx, seen) * sizes["kv_bytes_per_token"])
+            gbs = step_bytes / (sec / steps) / 1e9
+            row[arch] = dict(
+                active_parameters_per_layer_m=round(sizes["layer_params"] / layers / 1e6, 1),
+                prefill_tokens_per_s=round(T / (ms / 1e3)), prefill_ms=round(ms, 3), prefill_plain_ms=round(plain, 3),
+                prefill_frac_of_tensor_peak=round(flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12), 3),
+                decode_tokens_per_s=round(batch * steps / sec), decode_ms_per_step=round(sec / steps * 1e3, 4),
+                decode_launches_per_step=per_step, decode_step_mb=round(step_bytes / 1e6, 1), decode_gbs=round(gbs),
+                decode_frac_of_copy_bandwidth=round(gbs / pk["hbm_gbs"], 3))
+            del llm
+            torch.cuda.empty_cache()
+        rows[name] = row
+    print(json.dumps({"metric": "prefill and decode tokens/s of Kubedra beside Levolix at equal sizes (random weights)",
+                      "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic", "impl": "ours",
+                      "config": {"layers": layers, "vocab": vocab, "prompt_tokens": T, "decode_batch": batch,
+                                 "decode_context_from": T + warmup, "decode_steps": steps, "peaks": pk["source"],
+                                 "l2": "inputs larger than L2 (weights, states and cache read every step)"},
+                      "sizes": rows, "clocks": clocks.stop()}))
+    return 0
+
+
 WORKLOADS = {
     # name: (sizes, batch, what it is)
     "decode": ("0.6b", 8, "every sequence prefilled to half the context, then decoded"),
@@ -712,6 +813,7 @@ WORKLOADS = {
     "senotar": (None, 8, "Senotar beside Qwen3 at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
     "levolix": (None, 8, "Levolix beside Qwen3 at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
     "sominex": (None, 8, "Sominex beside Qwen3 at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
+    "kubedra": (None, 8, "Kubedra beside Levolix at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
     "mopitar": (None, 8, "Mopitar beside Sominex at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
 }
 
@@ -733,7 +835,7 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                     help="length of the prompt of the prefill figure (decode workload; default 2048)")
     ap.add_argument("--sizes-only", default=None,
-                    help="senotar, levolix, sominex and mopitar workloads: a comma-separated subset of " + ",".join(EQUAL_SIZES))
+                    help="senotar, levolix, sominex, mopitar and kubedra workloads: a comma-separated subset of " + ",".join(EQUAL_SIZES))
     a = ap.parse_args()
 
     if a.impl == "reference":
@@ -755,6 +857,8 @@ def main() -> int:
         return sominex_comparison(a, peaks())
     if a.workload == "mopitar":
         return mopitar_comparison(a, peaks())
+    if a.workload == "kubedra":
+        return kubedra_comparison(a, peaks())
 
     import numpy as np
     import torch

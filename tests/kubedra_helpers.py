@@ -85,12 +85,12 @@ def mixer_weights(rng, kind, m, d, pre="", decay_rank=16):
     H, D, V = m["heads"], m["dim"], m["vdim"]
     if kind == "latent_attention":
         qr, r = m["q_rank"], m["kv_rank"]
-        W[pre + "dq"], W[pre + "uq"] = mat(qr, d), mat(H * D, qr, 1.5)
-        W[pre + "dkv"], W[pre + "uk"], W[pre + "uv"] = mat(r, d), mat(H * D, r, 1.5), mat(H * V, r)
+        W[pre + "dq"], W[pre + "uq"] = mat(qr, d), mat(H * D, qr)
+        W[pre + "dkv"], W[pre + "uk"], W[pre + "uv"] = mat(r, d), mat(H * D, r), mat(H * V, r)
         W[pre + "dq.norm"], W[pre + "dkv.norm"] = 1 + 0.3 * rng.standard_normal(qr), 1 + 0.3 * rng.standard_normal(r)
         W[pre + "o"] = mat(d, H * V)
     elif kind == "gla":
-        W[pre + "q"], W[pre + "k"], W[pre + "v"] = mat(H * D, d, 2.0), mat(H * D, d, 2.0), mat(H * V, d)
+        W[pre + "q"], W[pre + "k"], W[pre + "v"] = mat(H * D, d), mat(H * D, d), mat(H * V, d)
         W[pre + "g"], W[pre + "o"] = mat(H * V, d, 2.0), mat(d, H * V)
         W[pre + "a1"], W[pre + "a2"] = mat(decay_rank, d), mat(H * D, decay_rank, 2.0)
         W[pre + "a2.b"] = rng.standard_normal(H * D) * 2.0
