@@ -169,7 +169,7 @@ static int launch_channel_step(const ChannelIn &a, float *state, const int *seq_
 // ---------------------------------------------------------------------------
 // prompts: what every column of a head needs of a token, once
 // ---------------------------------------------------------------------------
-#define CP_TOKENS 16
+#define CP_TOKENS 4
 #define CP_THREADS 128
 template <typename T>
 __global__ void __launch_bounds__(CP_THREADS)
@@ -178,20 +178,33 @@ channel_prep_kernel(const ChannelIn a, int n_tokens, float *__restrict__ qf, flo
   pdl_wait();
   extern __shared__ __align__(16) float cs_sm[];      // low vectors of the block's tokens [CP_TOKENS, R]
   const int D = a.D, R = a.R, h = blockIdx.y;
-  const int t0 = blockIdx.x * CP_TOKENS, nt = min(CP_TOKENS, n_tokens - t0);
-  for (int i = threadIdx.x; i < nt * R; i += CP_THREADS)
-    cs_sm[i] = to_f32(((const T *)a.low)[(size_t)(t0 + i / R) * a.low_stride + i % R]);
+  const int t0 = blockIdx.x * CP_TOKENS;
+  for (int i = threadIdx.x; i < CP_TOKENS * R; i += CP_THREADS)       // tokens behind the last one repeat it
+    cs_sm[i] = to_f32(((const T *)a.low)[(size_t)min(t0 + i / R, n_tokens - 1) * a.low_stride + i % R]);
   __syncthreads();
   const size_t row = (size_t)a.H * D;
   for (int d = threadIdx.x; d < D; d += CP_THREADS) {
     const size_t ch = (size_t)h * D + d;
+    float z[CP_TOKENS], qv[CP_TOKENS], kv[CP_TOKENS];
+#pragma unroll
+    for (int i = 0; i < CP_TOKENS; ++i) {
+      const size_t t = min(t0 + i, n_tokens - 1);
+      qv[i] = to_f32(((const T *)a.q)[t * a.q_stride + ch]);
+      kv[i] = to_f32(((const T *)a.k)[t * a.k_stride + ch]);
+      z[i] = 0.f;
+    }
     const T *w = (const T *)a.w_low + ch * R;
+    for (int r = 0; r < R; r += 8)
+#pragma unroll
+      for (int i = 0; i < CP_TOKENS; ++i) z[i] = low_dot(w + r, cs_sm + i * R + r, 8, z[i]);
     const float bias = a.bias[ch];
-    for (int i = 0; i < nt; ++i) {
-      const size_t t = t0 + i, at = t * row + ch;
-      af[at] = decay_of(low_dot(w, cs_sm + i * R, R, 0.f) + bias, a.inv_tau);
-      qf[at] = to_f32(((const T *)a.q)[t * a.q_stride + ch]) * a.q_scale;
-      kf[at] = to_f32(((const T *)a.k)[t * a.k_stride + ch]);
+#pragma unroll
+    for (int i = 0; i < CP_TOKENS; ++i) {
+      if (t0 + i >= n_tokens) break;
+      const size_t at = (size_t)(t0 + i) * row + ch;
+      af[at] = decay_of(z[i] + bias, a.inv_tau);
+      qf[at] = qv[i] * a.q_scale;
+      kf[at] = kv[i];
     }
   }
 }
@@ -204,11 +217,11 @@ __device__ __forceinline__ void cs_copy16(float *smem, const float *g) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(addr), "l"(g));
 }
 
-// 128 threads; L lanes hold CC = 2 columns, lane l of them the rows 4 (j L + l) .. + 3, j < RG (rows from D on are
-// zeros); tiles of `tile` tokens (a multiple of four) of k, a (and q) as float rows of Dp and of the columns' v, in
-// two buffers: the next tile is on its way while one is computed.
+// 128 threads; L lanes hold CC columns, lane l of them the rows 4 (j L + l) .. + 3, j < RG (rows from D on are zeros):
+// a row of k, a or q that a lane reads from shared memory serves CC columns, and the lanes of a warp read different
+// rows (one warp, one column group, where D is above 64).  Tiles of `tile` tokens (a multiple of four) of k, a (and q)
+// as float rows of Dp and of the columns' v, in two buffers: the next tile is on its way while one is computed.
 #define SEG_THREADS 128
-#define SEG_CC 2
 struct SegArgs {
   const float *qf, *kf, *af;          // [T, H, D]
   const void *v;
@@ -225,13 +238,37 @@ struct SegArgs {
 // segments of all sequences numbered without gaps that matter: distinct for distinct (sequence, segment)
 __device__ __forceinline__ int segment_id(int first_row, int tile_rows, int seq) { return first_row / tile_rows + seq; }
 
-template <typename T, int L, int RG, bool READ>
+// Sums over L lanes of N values a lane: halves of the values change hands until every lane has N / L of them (or, where
+// there are fewer values than lanes, lanes share one); returns the first of the lane's values' index.
+template <int N, int L>
+__device__ __forceinline__ int lanes_sum(float (&o)[N], int lane) {
+  int base = 0, n = N;
+#pragma unroll
+  for (int m = L >> 1; m > 0; m >>= 1) {
+    if (n > 1) {
+      n >>= 1;
+      const bool up = lane & m;
+#pragma unroll
+      for (int i = 0; i < N / 2; ++i)
+        if (i < n) {
+          const float send = up ? o[i] : o[i + n], keep = up ? o[i + n] : o[i];
+          o[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+        }
+      base += up ? n : 0;
+    } else {
+      o[0] += __shfl_xor_sync(0xffffffffu, o[0], m);
+    }
+  }
+  return base;
+}
+
+template <typename T, int L, int RG, int CC, bool READ>
 __global__ void __launch_bounds__(SEG_THREADS)
 channel_segment_kernel(const SegArgs a) {
   pdl_launch();
   pdl_wait();
   extern __shared__ __align__(16) float cs_sm[];
-  constexpr int COLS = SEG_THREADS / L * SEG_CC;
+  constexpr int COLS = SEG_THREADS / L * CC;
   constexpr int ROWS = READ ? 3 : 2;                 // k, a and, for read-outs, q
   const int4 tl = a.tiles[blockIdx.z];
   const int b = tl.x, first_row = tl.y, n = tl.z;
@@ -241,7 +278,7 @@ channel_segment_kernel(const SegArgs a) {
   const int D = a.D, V = a.V, H = a.H, Dp = a.Dp, TT = a.tile;
   const int h = blockIdx.y;
   const int lane = threadIdx.x % L, group = threadIdx.x / L;
-  const int c0 = blockIdx.x * COLS + group * SEG_CC;
+  const int c0 = blockIdx.x * COLS + group * CC;
   const int seg = segment_id(first_row, a.tile_rows, b);
   const size_t col_at = ((size_t)h * V + c0) * D;
   float *own = a.seg_state + (size_t)seg * H * V * D + col_at;
@@ -250,9 +287,9 @@ channel_segment_kernel(const SegArgs a) {
   float *sv = cs_sm + 2 * buf_floats;                // [2][TT, COLS]
   const bool vec = (D & 3) == 0;
 
-  float S[SEG_CC][RG][4], P[RG][4];
+  float S[CC][RG][4], P[RG][4];
 #pragma unroll
-  for (int c = 0; c < SEG_CC; ++c)
+  for (int c = 0; c < CC; ++c)
 #pragma unroll
     for (int j = 0; j < RG; ++j)
 #pragma unroll
@@ -309,64 +346,57 @@ channel_segment_kernel(const SegArgs a) {
     __syncthreads();
     if (t0 + TT < n) fetch(t0 + TT, min(TT, n - t0 - TT), buf ^ 1);
     const float *kp = cs_sm + buf * buf_floats + 4 * lane;
-    const float *vp = sv + buf * TT * COLS + group * SEG_CC;
+    const float *vp = sv + buf * TT * COLS + group * CC;
     for (int u = 0; u < nt; u += 4) {
-      float o[4 * SEG_CC];
+      float o[4 * CC];
 #pragma unroll
       for (int s = 0; s < 4; ++s) {
         const float *k4 = kp + (u + s) * Dp, *a4 = k4 + TT * Dp, *q4 = a4 + TT * Dp;
-        const float2 v = *reinterpret_cast<const float2 *>(vp + (u + s) * COLS);
-        float o0 = 0.f, o1 = 0.f;
+        float v[CC];
+#pragma unroll
+        for (int c = 0; c < CC; c += 2) {
+          const float2 x = *reinterpret_cast<const float2 *>(vp + (u + s) * COLS + c);
+          v[c] = x.x, v[c + 1] = x.y;
+        }
+#pragma unroll
+        for (int c = 0; c < CC; ++c) o[CC * s + c] = 0.f;
 #pragma unroll
         for (int j = 0; j < RG; ++j) {
           const float4 kd = *reinterpret_cast<const float4 *>(k4 + 4 * j * L);
           const float4 ad = *reinterpret_cast<const float4 *>(a4 + 4 * j * L);
-          S[0][j][0] = fmaf(ad.x, S[0][j][0], kd.x * v.x), S[1][j][0] = fmaf(ad.x, S[1][j][0], kd.x * v.y);
-          S[0][j][1] = fmaf(ad.y, S[0][j][1], kd.y * v.x), S[1][j][1] = fmaf(ad.y, S[1][j][1], kd.y * v.y);
-          S[0][j][2] = fmaf(ad.z, S[0][j][2], kd.z * v.x), S[1][j][2] = fmaf(ad.z, S[1][j][2], kd.z * v.y);
-          S[0][j][3] = fmaf(ad.w, S[0][j][3], kd.w * v.x), S[1][j][3] = fmaf(ad.w, S[1][j][3], kd.w * v.y);
-          if (READ) {
-            const float4 qd = *reinterpret_cast<const float4 *>(q4 + 4 * j * L);
-            o0 = fmaf(S[0][j][3], qd.w, fmaf(S[0][j][2], qd.z, fmaf(S[0][j][1], qd.y, fmaf(S[0][j][0], qd.x, o0))));
-            o1 = fmaf(S[1][j][3], qd.w, fmaf(S[1][j][2], qd.z, fmaf(S[1][j][1], qd.y, fmaf(S[1][j][0], qd.x, o1))));
-          } else if (track) {
-            P[j][0] *= ad.x, P[j][1] *= ad.y, P[j][2] *= ad.z, P[j][3] *= ad.w;
+          float4 qd = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (READ) qd = *reinterpret_cast<const float4 *>(q4 + 4 * j * L);
+#pragma unroll
+          for (int c = 0; c < CC; ++c) {
+            S[c][j][0] = fmaf(ad.x, S[c][j][0], kd.x * v[c]);
+            S[c][j][1] = fmaf(ad.y, S[c][j][1], kd.y * v[c]);
+            S[c][j][2] = fmaf(ad.z, S[c][j][2], kd.z * v[c]);
+            S[c][j][3] = fmaf(ad.w, S[c][j][3], kd.w * v[c]);
+            if (READ)
+              o[CC * s + c] = fmaf(S[c][j][3], qd.w, fmaf(S[c][j][2], qd.z, fmaf(S[c][j][1], qd.y,
+                                   fmaf(S[c][j][0], qd.x, o[CC * s + c]))));
           }
+          if (!READ && track) P[j][0] *= ad.x, P[j][1] *= ad.y, P[j][2] *= ad.z, P[j][3] *= ad.w;
         }
-        o[2 * s] = o0, o[2 * s + 1] = o1;
       }
       if (READ) {
-        // the lanes' shares of eight (token, column) sums: halves of the values change hands, so that lane i of
-        // eight ends with sum i after seven exchanges; then what is left of a column's L lanes
+        constexpr int N = 4 * CC, LEFT = N > L ? N / L : 1;          // values a lane ends with
+        const int first = lanes_sum<N, L>(o, lane);
+        if (N >= L || lane % (L / (N < L ? N : L)) == 0) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float send = (lane & 4) ? o[i] : o[i + 4];
-          const float keep = (lane & 4) ? o[i + 4] : o[i];
-          o[i] = keep + __shfl_xor_sync(0xffffffffu, send, 4);
+          for (int i = 0; i < LEFT; ++i) {
+            const int s = (first + i) / CC, c = (first + i) % CC;
+            if (u + s < nt && c0 + c < V)
+              a.out[(size_t)(first_row + t0 + u + s) * H * V + (size_t)h * V + c0 + c] = o[i];
+          }
         }
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const float send = (lane & 2) ? o[i] : o[i + 2];
-          const float keep = (lane & 2) ? o[i + 2] : o[i];
-          o[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
-        }
-        {
-          const float send = (lane & 1) ? o[0] : o[1];
-          const float keep = (lane & 1) ? o[1] : o[0];
-          o[0] = keep + __shfl_xor_sync(0xffffffffu, send, 1);
-        }
-#pragma unroll
-        for (int off = 8; off < L; off <<= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], off);
-        const int which = lane & 7, s = which >> 1, c = which & 1;       // value index 4 x + 2 y + z of the lane's bits
-        if (lane < 8 && u + s < nt && c0 + c < V)
-          a.out[(size_t)(first_row + t0 + u + s) * H * V + (size_t)h * V + c0 + c] = o[0];
       }
     }
   }
   float *dst = READ ? slot_state : own;
   if (!READ || is_last) {
 #pragma unroll
-    for (int c = 0; c < SEG_CC; ++c)
+    for (int c = 0; c < CC; ++c)
 #pragma unroll
       for (int j = 0; j < RG; ++j)
 #pragma unroll
@@ -413,27 +443,28 @@ channel_carry_kernel(const float *__restrict__ state, float *__restrict__ seg_st
   }
 }
 
-template <typename T, int L, int RG>
+template <typename T, int L, int RG, int CC>
 static void launch_segment(const SegArgs &a, int n_tiles, bool read, size_t smem, cudaStream_t stream) {
-  constexpr int COLS = SEG_THREADS / L * SEG_CC;
+  constexpr int COLS = SEG_THREADS / L * CC;
   const dim3 grid((a.V + COLS - 1) / COLS, a.H, n_tiles);
-  auto kr = channel_segment_kernel<T, L, RG, true>;
-  auto kw = channel_segment_kernel<T, L, RG, false>;
+  auto kr = channel_segment_kernel<T, L, RG, CC, true>;
+  auto kw = channel_segment_kernel<T, L, RG, CC, false>;
   if (smem > 48 * 1024) cudaFuncSetAttribute(read ? kr : kw, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   g2b_launch(read ? kr : kw, grid, dim3(SEG_THREADS), smem, stream, a);
 }
 
 template <typename T>
 static int segments(SegArgs a, int n_tiles, bool read, cudaStream_t stream) {
-  // lanes a pair of columns: 8 hold up to 128 rows, 16 up to 256, 32 up to 512
-  const int L = a.D <= 128 ? 8 : (a.D <= 256 ? 16 : 32);
+  // rows of the state: 4 a lane on 8, 16 or 32 lanes, or 8, 12 or 16 a lane on 32; 32 entries a lane in all (24 of 12 rows)
+  const int L = a.D <= 32 ? 8 : (a.D <= 64 ? 16 : 32);
   const int RG = (a.D + 4 * L - 1) / (4 * L);
+  const int CC = RG == 1 ? 8 : (RG == 2 ? 4 : 2);
   a.Dp = RG * 4 * L;
   a.tile = a.Dp <= 128 ? 8 : 4;
-  const int cols = SEG_THREADS / L * SEG_CC;
+  const int cols = SEG_THREADS / L * CC;
   const size_t smem = (size_t)(2 * (read ? 3 : 2) * a.tile * a.Dp + 2 * a.tile * cols) * sizeof(float);
-#define CS_CASE(L_, RG_) if (L == L_ && RG == RG_) { launch_segment<T, L_, RG_>(a, n_tiles, read, smem, stream); return 0; }
-  CS_CASE(8, 1) CS_CASE(8, 2) CS_CASE(8, 3) CS_CASE(8, 4) CS_CASE(16, 3) CS_CASE(16, 4) CS_CASE(32, 3) CS_CASE(32, 4)
+#define CS_CASE(L_, RG_, CC_) if (L == L_ && RG == RG_) { launch_segment<T, L_, RG_, CC_>(a, n_tiles, read, smem, stream); return 0; }
+  CS_CASE(8, 1, 8) CS_CASE(16, 1, 8) CS_CASE(32, 1, 8) CS_CASE(32, 2, 4) CS_CASE(32, 3, 2) CS_CASE(32, 4, 2)
 #undef CS_CASE
   return 1;
 }
