@@ -16,6 +16,9 @@ from .mopitar import ARCHITECTURE as MOPITAR_ARCHITECTURE, mopitar_model_spec
 
 from .kubedra import ARCHITECTURE as KUBEDRA_ARCHITECTURE, kubedra_model_spec
 
+from .nekotar import ARCHITECTURE as NEKOTAR_ARCHITECTURE, nekotar_model_spec
+
+register_architecture(NEKOTAR_ARCHITECTURE, nekotar_model_spec)
 register_architecture(KUBEDRA_ARCHITECTURE, kubedra_model_spec)
 register_architecture(SENOTAR_ARCHITECTURE, senotar_model_spec)
 register_architecture(MOPITAR_ARCHITECTURE, mopitar_model_spec)
@@ -23,5 +26,5 @@ register_architecture(SOMINEX_ARCHITECTURE, sominex_model_spec)
 register_architecture(LEVOLIX_ARCHITECTURE, levolix_model_spec)
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config",
-           "QWEN3_ARCHITECTURE", "SENOTAR_ARCHITECTURE", "senotar_model_spec", "LEVOLIX_ARCHITECTURE", "levolix_model_spec", "SOMINEX_ARCHITECTURE", "sominex_model_spec", "MOPITAR_ARCHITECTURE", "mopitar_model_spec", "KUBEDRA_ARCHITECTURE", "kubedra_model_spec", "model_spec_from_dict", "model_spec_from_folder",
+           "QWEN3_ARCHITECTURE", "SENOTAR_ARCHITECTURE", "senotar_model_spec", "LEVOLIX_ARCHITECTURE", "levolix_model_spec", "SOMINEX_ARCHITECTURE", "sominex_model_spec", "MOPITAR_ARCHITECTURE", "mopitar_model_spec", "KUBEDRA_ARCHITECTURE", "kubedra_model_spec", "NEKOTAR_ARCHITECTURE", "nekotar_model_spec", "model_spec_from_dict", "model_spec_from_folder",
            "read_config_json", "read_generation_stop_ids", "register_architecture", "registered_architectures"]

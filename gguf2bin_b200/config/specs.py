@@ -82,11 +82,16 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec                    # kind "lm_head" (tied or own matrix)
     stop_token_ids: tuple = ()
+    streams: int = 1                  # residual streams side by side; the head reads their sum
     source: Mapping[str, Any] = field(default_factory=dict, compare=False, hash=False)
 
     def validate(self) -> None:
         if self.hidden_size <= 0 or self.vocab_size <= 0 or self.max_positions <= 0:
             raise ConfigError("hidden_size, vocab_size and max_positions must be positive")
+        if self.streams < 1:
+            raise ConfigError("a model has at least one residual stream")
+        if self.streams > 1 and any(e.add_embedding for e in self.schedule):
+            raise ConfigError("the embedding cannot be added again to a model of several streams")
         if self.vocab_size >= 2 ** 31:
             raise ConfigError("vocab_size does not fit a 32-bit token id")
         if not self.layers or not self.schedule:

@@ -1,7 +1,10 @@
-// A matrix state per head with a decay per KEY CHANNEL (gated linear attention):
+// A matrix state per head with a decay per KEY CHANNEL (gated linear attention, time mixing with a bonus):
 //   S <- diag(a_t) S + k_t v_t^T,   o_t = S^T q_t,   S [D, V] per head
-// with a_t = sigmoid(z_t)^(1/tau), z_t = W_low l_t + bias: one number per token, head and key channel, from a
-// vector l_t of R entries per token (R small).  Everything but the inputs q, k, v, l, W_low is 32-bit.
+// with z_t = W_low l_t + bias: one number per token, head and key channel, from a vector l_t of R entries per token
+// (R small; its entries may pass tanh first), and a_t = sigmoid(z_t)^(1/tau) or exp(-exp(z_t)).
+// With a bonus u [H, D] the read-out comes before the update and the token's own key counts u times:
+//   o_t = (S + diag(u) k_t v_t^T)^T q_t = S^T q_t + (sum_d q_d u_d k_d) v_t,   then the update.
+// Everything but the inputs q, k, v, l, W_low is 32-bit (l may be, too).
 // The state is stored column by column ([slot, head, V, D]), as in seq_mix.cu.
 //
 //   channel_step      one token per sequence: decays, update and read-out in one launch
@@ -25,6 +28,7 @@ G2B_DEFINE_LAST_ERROR
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 // sigmoid(z)^(1/tau) through its logarithm
 __device__ __forceinline__ float decay_of(float z, float inv_tau) { return expf(-softplus_f(-z) * inv_tau); }
+enum { DECAY_SIGMOID_ROOT = 0, DECAY_DOUBLE_EXP = 1 };
 
 // sum over r of w[r] * low[r], R a multiple of eight, ascending r
 __device__ __forceinline__ float low_dot(const float *w, const float *low, int R, float acc) {
@@ -55,7 +59,17 @@ struct ChannelIn {
   const float *bias;                  // [H * D]
   int H, D, V, R;
   float q_scale, inv_tau;
+  int decay;                          // which form turns z into a decay
+  int low_tanh, low_f32;              // l passes tanh; l is float whatever the compute type
+  const float *bonus;                 // [H, D] or null
 };
+__device__ __forceinline__ float decay_form(const ChannelIn &a, float z) {
+  return a.decay == DECAY_DOUBLE_EXP ? expf(-expf(z)) : decay_of(z, a.inv_tau);
+}
+template <typename T> __device__ __forceinline__ float low_entry(const ChannelIn &a, size_t t, int r) {
+  const float v = a.low_f32 ? ((const float *)a.low)[t * a.low_stride + r] : to_f32(((const T *)a.low)[t * a.low_stride + r]);
+  return a.low_tanh ? tanhf(v) : v;
+}
 
 // ---------------------------------------------------------------------------
 // one token per sequence
@@ -93,8 +107,7 @@ channel_step_kernel(const ChannelIn a, float *__restrict__ state, const int *__r
         S[c][r][0] = in ? sp[(size_t)c * D + d] : 0.f;
       }
     }
-  const T *lp = (const T *)a.low + (size_t)b * a.low_stride;
-  for (int r = threadIdx.x; r < R; r += CS_THREADS) low[r] = to_f32(lp[r]);
+  for (int r = threadIdx.x; r < R; r += CS_THREADS) low[r] = low_entry<T>(a, b, r);
   __syncthreads();
   const T *qp = (const T *)a.q + (size_t)b * a.q_stride + (size_t)h * D;
   const T *kp = (const T *)a.k + (size_t)b * a.k_stride + (size_t)h * D;
@@ -103,9 +116,16 @@ channel_step_kernel(const ChannelIn a, float *__restrict__ state, const int *__r
     sq[d] = in ? to_f32(qp[d]) * a.q_scale : 0.f;
     sk[d] = in ? to_f32(kp[d]) : 0.f;
     const size_t ch = (size_t)h * D + d;
-    sa[d] = in ? decay_of(low_dot((const T *)a.w_low + ch * R, low, R, 0.f) + a.bias[ch], a.inv_tau) : 0.f;
+    sa[d] = in ? decay_form(a, low_dot((const T *)a.w_low + ch * R, low, R, 0.f) + a.bias[ch]) : 0.f;
   }
   __syncthreads();
+  float own = 0.f;                                   // what the token's own value counts in its read-out
+  const bool bonus = a.bonus;
+  if (bonus) {
+    __shared__ float scratch[32];
+    for (int d = threadIdx.x; d < D; d += CS_THREADS) own = fmaf(sq[d] * sk[d], a.bonus[(size_t)h * D + d], own);
+    own = block_sum(own, scratch);
+  }
   const T *vp = (const T *)a.v + (size_t)b * a.v_stride + (size_t)h * V;
   float o[CS_COLS];
 #pragma unroll
@@ -118,8 +138,9 @@ channel_step_kernel(const ChannelIn a, float *__restrict__ state, const int *__r
       if (d < D) {
 #pragma unroll
         for (int i = 0; i < VEC; ++i) {
-          S[c][r][i] = fmaf(sa[d + i], S[c][r][i], sk[d + i] * v);
-          o[c] = fmaf(S[c][r][i], sq[d + i], o[c]);
+          const float before = S[c][r][i];
+          S[c][r][i] = fmaf(sa[d + i], before, sk[d + i] * v);
+          o[c] = fmaf(bonus ? before : S[c][r][i], sq[d + i], o[c]);
         }
         if (c0 + c < V) {
           if (VEC == 4)
@@ -137,7 +158,8 @@ channel_step_kernel(const ChannelIn a, float *__restrict__ state, const int *__r
   if (lane == 0) {
 #pragma unroll
     for (int c = 0; c < CS_COLS; ++c)
-      if (c0 + c < V) out[(size_t)b * H * V + (size_t)h * V + c0 + c] = o[c];
+      if (c0 + c < V)
+        out[(size_t)b * H * V + (size_t)h * V + c0 + c] = bonus ? fmaf(own, to_f32(vp[c0 + c]), o[c]) : o[c];
   }
 }
 
@@ -173,18 +195,23 @@ static int launch_channel_step(const ChannelIn &a, float *state, const int *seq_
 #define CP_THREADS 128
 template <typename T>
 __global__ void __launch_bounds__(CP_THREADS)
-channel_prep_kernel(const ChannelIn a, int n_tokens, float *__restrict__ qf, float *__restrict__ kf, float *__restrict__ af) {
+channel_prep_kernel(const ChannelIn a, int n_tokens, float *__restrict__ qf, float *__restrict__ kf, float *__restrict__ af,
+                    float *__restrict__ own) {
   pdl_launch();
   pdl_wait();
   extern __shared__ __align__(16) float cs_sm[];      // low vectors of the block's tokens [CP_TOKENS, R]
   const int D = a.D, R = a.R, h = blockIdx.y;
   const int t0 = blockIdx.x * CP_TOKENS;
   for (int i = threadIdx.x; i < CP_TOKENS * R; i += CP_THREADS)       // tokens behind the last one repeat it
-    cs_sm[i] = to_f32(((const T *)a.low)[(size_t)min(t0 + i / R, n_tokens - 1) * a.low_stride + i % R]);
+    cs_sm[i] = low_entry<T>(a, min(t0 + i / R, n_tokens - 1), i % R);
   __syncthreads();
   const size_t row = (size_t)a.H * D;
+  float sum[CP_TOKENS];
+#pragma unroll
+  for (int i = 0; i < CP_TOKENS; ++i) sum[i] = 0.f;
   for (int d = threadIdx.x; d < D; d += CP_THREADS) {
     const size_t ch = (size_t)h * D + d;
+    const float u = a.bonus ? a.bonus[ch] : 0.f;
     float z[CP_TOKENS], qv[CP_TOKENS], kv[CP_TOKENS];
 #pragma unroll
     for (int i = 0; i < CP_TOKENS; ++i) {
@@ -202,10 +229,18 @@ channel_prep_kernel(const ChannelIn a, int n_tokens, float *__restrict__ qf, flo
     for (int i = 0; i < CP_TOKENS; ++i) {
       if (t0 + i >= n_tokens) break;
       const size_t at = (size_t)(t0 + i) * row + ch;
-      af[at] = decay_of(z[i] + bias, a.inv_tau);
+      af[at] = decay_form(a, z[i] + bias);
       qf[at] = qv[i] * a.q_scale;
       kf[at] = kv[i];
+      sum[i] = fmaf(qv[i] * a.q_scale * kv[i], u, sum[i]);
     }
+  }
+  if (!a.bonus) return;
+  __shared__ float scratch[32];
+#pragma unroll
+  for (int i = 0; i < CP_TOKENS; ++i) {
+    const float s = block_sum(sum[i], scratch);
+    if (threadIdx.x == 0 && t0 + i < n_tokens) own[(size_t)(t0 + i) * a.H + h] = s;
   }
 }
 
@@ -233,6 +268,7 @@ struct SegArgs {
   float *seg_state;                   // [segments, H, V, D]: end states, then the states in front
   float *seg_decay;                   // [segments, H, D]: products of the decays
   float *out;                         // [T, H * V]
+  const float *own;                   // [T, H] with a bonus: what a token's own value counts in its read-out
   int Dp, tile;
 };
 // segments of all sequences numbered without gaps that matter: distinct for distinct (sequence, segment)
@@ -262,7 +298,7 @@ __device__ __forceinline__ int lanes_sum(float (&o)[N], int lane) {
   return base;
 }
 
-template <typename T, int L, int RG, int CC, bool READ>
+template <typename T, int L, int RG, int CC, bool READ, bool BONUS>
 __global__ void __launch_bounds__(SEG_THREADS)
 channel_segment_kernel(const SegArgs a) {
   pdl_launch();
@@ -285,6 +321,7 @@ channel_segment_kernel(const SegArgs a) {
   float *slot_state = a.state + (size_t)slot * H * V * D + col_at;
   const int buf_floats = ROWS * TT * Dp;
   float *sv = cs_sm + 2 * buf_floats;                // [2][TT, COLS]
+  float *so = sv + 2 * TT * COLS;                    // [2][TT] with a bonus
   const bool vec = (D & 3) == 0;
 
   float S[CC][RG][4], P[RG][4];
@@ -335,6 +372,7 @@ channel_segment_kernel(const SegArgs a) {
       const int tt = i / COLS, cc = i % COLS;
       dv[i] = tt < nt && blockIdx.x * COLS + cc < V ? to_f32(vg[(size_t)tt * a.v_stride + cc]) : 0.f;
     }
+    if (BONUS && threadIdx.x < nt) so[buf * TT + threadIdx.x] = a.own[(size_t)(first_row + t0 + threadIdx.x) * H + h];
   };
 
   fetch(0, min(TT, n), 0);
@@ -368,11 +406,14 @@ channel_segment_kernel(const SegArgs a) {
           if (READ) qd = *reinterpret_cast<const float4 *>(q4 + 4 * j * L);
 #pragma unroll
           for (int c = 0; c < CC; ++c) {
+            if (READ && BONUS)                         // the state in front of the token
+              o[CC * s + c] = fmaf(S[c][j][3], qd.w, fmaf(S[c][j][2], qd.z, fmaf(S[c][j][1], qd.y,
+                                   fmaf(S[c][j][0], qd.x, o[CC * s + c]))));
             S[c][j][0] = fmaf(ad.x, S[c][j][0], kd.x * v[c]);
             S[c][j][1] = fmaf(ad.y, S[c][j][1], kd.y * v[c]);
             S[c][j][2] = fmaf(ad.z, S[c][j][2], kd.z * v[c]);
             S[c][j][3] = fmaf(ad.w, S[c][j][3], kd.w * v[c]);
-            if (READ)
+            if (READ && !BONUS)
               o[CC * s + c] = fmaf(S[c][j][3], qd.w, fmaf(S[c][j][2], qd.z, fmaf(S[c][j][1], qd.y,
                                    fmaf(S[c][j][0], qd.x, o[CC * s + c]))));
           }
@@ -386,8 +427,10 @@ channel_segment_kernel(const SegArgs a) {
 #pragma unroll
           for (int i = 0; i < LEFT; ++i) {
             const int s = (first + i) / CC, c = (first + i) % CC;
-            if (u + s < nt && c0 + c < V)
+            if (u + s < nt && c0 + c < V) {
+              if (BONUS) o[i] = fmaf(so[buf * TT + u + s], vp[(u + s) * COLS + c], o[i]);
               a.out[(size_t)(first_row + t0 + u + s) * H * V + (size_t)h * V + c0 + c] = o[i];
+            }
           }
         }
       }
@@ -447,8 +490,8 @@ template <typename T, int L, int RG, int CC>
 static void launch_segment(const SegArgs &a, int n_tiles, bool read, size_t smem, cudaStream_t stream) {
   constexpr int COLS = SEG_THREADS / L * CC;
   const dim3 grid((a.V + COLS - 1) / COLS, a.H, n_tiles);
-  auto kr = channel_segment_kernel<T, L, RG, CC, true>;
-  auto kw = channel_segment_kernel<T, L, RG, CC, false>;
+  auto kr = a.own ? channel_segment_kernel<T, L, RG, CC, true, true> : channel_segment_kernel<T, L, RG, CC, true, false>;
+  auto kw = channel_segment_kernel<T, L, RG, CC, false, false>;
   if (smem > 48 * 1024) cudaFuncSetAttribute(read ? kr : kw, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   g2b_launch(read ? kr : kw, grid, dim3(SEG_THREADS), smem, stream, a);
 }
@@ -462,7 +505,7 @@ static int segments(SegArgs a, int n_tiles, bool read, cudaStream_t stream) {
   a.Dp = RG * 4 * L;
   a.tile = a.Dp <= 128 ? 8 : 4;
   const int cols = SEG_THREADS / L * CC;
-  const size_t smem = (size_t)(2 * (read ? 3 : 2) * a.tile * a.Dp + 2 * a.tile * cols) * sizeof(float);
+  const size_t smem = (size_t)(2 * (read ? 3 : 2) * a.tile * a.Dp + 2 * a.tile * (cols + 1)) * sizeof(float);
 #define CS_CASE(L_, RG_, CC_) if (L == L_ && RG == RG_) { launch_segment<T, L_, RG_, CC_>(a, n_tiles, read, smem, stream); return 0; }
   CS_CASE(8, 1, 8) CS_CASE(16, 1, 8) CS_CASE(32, 1, 8) CS_CASE(32, 2, 4) CS_CASE(32, 3, 2) CS_CASE(32, 4, 2)
 #undef CS_CASE
@@ -471,7 +514,8 @@ static int segments(SegArgs a, int n_tiles, bool read, cudaStream_t stream) {
 
 extern "C" int g2b_channel_scan(int dtype, const void *q, int q_stride, const void *k, int k_stride, const void *v,
                                 int v_stride, const void *low, int low_stride, const void *w_low, const float *bias, int H,
-                                int D, int V, int R, float q_scale, float inv_tau, float *state, const int *seq_slots,
+                                int D, int V, int R, float q_scale, float inv_tau, int decay, int low_tanh, int low_f32,
+                                const float *bonus, float *own, float *state, const int *seq_slots,
                                 const int *seq_meta, int n_tokens, int n_seqs, const int *tiles, int n_tiles, int tile_rows,
                                 float *qf, float *kf, float *af, float *seg_state, float *seg_decay, float *out,
                                 cudaStream_t stream) {
@@ -481,24 +525,30 @@ extern "C" int g2b_channel_scan(int dtype, const void *q, int q_stride, const vo
   if ((uintptr_t)w_low & 15) G2B_REFUSE("channel_scan: the decay matrix must start on 16 bytes");
   if (dtype != G2B_F32 && dtype != G2B_BF16) G2B_REFUSE("channel_scan: unknown dtype %d", dtype);
   if (H > 65535 || n_seqs > 65535 || n_tiles > 65535) G2B_REFUSE("channel_scan: %d heads, %d sequences or %d tiles are too many", H, n_seqs, n_tiles);
-  ChannelIn in = {q, k, v, low, q_stride, k_stride, v_stride, low_stride, w_low, bias, H, D, V, R, q_scale, inv_tau};
+  if (decay != DECAY_SIGMOID_ROOT && decay != DECAY_DOUBLE_EXP) G2B_REFUSE("channel_scan: unknown form of decay %d", decay);
+  ChannelIn in = {q, k, v, low, q_stride, k_stride, v_stride, low_stride, w_low, bias, H, D, V, R, q_scale, inv_tau,
+                  decay, low_tanh, low_f32, bonus};
   if (n_tokens == n_seqs)                            // one token per sequence
     return dtype == G2B_F32 ? launch_channel_step<float>(in, state, seq_slots, n_seqs, out, stream)
                             : launch_channel_step<bf16>(in, state, seq_slots, n_seqs, out, stream);
-  if (!seq_meta || !tiles || n_tiles <= 0 || tile_rows <= 0 || !qf || !kf || !af || !seg_state || !seg_decay)
+  if (!seq_meta || !tiles || n_tiles <= 0 || tile_rows <= 0 || !qf || !kf || !af || !seg_state || !seg_decay ||
+      (bonus && !own))
     G2B_REFUSE("channel_scan: a prompt step needs its tables and scratch buffers");
   const dim3 prep_grid((n_tokens + CP_TOKENS - 1) / CP_TOKENS, H);
   const size_t prep_smem = (size_t)CP_TOKENS * R * sizeof(float);
   if (dtype == G2B_F32) {
     if (prep_smem > 48 * 1024) cudaFuncSetAttribute(channel_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem);
-    g2b_launch(channel_prep_kernel<float>, prep_grid, dim3(CP_THREADS), prep_smem, stream, in, n_tokens, qf, kf, af);
+    g2b_launch(channel_prep_kernel<float>, prep_grid, dim3(CP_THREADS), prep_smem, stream, in, n_tokens, qf, kf, af,
+               own);
   } else {
     if (prep_smem > 48 * 1024) cudaFuncSetAttribute(channel_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem);
-    g2b_launch(channel_prep_kernel<bf16>, prep_grid, dim3(CP_THREADS), prep_smem, stream, in, n_tokens, qf, kf, af);
+    g2b_launch(channel_prep_kernel<bf16>, prep_grid, dim3(CP_THREADS), prep_smem, stream, in, n_tokens, qf, kf, af,
+               own);
   }
   SegArgs a;
   a.qf = qf; a.kf = kf; a.af = af; a.v = v; a.v_stride = v_stride; a.H = H; a.D = D; a.V = V; a.tiles = (const int4 *)tiles;
   a.tile_rows = tile_rows; a.seq_meta = seq_meta; a.state = state; a.seg_state = seg_state; a.seg_decay = seg_decay; a.out = out;
+  a.own = bonus ? own : nullptr;
   a.Dp = a.tile = 0;
   int rc = 0;
   if (n_tiles > n_seqs) {                            // some sequence has several segments

@@ -59,6 +59,47 @@ extern "C" int g2b_embed_rows(const void *table, int table_dtype, const int *ids
   return g2b_check_launch("embed_rows");
 }
 
+// The same rows divided by their root mean square, times w, written `copies` times side by side: out [T, copies, H].
+template <typename TW>
+__global__ void __launch_bounds__(256)
+embed_norm_rows_kernel(const TW *__restrict__ table, const int *__restrict__ ids, const float *__restrict__ w, float eps,
+                       float *__restrict__ out, int copies, int H, int V, float scale) {
+  pdl_launch();
+  pdl_wait();
+  __shared__ float scratch[32];
+  const int t = blockIdx.x;
+  int id = ids[t];
+  const bool ok = (id >= 0 && id < V);
+  if (!ok) id = 0;                                   // host validates ids; never read outside
+  const TW *row = table + (size_t)id * H;
+  float ss = 0.f;
+  for (int j = threadIdx.x; j < H; j += blockDim.x) {
+    const float v = ok ? to_f32(row[j]) * scale : 0.f;
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
+  for (int j = threadIdx.x; j < H; j += blockDim.x) {
+    const float v = ((ok ? to_f32(row[j]) * scale : 0.f) * inv) * (w ? w[j] : 1.f);
+    for (int c = 0; c < copies; ++c) out[((size_t)t * copies + c) * H + j] = v;
+  }
+}
+
+extern "C" int g2b_embed_norm_rows(const void *table, int table_dtype, const int *ids, const float *w, float eps, float *out,
+                                   int copies, int T, int H, int V, float scale, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || V <= 0 || copies <= 0) G2B_REFUSE("embed_norm_rows: bad sizes H=%d V=%d copies=%d", H, V, copies);
+  const int threads = H >= 256 ? 256 : 64;
+  if (table_dtype == G2B_F32)
+    g2b_launch(embed_norm_rows_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float *)table, ids, w, eps, out, copies,
+               H, V, scale);
+  else if (table_dtype == G2B_BF16)
+    g2b_launch(embed_norm_rows_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16 *)table, ids, w, eps, out, copies,
+               H, V, scale);
+  else
+    G2B_REFUSE("embed_norm_rows: unknown table dtype %d", table_dtype);
+  return g2b_check_launch("embed_norm_rows");
+}
+
 // ---------------------------------------------------------------------------
 // rmsnorm over rows of the 32-bit stream; rows == nullptr means rows 0..n_rows-1;
 // w == nullptr means no per-channel weight (it was multiplied into the next matrix)
@@ -659,6 +700,93 @@ extern "C" int g2b_norm_shift(const float *x, const float *w, const float *mu, f
 }
 
 // ---------------------------------------------------------------------------
+// One row mixed with the row in front of it in several ways: out[i, t] = h_t + (h_prev - h_t) * mu[i], i < n, 32-bit
+// arithmetic on rows of the compute type.  h_prev is the row above in this step where it is the same sequence's, else
+// the sequence's kept row (`kept` [slots, H] in the compute type; zeros in front of position 0).  The block of a
+// sequence's first row reads the kept row and then replaces it with the sequence's last row of the step (an input), so
+// nobody else touches that slot's place in this launch.  A block per (token, stretch of columns); tables as above.
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+shift_mix_kernel(const T *__restrict__ h, int h_stride, const float *__restrict__ mu, int n, T *__restrict__ kept,
+                 const int *__restrict__ tok_seq, const int *__restrict__ tok_pos, const int *__restrict__ seq_slots,
+                 const int *__restrict__ seq_meta, int n_tokens, int H, T *__restrict__ out) {
+  pdl_launch();
+  pdl_wait();
+  const int t = blockIdx.x, j = blockIdx.y * 256 + threadIdx.x;
+  if (j >= H) return;
+  const int b = tok_seq[t];
+  const int first_row = seq_meta ? seq_meta[4 * b + 0] : t, rows = seq_meta ? seq_meta[4 * b + 1] : 1;
+  const int past = seq_meta ? seq_meta[4 * b + 2] : tok_pos[t];
+  const int slot = seq_meta ? seq_meta[4 * b + 3] : seq_slots[b];
+  const bool first = t == first_row;
+  T *keep = kept + (size_t)slot * H + j;
+  const T *own = h + (size_t)t * h_stride + j;
+  const float x = to_f32(*own);
+  const float d = (first ? (past > 0 ? to_f32(*keep) : 0.f) : to_f32(*(own - h_stride))) - x;
+  for (int m = 0; m < n; ++m) out[((size_t)m * n_tokens + t) * H + j] = from_f32<T>(fmaf(d, mu[(size_t)m * H + j], x));
+  if (first) *keep = h[(size_t)(first_row + rows - 1) * h_stride + j];       // this thread alone reads and writes that entry
+}
+
+// four bfloat16 neighbours a thread, 8-byte accesses
+__global__ void __launch_bounds__(256)
+shift_mix4_kernel(const bf16 *__restrict__ h, int h_stride, const float *__restrict__ mu, int n, bf16 *__restrict__ kept,
+                  const int *__restrict__ tok_seq, const int *__restrict__ tok_pos, const int *__restrict__ seq_slots,
+                  const int *__restrict__ seq_meta, int n_tokens, int H, bf16 *__restrict__ out) {
+  pdl_launch();
+  pdl_wait();
+  const int t = blockIdx.x, j = (blockIdx.y * 256 + threadIdx.x) * 4;
+  if (j >= H) return;
+  const int b = tok_seq[t];
+  const int first_row = seq_meta ? seq_meta[4 * b + 0] : t, rows = seq_meta ? seq_meta[4 * b + 1] : 1;
+  const int past = seq_meta ? seq_meta[4 * b + 2] : tok_pos[t];
+  const int slot = seq_meta ? seq_meta[4 * b + 3] : seq_slots[b];
+  const bool first = t == first_row;
+  bf16 *keep = kept + (size_t)slot * H + j;
+  const bf16 *own = h + (size_t)t * h_stride + j;
+  const uint2 xr = *reinterpret_cast<const uint2 *>(own);
+  uint2 pr = make_uint2(0u, 0u);
+  if (!first) pr = *reinterpret_cast<const uint2 *>(own - h_stride);
+  else if (past > 0) pr = *reinterpret_cast<const uint2 *>(keep);
+  const float x[4] = {__uint_as_float(xr.x << 16), __uint_as_float(xr.x & 0xffff0000u), __uint_as_float(xr.y << 16),
+                      __uint_as_float(xr.y & 0xffff0000u)};
+  const float d[4] = {__uint_as_float(pr.x << 16) - x[0], __uint_as_float(pr.x & 0xffff0000u) - x[1],
+                      __uint_as_float(pr.y << 16) - x[2], __uint_as_float(pr.y & 0xffff0000u) - x[3]};
+  for (int m = 0; m < n; ++m) {
+    const float4 w = *reinterpret_cast<const float4 *>(mu + (size_t)m * H + j);
+    uint2 r;
+    *reinterpret_cast<__nv_bfloat162 *>(&r.x) = __floats2bfloat162_rn(fmaf(d[0], w.x, x[0]), fmaf(d[1], w.y, x[1]));
+    *reinterpret_cast<__nv_bfloat162 *>(&r.y) = __floats2bfloat162_rn(fmaf(d[2], w.z, x[2]), fmaf(d[3], w.w, x[3]));
+    *reinterpret_cast<uint2 *>(out + ((size_t)m * n_tokens + t) * H + j) = r;
+  }
+  if (first) *reinterpret_cast<uint2 *>(keep) = *reinterpret_cast<const uint2 *>(h + (size_t)(first_row + rows - 1) * h_stride + j);
+}
+
+extern "C" int g2b_shift_mix(const void *h, int h_stride, const float *mu, int n, void *kept, const int *tok_seq,
+                             const int *tok_pos, const int *seq_slots, const int *seq_meta, int T_tokens, int H, void *out,
+                             int dtype, cudaStream_t stream) {
+  if (T_tokens <= 0) return 0;
+  if (!mu || n <= 0 || !kept || !tok_seq || (!seq_meta && (!tok_pos || !seq_slots)))
+    G2B_REFUSE("shift_mix: mixing weights, kept rows and the step's tables are needed");
+  if (dtype == G2B_BF16 && H % 4 == 0 && h_stride % 4 == 0 && !(((uintptr_t)h | (uintptr_t)kept | (uintptr_t)out) & 7) && !((uintptr_t)mu & 15)) {
+    g2b_launch(shift_mix4_kernel, dim3(T_tokens, (H / 4 + 255) / 256), dim3(256), 0, stream, (const bf16 *)h, h_stride, mu, n,
+               (bf16 *)kept, tok_seq, tok_pos, seq_slots, seq_meta, T_tokens, H, (bf16 *)out);
+    return g2b_check_launch("shift_mix");
+  }
+  const dim3 grid(T_tokens, (H + 255) / 256);
+  if (grid.y > 65535) G2B_REFUSE("shift_mix: rows of %d", H);
+  if (dtype == G2B_F32)
+    g2b_launch(shift_mix_kernel<float>, grid, dim3(256), 0, stream, (const float *)h, h_stride, mu, n, (float *)kept, tok_seq,
+               tok_pos, seq_slots, seq_meta, T_tokens, H, (float *)out);
+  else if (dtype == G2B_BF16)
+    g2b_launch(shift_mix_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16 *)h, h_stride, mu, n, (bf16 *)kept, tok_seq,
+               tok_pos, seq_slots, seq_meta, T_tokens, H, (bf16 *)out);
+  else
+    G2B_REFUSE("shift_mix: unknown dtype %d", dtype);
+  return g2b_check_launch("shift_mix");
+}
+
+// ---------------------------------------------------------------------------
 // SiLU gate on a fused gate/up projection.  Rows of the fused matrix alternate in
 // blocks of `blk`: columns [2*blk*b, 2*blk*b+blk) are gate_{blk*b ..}, the next blk are
 // up_{blk*b ..}; blk == I means "all gates, then all ups".
@@ -927,4 +1055,30 @@ extern "C" int g2b_relu2(const void *z, int z_stride, int dtype, int T_tokens, i
   else
     G2B_REFUSE("relu2: unknown dtype %d", dtype);
   return g2b_check_launch("relu2");
+}
+
+// out = z * sigmoid(z (c1 + c3 z^2)): an activation of glu.cuh's form without a second input
+template <typename T>
+__global__ void __launch_bounds__(256)
+act_form_kernel(const T *__restrict__ z, int z_stride, T *__restrict__ out, long long total, int F, GluForm form) {
+  pdl_launch();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= total) return;
+  out[i] = from_f32<T>(glu_value(to_f32(z[(size_t)(i / F) * z_stride + (i % F)]), 1.f, form));
+}
+
+extern "C" int g2b_act_form(const void *z, int z_stride, int dtype, int T_tokens, int F, void *out, float c1, float c3,
+                            cudaStream_t stream) {
+  if (T_tokens <= 0 || F <= 0) return 0;
+  const long long total = (long long)T_tokens * F;
+  const unsigned blocks = (unsigned)((total + 255) / 256);
+  const GluForm form = {INFINITY, 0.f, c1, c3};
+  if (dtype == G2B_F32)
+    g2b_launch(act_form_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float *)z, z_stride, (float *)out, total, F, form);
+  else if (dtype == G2B_BF16)
+    g2b_launch(act_form_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16 *)z, z_stride, (bf16 *)out, total, F, form);
+  else
+    G2B_REFUSE("act_form: unknown dtype %d", dtype);
+  return g2b_check_launch("act_form");
 }

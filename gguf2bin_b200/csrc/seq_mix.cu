@@ -7,7 +7,7 @@
 //                         at once, times a weight; rotation of the first `rot` entries of every
 //                         head, pairs (i, i + rot/2) or (2i, 2i + 1); q out, k and v into the
 //                         layer's pages.  Key and value heads may differ in size: both are
-//                         stored zero-filled to the larger, and so is q.  Options: the norm per
+//                         stored zero-filled to one row size, and so is q.  Options: the norm per
 //                         head instead (a weight of one head's size), every head of q and k
 //                         divided by its root mean square after the rotation, fewer value heads
 //                         than key heads, and no keys and values at all (q only).
@@ -70,14 +70,13 @@ proj_norm_rope_cache_kernel(const T *__restrict__ qkv, int row_stride, const flo
                             int rot, int interleaved, const int *__restrict__ tok_pos,
                             const int *__restrict__ tok_seq, const int *__restrict__ page_table, int P,
                             T *__restrict__ cache, int page_size, T *__restrict__ q_out, float v_norm_eps,
-                            int norm_per_head, float unit_eps, int nvh) {
+                            int norm_per_head, float unit_eps, int nvh, int hd) {
   pdl_launch();
   pdl_wait();
   extern __shared__ float sm[];                     // q [nh*D], k [nkv*D], one factor per value head [nvh]
   __shared__ float scratch[32];
   const int t = blockIdx.x;
   const int nq = nh * D, nk = nkv * D;
-  const int hd = D > V ? D : V;
   const T *src = qkv + (size_t)t * row_stride;
   float *xq = sm, *xk = sm + nq;
   float sq = 0.f, sk = 0.f;
@@ -162,7 +161,7 @@ proj_norm_rope_cache_kernel(const T *__restrict__ qkv, int row_stride, const flo
 // The same prologue where nothing spans the heads (no norm over the whole projection): a warp a (token, head),
 // no block-wide wait.  Heads count through q (nh), then keys (nkv), then values (nvh); every warp stages its head
 // in shared memory, norms it (a weight of one head's size), rotates it, may divide it by its root mean square,
-// and writes it out: q into q_out, keys and values into the token's page, all zero-filled to hd = max(D, V).
+// and writes it out: q into q_out, keys and values into the token's page, all zero-filled to hd (at least D and V).
 #define HEADWISE_WARPS 8
 template <typename T>
 __global__ void __launch_bounds__(HEADWISE_WARPS * 32)
@@ -172,7 +171,7 @@ proj_rope_cache_headwise_kernel(const T *__restrict__ qkv, int row_stride, const
                                 const int *__restrict__ tok_pos, const int *__restrict__ tok_seq,
                                 const int *__restrict__ page_table, int P, T *__restrict__ cache, int page_size,
                                 T *__restrict__ q_out, float v_norm_eps, int norm_per_head, float unit_eps, int nvh,
-                                long long n_items) {
+                                int hd, long long n_items) {
   pdl_launch();
   pdl_wait();
   extern __shared__ float sm[];                     // a head per warp
@@ -181,7 +180,6 @@ proj_rope_cache_headwise_kernel(const T *__restrict__ qkv, int row_stride, const
   if (item >= n_items) return;
   const int heads = nh + nkv + nvh;
   const int t = (int)(item / heads), h = (int)(item % heads);
-  const int hd = D > V ? D : V;
   const bool is_v = h >= nh + nkv;
   const int n = is_v ? V : D;                       // entries of this head
   const int col = is_v ? (nh + nkv) * D + (h - nh - nkv) * V : h * D;
@@ -233,13 +231,13 @@ extern "C" int g2b_proj_norm_rope_cache(const void *qkv, int dtype, int row_stri
                                         const float *k_w, float eps, const float *rope, int rot, int interleaved,
                                         const int *tok_pos, const int *tok_seq, const int *page_table, int P,
                                         void *cache, int page_size, void *q_out, float v_norm_eps,
-                                        int norm_per_head, float unit_eps, int nvh, cudaStream_t stream) {
+                                        int norm_per_head, float unit_eps, int nvh, int hd, cudaStream_t stream) {
   if (T_tokens <= 0) return 0;
   if (rope && (rot <= 0 || rot > D || (rot & 1))) G2B_REFUSE("proj_norm_rope_cache: %d rotated entries of a head of %d", rot, D);
   if (nkv < 0 || nvh < 0 || nvh > nkv) G2B_REFUSE("proj_norm_rope_cache: %d value heads beside %d key heads", nvh, nkv);
+  if (hd < D || hd < V) G2B_REFUSE("proj_norm_rope_cache: heads of %d and %d in rows of %d", D, V, hd);
   if (nkv > 0 && !cache) G2B_REFUSE("proj_norm_rope_cache: keys without pages to write them to");
   if (norm_per_head || (!q_w && !k_w)) {                // nothing spans the heads: a warp a (token, head)
-    const int hd = D > V ? D : V;
     const long long n_items = (long long)T_tokens * (nh + nkv + nvh);
     const long long blocks = (n_items + HEADWISE_WARPS - 1) / HEADWISE_WARPS;
     const size_t smem_h = (size_t)HEADWISE_WARPS * hd * sizeof(float);
@@ -248,12 +246,12 @@ extern "C" int g2b_proj_norm_rope_cache(const void *qkv, int dtype, int row_stri
         g2b_launch(proj_rope_cache_headwise_kernel<float>, dim3((unsigned)blocks), dim3(HEADWISE_WARPS * 32), smem_h, stream,
                    (const float *)qkv, row_stride, bias, nh, nkv, D, V, q_w, k_w, eps, (const float2 *)rope, rot, interleaved,
                    tok_pos, tok_seq, page_table, P, (float *)cache, page_size, (float *)q_out, v_norm_eps, norm_per_head,
-                   unit_eps, nvh, n_items);
+                   unit_eps, nvh, hd, n_items);
       else if (dtype == G2B_BF16)
         g2b_launch(proj_rope_cache_headwise_kernel<bf16>, dim3((unsigned)blocks), dim3(HEADWISE_WARPS * 32), smem_h, stream,
                    (const bf16 *)qkv, row_stride, bias, nh, nkv, D, V, q_w, k_w, eps, (const float2 *)rope, rot, interleaved,
                    tok_pos, tok_seq, page_table, P, (bf16 *)cache, page_size, (bf16 *)q_out, v_norm_eps, norm_per_head,
-                   unit_eps, nvh, n_items);
+                   unit_eps, nvh, hd, n_items);
       else
         G2B_REFUSE("proj_norm_rope_cache: unknown dtype %d", dtype);
       return g2b_check_launch("proj_norm_rope_cache");
@@ -266,13 +264,13 @@ extern "C" int g2b_proj_norm_rope_cache(const void *qkv, int dtype, int row_stri
     if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     g2b_launch(k, dim3(T_tokens), dim3(256), smem, stream, (const float *)qkv, row_stride, bias, nh, nkv, D, V, q_w, k_w,
                eps, (const float2 *)rope, rot, interleaved, tok_pos, tok_seq, page_table, P, (float *)cache, page_size,
-               (float *)q_out, v_norm_eps, norm_per_head, unit_eps, nvh);
+               (float *)q_out, v_norm_eps, norm_per_head, unit_eps, nvh, hd);
   } else if (dtype == G2B_BF16) {
     auto k = proj_norm_rope_cache_kernel<bf16>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     g2b_launch(k, dim3(T_tokens), dim3(256), smem, stream, (const bf16 *)qkv, row_stride, bias, nh, nkv, D, V, q_w, k_w,
                eps, (const float2 *)rope, rot, interleaved, tok_pos, tok_seq, page_table, P, (bf16 *)cache, page_size,
-               (bf16 *)q_out, v_norm_eps, norm_per_head, unit_eps, nvh);
+               (bf16 *)q_out, v_norm_eps, norm_per_head, unit_eps, nvh, hd);
   } else {
     G2B_REFUSE("proj_norm_rope_cache: unknown dtype %d", dtype);
   }

@@ -429,6 +429,82 @@ extern "C" int g2b_latent_pair(const void *d, int rank, int width, const float *
 }
 
 // ---------------------------------------------------------------------------
+// a latent with rotated entries behind it: d [T, rank + rot] becomes a row of `width` in the page of the token's
+// position, the first `rank` entries divided by their root mean square and times norm_w, the next `rot` turned by the
+// step's (cos, sin) table, zeros behind them; and the last `rot` entries of every query head are turned on their way
+// from q_in (head h at column h * in_head) to q_out (at h * out_head; the two may be the same place).  A block a token:
+// its first warp makes the row, where there is one (d null: another layer's rows are read), the others turn queries.
+// ---------------------------------------------------------------------------
+#define LROPE_WARPS 4
+template <typename TA>
+__global__ void __launch_bounds__(LROPE_WARPS * 32)
+latent_rope_kernel(const TA *__restrict__ d, int d_stride, int rank, int rot, int width, const float *__restrict__ norm_w,
+                   float eps, TA *__restrict__ pages, const int *__restrict__ page_table, int P, int page_size,
+                   const int *__restrict__ tok_pos, const int *__restrict__ tok_seq, const TA *q_in, int in_stride,
+                   int in_head, TA *q_out, int out_stride, int out_head, int heads, const float2 *__restrict__ rope,
+                   int interleaved) {
+  pdl_launch();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int half = rot >> 1;
+  const float2 *cs = rope + (size_t)t * half;
+  if (d && warp == 0) {
+    const TA *src = d + (size_t)t * d_stride;
+    const int pos = tok_pos[t];
+    const int page = page_table[(size_t)tok_seq[t] * P + pos / page_size];
+    TA *dst = pages + ((size_t)page * page_size + pos % page_size) * width;
+    float ss = 0.f;
+    for (int j = lane; j < rank; j += 32) {
+      const float v = to_f32(src[j]);
+      ss = fmaf(v, v, ss);
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)rank + eps);
+    for (int j = lane; j < rank; j += 32) dst[j] = from_f32<TA>((to_f32(src[j]) * inv) * norm_w[j]);
+    for (int i = lane; i < half; i += 32) {
+      const float2 r = cs[i];
+      const int a = rank + (interleaved ? 2 * i : i), b = rank + (interleaved ? 2 * i + 1 : i + half);
+      const float u = to_f32(src[a]), v = to_f32(src[b]);
+      dst[a] = from_f32<TA>(u * r.x - v * r.y);
+      dst[b] = from_f32<TA>(v * r.x + u * r.y);
+    }
+    for (int j = rank + rot + lane; j < width; j += 32) dst[j] = from_f32<TA>(0.f);
+    return;
+  }
+  const int w0 = d ? warp - 1 : warp, warps = d ? LROPE_WARPS - 1 : LROPE_WARPS;
+  const TA *qi = q_in + (size_t)t * in_stride;
+  TA *qo = q_out + (size_t)t * out_stride;
+  for (int i = w0 * 32 + lane; i < heads * half; i += warps * 32) {
+    const int h = i / half, k = i - h * half;
+    const float2 r = cs[k];
+    const int a = interleaved ? 2 * k : k, b = interleaved ? 2 * k + 1 : k + half;
+    const float u = to_f32(qi[(size_t)h * in_head + a]), v = to_f32(qi[(size_t)h * in_head + b]);
+    qo[(size_t)h * out_head + a] = from_f32<TA>(u * r.x - v * r.y);
+    qo[(size_t)h * out_head + b] = from_f32<TA>(v * r.x + u * r.y);
+  }
+}
+
+extern "C" int g2b_latent_rope(const void *d, int d_stride, int rank, int rot, int width, const float *norm_w, float eps,
+                               void *pages, const int *page_table, int P, int page_size, const int *tok_pos,
+                               const int *tok_seq, const void *q_in, int in_stride, int in_head, void *q_out, int out_stride,
+                               int out_head, int heads, const float *rope, int interleaved, int T, int dtype,
+                               cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (rot <= 0 || (rot & 1) || heads <= 0 || !rope) G2B_REFUSE("latent_rope: %d rotated entries of %d heads", rot, heads);
+  if (d && (rank <= 0 || width < rank + rot || page_size <= 0)) G2B_REFUSE("latent_rope: %d + %d entries in rows of %d", rank, rot, width);
+  if (dtype == G2B_F32)
+    g2b_launch(latent_rope_kernel<float>, dim3(T), dim3(LROPE_WARPS * 32), 0, stream, (const float *)d, d_stride, rank, rot, width,
+               norm_w, eps, (float *)pages, page_table, P, page_size, tok_pos, tok_seq, (const float *)q_in, in_stride, in_head,
+               (float *)q_out, out_stride, out_head, heads, (const float2 *)rope, interleaved);
+  else if (dtype == G2B_BF16)
+    g2b_launch(latent_rope_kernel<bf16>, dim3(T), dim3(LROPE_WARPS * 32), 0, stream, (const bf16 *)d, d_stride, rank, rot, width,
+               norm_w, eps, (bf16 *)pages, page_table, P, page_size, tok_pos, tok_seq, (const bf16 *)q_in, in_stride, in_head,
+               (bf16 *)q_out, out_stride, out_head, heads, (const float2 *)rope, interleaved);
+  else
+    G2B_REFUSE("latent_rope: unknown dtype %d", dtype);
+  return g2b_check_launch("latent_rope");
+}
+
+// ---------------------------------------------------------------------------
 // products with one small matrix per head.  W [heads * n, r] (rows of head h: h*n .. h*n+n-1).
 //   absorb: out[t, h, 0..r)  = sum_i W[h*n + i, :] * in[t, h, i]        (W_h^T applied; in has n per head)
 //   expand: out[t, h, 0..n)  = W[h*n + i, :] . in[t, h, :], times sigmoid(gate[t, h]) when gate

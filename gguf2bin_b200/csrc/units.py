@@ -5,7 +5,7 @@ from __future__ import annotations
 
 GENERIC_UNITS = [("elementwise.cu", ()), ("gemm_simt.cu", ()), ("attn_generic.cu", ()),
                  ("sampling.cu", ()), ("random_init.cu", ()), ("stream_ops.cu", ()),
-                 ("seq_mix.cu", ()), ("moe.cu", ()), ("channel_scan.cu", ())]
+                 ("seq_mix.cu", ()), ("moe.cu", ()), ("channel_scan.cu", ()), ("streams.cu", ())]
 
 # head sizes built ahead of time (what the tests and the benchmark use)
 HEAD_SIZES = (64, 128)

@@ -19,7 +19,7 @@ from ..config.specs import ConfigError
 from ..csrc.build import _log
 from ..parts import block_class, embedding_class, head_class, norm_class
 from ..parts.base import StepContext
-from ..parts.norms import bind_norm
+from ..parts.norms import RMSNorm, bind_norm
 from ..weights.loader import load_weights
 
 _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.float32,
@@ -67,6 +67,7 @@ class Model:
         self.head = head_class(spec.head)(spec.head, spec.vocab_size, spec.hidden_size, self.dtype,
                                           self.device)
         self.n_params = 0
+        self.streams = spec.streams
         self.rejoins = any(e.add_embedding for e in spec.schedule)
 
     # ---- construction ---------------------------------------------------------
@@ -181,10 +182,12 @@ class Model:
         with ``n_want == 0`` only the cache is updated."""
         ws = ctx.workspace
         ctx.step_cache.clear()                     # per-step tables are rebuilt from this step's tokens
-        x = ws.buffer("stream", (ctx.n_tokens, self.hidden), torch.float32)
+        x = ws.buffer("stream", (ctx.n_tokens, self.hidden), torch.float32) if self.streams == 1 else None
         # the embedding's output, kept where a later position of the schedule adds it to the stream again
         start = ws.buffer("stream.start", (ctx.n_tokens, self.hidden), torch.float32) if self.rejoins else None
-        if hasattr(self.embedding, "cache_need"):
+        if x is None:
+            x = self._spread_embedding(ctx, cache)
+        elif hasattr(self.embedding, "cache_need"):
             # an embedding that keeps something per sequence (the previous token, say) has the
             # storage of one more position behind the schedule's
             self.embedding.forward(ctx.tok_ids[:ctx.n_tokens], x, ctx, cache.view(len(self.spec.schedule)))
@@ -213,6 +216,24 @@ class Model:
         logits = logits_out if logits_out is not None else \
             ws.buffer("head.logits", (n_want, self.vocab), torch.float32)
         h = ws.buffer("head.normed", (n_want, self.hidden), self.dtype)
-        self.final_norm.forward(x, h, want_rows)
+        if self.streams > 1 and isinstance(self.final_norm, RMSNorm):
+            kernels.streams_read(x, None, self.final_norm.weight, self.final_norm.eps, h, want_rows)
+        else:
+            self.final_norm.forward(x if self.streams == 1 else x.sum(dim=1), h, want_rows)
         self.head.forward(h, logits, ctx)
         return logits
+
+    def _spread_embedding(self, ctx: StepContext, cache: Cache) -> torch.Tensor:
+        """The streams in front of the first layer, float32 [tokens, streams, hidden]: the embedding's row in every one."""
+        ids, e = ctx.tok_ids[:ctx.n_tokens], self.embedding
+        x = ctx.workspace.buffer("streams", (ctx.n_tokens, self.streams, self.hidden), torch.float32)
+        if getattr(e, "writes_copies", False):
+            e.forward(ids, x, ctx)
+            return x
+        row = ctx.workspace.buffer("stream", (ctx.n_tokens, self.hidden), torch.float32)
+        if hasattr(e, "cache_need"):
+            e.forward(ids, row, ctx, cache.view(len(self.spec.schedule)))
+        else:
+            e.forward(ids, row, ctx)
+        x.copy_(row[:, None, :].expand_as(x))
+        return x

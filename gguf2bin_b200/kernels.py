@@ -22,7 +22,7 @@ __all__ = ["KernelError", "KernelBuildError", "embed_rows", "rmsnorm", "qknorm_r
            "canon_conv", "norm_canon_single", "latent_keep", "head_product", "head_gate", "gated_add", "xielu",
            "proj_norm_rope_cache", "rotate_heads", "short_conv", "state_scan", "head_norm_gate", "gate_mul",
            "norm_add", "norm_shift", "scan_gates_step", "scan_gates_max", "state_readout", "pool_update", "moe_route", "moe_plan", "moe_gemm", "moe_gemv", "moe_gather", "moe_gemm_tc", "moe_combine", "moe_combine_norm_add", "moe_tile_rows", "tanh_norm", "scaled_join", "relu2", "selective_scan", "diff_combine", "GluForm", "norm_join", "moe_combine_join", "latent_pair",
-           "channel_scan", "stream_add"]
+           "channel_scan", "stream_add", "embed_norm_rows", "streams_read", "streams_join", "shift_mix", "latent_rope", "act_form"]
 
 F32, BF16 = 0, 1
 EPI_STORE_F32, EPI_STORE_BF16, EPI_ACCUM_F32 = 0, 1, 2
@@ -171,6 +171,21 @@ def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale:
           _ptr(again), _stream())
 
 
+def embed_norm_rows(table: torch.Tensor, ids: torch.Tensor, w, eps: float, out: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t, c] = the row table[ids[t]] * scale over its root mean square, times ``w``, in 32-bit, once for every c;
+    ids int32 [T], out float32 [T, copies, H] (or [T, H])."""
+    _need(ids, torch.int32, "ids")
+    _need(out, torch.float32, "out")
+    if w is not None:
+        _need(w, torch.float32, "norm weight")
+    V, H = table.shape
+    copies = out.shape[1] if out.dim() == 3 else 1
+    f = _fn("elementwise.cu", "g2b_embed_norm_rows",
+            [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    _call(f, _ptr(table), _code(table.dtype), _ptr(ids), _ptr(w), float(eps), _ptr(out), copies, out.shape[0], H, V,
+          float(scale), _stream())
+
+
 def stream_add(x32: torch.Tensor, y32: torch.Tensor) -> None:
     """x += y, both float32 of one shape: what a model adds to its stream between two layers where no kernel of
     the layers takes it along."""
@@ -240,6 +255,17 @@ def relu2(z, out) -> None:
         raise KernelError("relu2: dense rows of one dtype")
     f = _fn("elementwise.cu", "g2b_relu2", [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     _call(f, _ptr(z), z.stride(0), _code(z.dtype), z.shape[0], z.shape[1], _ptr(out), _stream())
+
+
+def act_form(z, out, form: "GluForm") -> None:
+    """out = z sigmoid(z (c1 + c3 z^2)) with the numbers of ``form`` (``GluForm.gelu_tanh()``: the tanh form of GELU);
+    z [T, F] a view with any row stride, out [T, F] contiguous, one dtype."""
+    if z.stride(1) != 1 or out.dtype != z.dtype or not out.is_contiguous():
+        raise KernelError("act_form: dense rows of one dtype")
+    if form.offset or form.limit != math.inf:
+        raise KernelError("act_form: an activation has neither an offset nor a limit")
+    f = _fn("elementwise.cu", "g2b_act_form", [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_void_p])
+    _call(f, _ptr(z), z.stride(0), _code(z.dtype), z.shape[0], z.shape[1], _ptr(out), form.c1, form.c3, _stream())
 
 
 def rope_table(tok_pos: torch.Tensor, inv_freq: torch.Tensor, table: torch.Tensor, mult: float = 1.0) -> None:
@@ -317,6 +343,21 @@ def norm_shift(x32, w, mu, kept, ctx, eps: float, h_out, hs_out) -> None:
     _call(f, _ptr(x32), _ptr(w), _ptr(mu), _ptr(kept), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(ctx.seq_slots),
           _ptr(ctx.seq_meta), T, H, float(eps),
           _ptr(h_out), _ptr(hs_out), _code(h_out.dtype), _stream())
+
+
+def shift_mix(h, mu, kept, ctx, out) -> None:
+    """out[i, t] = h_t + (h_prev - h_t) * mu[i]: every row mixed with the row in front of it in its sequence, in as many
+    ways as ``mu`` (float32 [n, H]) has rows; ``kept`` [slots, H] (h's dtype) holds every sequence's last row between
+    steps and is brought up to date (zeros in front of position 0).  h [T, H], rows may lie apart; out [n, T, H]."""
+    _need(mu, torch.float32, "mixing weights")
+    n, H = mu.shape
+    if kept.dtype != h.dtype or out.dtype != h.dtype or not out.is_contiguous() or tuple(out.shape) != (n, h.shape[0], H):
+        raise KernelError("shift_mix: rows, kept rows and output have one dtype, the output is [mixes, tokens, width]")
+    f = _fn("elementwise.cu", "g2b_shift_mix",
+            [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
+             c_int, c_void_p])
+    _call(f, _ptr(h), _dense_rows(h, "h"), _ptr(mu), n, _ptr(kept), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(ctx.seq_slots),
+          _ptr(ctx.seq_meta), h.shape[0], H, _ptr(out), _code(h.dtype), _stream())
 
 
 def advance_positions(tok_pos: torch.Tensor, n: int) -> None:
@@ -438,6 +479,29 @@ def latent_pair(d, width: int, d_w, pages, e, e_w, e_out, eps: float, ctx) -> No
     _call(f, _ptr(d), d.shape[1], width, _ptr(d_w), _ptr(pages), _ptr(ctx.page_table), ctx.page_table.shape[1],
           ctx.page_size, _ptr(ctx.tok_pos), _ptr(ctx.tok_seq), _ptr(e), e.shape[1], _ptr(e_w), _ptr(e_out), d.stride(0),
           float(eps), d.shape[0], _code(d.dtype), _stream())
+
+
+def latent_rope(d, rank: int, width: int, norm_w, eps: float, pages, q_in, in_head: int, q_out, out_head: int, heads: int,
+                rot: int, rope, interleaved: bool, ctx) -> None:
+    """A latent with rotated entries behind it, and the queries' rotated entries.  d [T, rank + rot] (None: another layer's
+    rows are read): its first ``rank`` entries over their root mean square times ``norm_w``, then the ``rot`` others turned
+    by the step's ``rope`` table, into the pages at the tokens' positions, rows of ``width`` entries with zeros behind.
+    Head h's ``rot`` entries of ``q_in`` (from column h * in_head) turn on their way to ``q_out`` (from h * out_head); the
+    two may be one place."""
+    _need(rope, torch.float32, "rotation table")
+    if q_in.dtype != q_out.dtype or (d is not None and (d.dtype != q_in.dtype or pages.dtype != d.dtype or d.shape[1] != rank + rot
+                                                        or pages.shape[-1] != width)):
+        raise KernelError("latent_rope: latents, queries and pages have one dtype, pages rows of the given width")
+    if d is not None:
+        _need(norm_w, torch.float32, "latent norm weight")
+    f = _fn("stream_ops.cu", "g2b_latent_rope",
+            [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
+             c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
+    _call(f, _ptr(d), _dense_rows(d, "latents") if d is not None else 0, rank, rot, width, _ptr(norm_w) if d is not None else None,
+          float(eps), _ptr(pages) if d is not None else None, _ptr(ctx.page_table), ctx.page_table.shape[1], ctx.page_size,
+          _ptr(ctx.tok_pos), _ptr(ctx.tok_seq), _ptr(q_in), _dense_rows(q_in, "queries"), in_head, _ptr(q_out),
+          _dense_rows(q_out, "queries"), out_head, heads, _ptr(rope), 1 if interleaved else 0, q_in.shape[0],
+          _code(q_in.dtype), _stream())
 
 
 def head_product(x, w, out, heads: int, expand: bool, gate=None) -> None:
@@ -743,11 +807,12 @@ def _dense_rows(t: torch.Tensor, what: str) -> int:
 
 def proj_norm_rope_cache(qkv, bias, n_heads, n_kv_heads, qk_dim, v_dim, q_w, k_w, eps, rope, rotary_dim,
                          interleaved, ctx, cache_pages, page_size, q_out, v_norm_eps: float = 0.0,
-                         norm_per_head: bool = False, unit_eps: float = 0.0, n_v_heads: Optional[int] = None) -> None:
+                         norm_per_head: bool = False, unit_eps: float = 0.0, n_v_heads: Optional[int] = None,
+                         store_dim: int = 0) -> None:
     """q, k, v side by side in ``qkv`` [T, nh*D + nkv*D + nkv*V] (+ ``bias``, float32); RMS norm over
     ALL of q and over all of k (weights ``q_w`` [nh*D], ``k_w`` [nkv*D]; None: no norm); rotation by
     the step's ``rope`` table, pairs (i, i + r/2) or, ``interleaved``, (2i, 2i + 1); q to ``q_out``
-    [T, nh*hd] and k, v into the pages, heads zero-filled to hd = max(D, V).  ``v_norm_eps`` > 0: every
+    [T, nh*hd] and k, v into the pages, heads zero-filled to hd = max(D, V) (or ``store_dim``).  ``v_norm_eps`` > 0: every
     value head is divided by its root mean square (that eps inside the root) before it is stored.
     ``norm_per_head``: the norm runs over every head of q and k by itself, the weights ``q_w``, ``k_w`` [D]
     shared by the heads.  ``unit_eps`` > 0: after the rotation every head of q and k is divided by its
@@ -757,7 +822,7 @@ def proj_norm_rope_cache(qkv, bias, n_heads, n_kv_heads, qk_dim, v_dim, q_w, k_w
     f = _fn("seq_mix.cu", "g2b_proj_norm_rope_cache",
             [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
              c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float,
-             c_int, c_float, c_int, c_void_p])
+             c_int, c_float, c_int, c_int, c_void_p])
     if q_out.dtype != qkv.dtype or (cache_pages is not None and cache_pages.dtype != qkv.dtype) or not q_out.is_contiguous():
         raise KernelError("proj_norm_rope_cache: q_out and the cache must have the input's dtype")
     for t in (bias, q_w, k_w):
@@ -767,7 +832,7 @@ def proj_norm_rope_cache(qkv, bias, n_heads, n_kv_heads, qk_dim, v_dim, q_w, k_w
           qk_dim, v_dim, _ptr(q_w), _ptr(k_w), eps, _ptr(rope), rotary_dim, 1 if interleaved else 0,
           _ptr(ctx.tok_pos), _ptr(ctx.tok_seq), _ptr(ctx.page_table), ctx.page_table.shape[1],
           _ptr(cache_pages), page_size, _ptr(q_out), float(v_norm_eps), 1 if norm_per_head else 0, float(unit_eps),
-          n_kv_heads if n_v_heads is None else int(n_v_heads), _stream())
+          n_kv_heads if n_v_heads is None else int(n_v_heads), int(store_dim) or max(qk_dim, v_dim), _stream())
 
 
 def rotate_heads(x, heads, head_dim, rope, rotary_dim, interleaved, scale: float = 1.0) -> None:
@@ -1160,11 +1225,14 @@ CHANNEL_TILES_WIDE_FROM = 4096      # tokens of a step from which its segments a
 
 
 def channel_scan(q, k, v, low, w_low, bias32, state, ctx, out32, heads: int, qk_dim: int, v_dim: int, q_scale: float,
-                 tau: float) -> None:
+                 tau: float = 1.0, *, decay: str = "sigmoid_root", low_tanh: bool = False, bonus=None) -> None:
     """S <- diag(a_t) S + k_t v_t^T, o_t = S^T (q_t q_scale) per head, a_t = sigmoid(w_low low_t + bias)^(1/tau) per key
     channel; over the step's tokens in order, 32-bit.  q, k [T, heads*qk_dim], v [T, heads*v_dim], low [T, R]: rows of
     wider buffers in the compute type; ``w_low`` [heads*qk_dim, R] (R a multiple of 8), ``bias32`` float32; ``state``
     float32 [slots, heads, v_dim, qk_dim] is read and left up to date; ``out32`` float32 [T, heads*v_dim].
+    ``decay`` = "double_exp": a_t = exp(-exp(w_low low_t + bias)) instead.  ``low_tanh``: the entries of low pass tanh
+    first.  ``low`` may be float32 beside bfloat16 q, k and v.  ``bonus`` (float32 [heads, qk_dim]): the read-out comes
+    before the update and counts the token's own key ``bonus`` times, o_t = (S + diag(bonus) k_t v_t^T)^T q_t.
     A prompt step walks the segments of its sequences (the tiles of the attention's work list) side by side."""
     T, R = q.shape[0], w_low.shape[1]
     for t, what in ((state, "state"), (out32, "scan output"), (bias32, "decay bias")):
@@ -1173,13 +1241,19 @@ def channel_scan(q, k, v, low, w_low, bias32, state, ctx, out32, heads: int, qk_
             or w_low.shape[0] != heads * qk_dim or low.shape[1] != R or not w_low.is_contiguous():
         raise KernelError(f"channel_scan: state {tuple(state.shape)}, output {tuple(out32.shape)} or decay matrix "
                           f"{tuple(w_low.shape)} do not fit {heads} heads of {v_dim} columns of {qk_dim}")
-    if any(t.dtype != q.dtype for t in (k, v, low, w_low)):
-        raise KernelError("channel_scan: q, k, v, low and the decay matrix must have one dtype")
+    if any(t.dtype != q.dtype for t in (k, v, w_low)) or low.dtype not in (q.dtype, torch.float32):
+        raise KernelError("channel_scan: q, k, v, the decay matrix and low must have one dtype (low may be float32)")
+    if decay not in ("sigmoid_root", "double_exp"):
+        raise KernelError(f"channel_scan: no decay of form {decay!r}")
+    if bonus is not None:
+        _need(bonus, torch.float32, "bonus")
+        if bonus.numel() != heads * qk_dim:
+            raise KernelError("channel_scan: one bonus per head and key channel")
     f = _fn("channel_scan.cu", "g2b_channel_scan",
             [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-             c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
-             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
-    tiles, n_tiles, rows, scratch = None, 0, 0, (None,) * 5
+             c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+             c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
+    tiles, n_tiles, rows, scratch, own = None, 0, 0, (None,) * 5, None
     if T > ctx.n_seqs:
         wide = T >= CHANNEL_TILES_WIDE_FROM
         tiles, n_tiles, rows = (ctx.attn_tiles_wide, ctx.n_attn_tiles_wide, 128) if wide else \
@@ -1189,8 +1263,60 @@ def channel_scan(q, k, v, low, w_low, bias32, state, ctx, out32, heads: int, qk_
         scratch = tuple(ws.buffer(f"channel.{n}", (T, heads * qk_dim), f32) for n in ("q", "k", "decay")) + (
             ws.buffer("channel.states", (segments, heads, v_dim, qk_dim), f32),
             ws.buffer("channel.decays", (segments, heads, qk_dim), f32))
+        if bonus is not None:
+            own = ws.buffer("channel.own", (T, heads), f32)
         count_launches(3 if n_tiles > ctx.n_seqs else 1)
     _call(f, _code(q.dtype), _ptr(q), _dense_rows(q, "q"), _ptr(k), _dense_rows(k, "k"), _ptr(v), _dense_rows(v, "v"),
           _ptr(low), _dense_rows(low, "low"), _ptr(w_low), _ptr(bias32), heads, qk_dim, v_dim, R, float(q_scale),
-          1.0 / float(tau), _ptr(state), _ptr(ctx.seq_slots), _ptr(ctx.seq_meta), T, ctx.n_seqs, _ptr(tiles), n_tiles, rows,
+          1.0 / float(tau), 1 if decay == "double_exp" else 0, 1 if low_tanh else 0,
+          1 if low.dtype == torch.float32 else 0, _ptr(bonus), _ptr(own), _ptr(state), _ptr(ctx.seq_slots), _ptr(ctx.seq_meta), T, ctx.n_seqs, _ptr(tiles), n_tiles, rows,
           *(_ptr(t) for t in scratch), _ptr(out32), _stream())
+
+
+# ---------------------------------------------------------------------------
+# streams.cu: several residual streams side by side
+# ---------------------------------------------------------------------------
+MAX_STREAMS = 16
+
+
+def _streams_check(X, *coefficients) -> None:
+    _need(X, torch.float32, "streams")
+    if X.dim() != 3 or not 1 <= X.shape[1] <= MAX_STREAMS:
+        raise KernelError(f"streams: [tokens, 1 to {MAX_STREAMS} streams, width], not {list(X.shape)}")
+    for t, n in coefficients:
+        if t is not None:
+            _need(t, torch.float32, "streams' coefficients and weights")
+            if t.numel() != n:
+                raise KernelError(f"streams: {t.numel()} coefficients or weights where {n} are needed")
+
+
+def streams_read(X, a, w, eps: float, out, rows: Optional[torch.Tensor] = None) -> None:
+    """out[r] = u / sqrt(mean(u^2) + eps) * w with u = sum_s a[s] X[row_r, s] (``a`` None: ones); X float32 [T, S, H],
+    ``rows`` (int32) gathers tokens."""
+    T, S, H = X.shape
+    _streams_check(X, (a, S), (w, H))
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    if not out.is_contiguous() or out.shape[1] != H:
+        raise KernelError("streams_read: a contiguous output of the streams' width")
+    f = _fn("streams.cu", "g2b_streams_read",
+            [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p])
+    _call(f, _ptr(X), _ptr(a), _ptr(w), float(eps), _ptr(rows), out.shape[0], S, H, _ptr(out), _code(out.dtype), _stream())
+
+
+def streams_join(X, y32, mix, out_w, mult: float, next_read=None, next_out=None) -> None:
+    """X[:, t] = sum_s mix[s, t] X[:, s] + mult * out_w[t] * y, every stream from the old ones; X float32 [T, S, H], y float32
+    [T, H].  ``next_read`` = (a, w, eps) with ``next_out`` [T, H] (compute type): what ``streams_read`` would make of the
+    new streams, in the same pass."""
+    T, S, H = X.shape
+    a, w, eps = next_read if next_read is not None else (None, None, 0.0)
+    _streams_check(X, (mix, S * S), (out_w, S), (a, S), (w, H))
+    _need(y32, torch.float32, "sublayer output")
+    if (next_read is None) != (next_out is None) or tuple(y32.shape) != (T, H) \
+            or (next_out is not None and (tuple(next_out.shape) != (T, H) or not next_out.is_contiguous())):
+        raise KernelError("streams_join: a result, and the next reader with its output, of the streams' tokens and width")
+    f = _fn("streams.cu", "g2b_streams_join",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int,
+             c_void_p])
+    _call(f, _ptr(X), _ptr(y32), _ptr(mix), _ptr(out_w), float(mult), T, S, H, _ptr(a), _ptr(w), float(eps), _ptr(next_out),
+          _code(next_out.dtype) if next_out is not None else F32, _stream())

@@ -9,7 +9,9 @@ it, and the mixer's copy is mixed with the token before, channel by channel.
 ``parallel_scaled``: h = norm(x); x += s1 * mixer(h) + s2 * feed_forward(h): one norm of any registered kind,
 both sublayers read it, and each result is multiplied by a learned number per channel before the sum.
 ``sandwich_norm``: x += norm(mixer(norm(x))); x += norm(feed_forward(norm(x))): an RMS norm on either side of every
-sublayer."""
+sublayer.
+``hyper_prenorm``: several streams instead of one x; a sublayer reads a weighted sum of them, normed, and its result
+joins every stream together with a mix of all of them."""
 from __future__ import annotations
 
 import torch
@@ -657,7 +659,126 @@ class SandwichNormBlock:
         kernels.norm_join(x32, y, norm.weight, norm.eps, self._next(after), h if after is not None else None, add)
 
 
+class HyperPreNormBlock:
+    """``hyper_prenorm`` (hyper-connections): the stream is ``streams`` rows x_1 .. x_s a token.  A sublayer q reads
+    u = sum_s in_q[s] x_s, y = f(norm(u)), and then, all streams at once from the old ones,
+    x_t <- sum_s mix_q[s, t] x_s + residual_mult * out_q[t] * y.  The coefficients are stored tensors ([s], [s, s], [s];
+    names ``mixer_in``, ``mixer_mix``, ``mixer_out`` and ``ffn_...``).  A layer may have no feed-forward.  Any mixer and
+    feed-forward of the library fit: a sublayer stores into a 32-bit buffer where it can (``forward_store``,
+    ``forward_into``) and adds into a cleared one where it cannot.
+
+    One launch a sublayer does everything between two products: the mix of the streams, the result's share, and the
+    next sublayer's weighted sum and norm, the next block's among them (``StepContext.step_cache`` hands its rows over)."""
+
+    def __init__(self, layer: LayerSpec, hidden_size: int, dtype: torch.dtype, device):
+        self.names = dict(layer.block["names"])
+        self.hidden, self.dtype = int(hidden_size), dtype
+        self.streams = int(layer.block["streams"])
+        if not 1 <= self.streams <= kernels.MAX_STREAMS:
+            raise ConfigError(f"hyper_prenorm: {self.streams} streams (1 to {kernels.MAX_STREAMS})")
+        mult = layer.block.get("residual_mult")
+        self.mult = float(mult) if mult is not None else 1.0
+
+        def norm(spec):
+            made = norm_class(spec)(spec, hidden_size, dtype, device)
+            if not isinstance(made, RMSNorm):
+                raise ConfigError("hyper_prenorm: the norm in front of a sublayer is an rmsnorm")
+            return made
+        self.mixer_norm = norm(layer.norm)
+        self.mixer = mixer_class(layer.mixer)(layer.mixer, hidden_size, dtype, device)
+        self.feed_forward = self.ffn_norm = None
+        if layer.feed_forward is not None:
+            self.ffn_norm = norm(layer.ffn_norm or layer.norm)
+            self.feed_forward = feed_forward_class(layer.feed_forward)(layer.feed_forward, hidden_size, dtype, device)
+        self.mixer_hc = self.ffn_hc = None             # (in, mix, out) of each sublayer, 32-bit
+
+    @classmethod
+    def expected(cls, layer: LayerSpec, hidden_size: int) -> dict:
+        names, s = dict(layer.block["names"]), int(layer.block["streams"])
+
+        def connection(which):
+            return {names[which + "_in"]: Expected((s,), init="scale"), names[which + "_out"]: Expected((s,), init="scale"),
+                    names[which + "_mix"]: Expected((s, s), init="mixing")}
+        out = connection("mixer")
+        out.update(norm_class(layer.norm).expected(layer.norm, hidden_size, names["mixer_norm"]))
+        out.update(mixer_class(layer.mixer).expected(layer.mixer, hidden_size))
+        if layer.feed_forward is not None:
+            ffn_norm = layer.ffn_norm or layer.norm
+            out.update(connection("ffn"))
+            out.update(norm_class(ffn_norm).expected(ffn_norm, hidden_size, names["ffn_norm"]))
+            out.update(feed_forward_class(layer.feed_forward).expected(layer.feed_forward, hidden_size))
+        return out
+
+    def bind(self, tensors: dict) -> None:
+        n = self.names
+
+        def connection(which):
+            return tuple(tensors[n[f"{which}_{k}"]].to(torch.float32).contiguous() for k in ("in", "mix", "out"))
+        self.mixer_hc = connection("mixer")
+        self.mixer_norm.bind(tensors[n["mixer_norm"]])
+        self.mixer.bind(tensors)
+        if self.feed_forward is not None:
+            self.ffn_hc = connection("ffn")
+            self.ffn_norm.bind(tensors[n["ffn_norm"]])
+            self.feed_forward.bind(tensors)
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def parts(self) -> tuple:
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward) if p is not None)
+
+    def weights(self):
+        for part in self.parts():
+            yield from getattr(part, "weights", tuple)()
+        for hc in (self.mixer_hc, self.ffn_hc):
+            yield from hc or ()
+
+    def notices(self) -> list:
+        return [line for part in self.parts() for line in getattr(part, "notices", list)()]
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(part, "graph_safe", False) for part in self.parts())
+
+    def _reader(self) -> tuple:
+        """How the block's first sublayer reads the streams."""
+        return self.mixer_hc[0], self.mixer_norm.weight, self.mixer_norm.eps
+
+    def forward(self, x32: torch.Tensor, ctx, cache_view) -> None:
+        T, H, ws = x32.shape[0], self.hidden, ctx.workspace
+        X = x32.view(T, self.streams, H)
+        key = ("hyper_prenorm.normed", x32.data_ptr())
+        h = ctx.step_cache.pop(key, None)
+        if h is None:                              # the block in front left no normed rows
+            h = ws.buffer("hyper.normed", (T, H), self.dtype)
+            kernels.streams_read(X, *self._reader(), h)
+        follower = ctx.next_block if isinstance(ctx.next_block, HyperPreNormBlock) else None
+        after = follower._reader() if follower is not None else None
+        y = ws.buffer("hyper.result", (T, H), torch.float32)
+        if hasattr(self.mixer, "forward_store"):
+            self.mixer.forward_store(h, ctx, cache_view, y)
+        else:
+            y.zero_()
+            self.mixer.forward(h, ctx, cache_view, y)
+        # a sublayer has read h by the time the launch that overwrites it runs (stream order)
+        ff = self.feed_forward
+        _, mix, out = self.mixer_hc
+        if ff is not None:
+            kernels.streams_join(X, y, mix, out, self.mult, (self.ffn_hc[0], self.ffn_norm.weight, self.ffn_norm.eps), h)
+            if hasattr(ff, "forward_into"):
+                ff.forward_into(h, ctx, y)
+            else:
+                y.zero_()
+                ff.forward(h, ctx, y)
+            _, mix, out = self.ffn_hc
+        kernels.streams_join(X, y, mix, out, self.mult, after, h if after is not None else None)
+        if follower is not None:
+            ctx.step_cache[key] = h
+
+
 register_block("prenorm", PreNormBlock)
+register_block("hyper_prenorm", HyperPreNormBlock)
 register_block("sandwich_norm", SandwichNormBlock)
 register_block("parallel_scaled", ParallelScaledBlock)
 register_block("parallel_shift", ParallelShiftBlock)

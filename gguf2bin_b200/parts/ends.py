@@ -3,7 +3,9 @@ into logits.
 
 ``token_embedding``: row ``id`` of the table, widened to float32
 (src/l5_model.c:488-492 of AnonymoDGH/gguf2bin), times ``scale`` when the spec has one; with
-``positions`` (a name, and ``n_positions``) plus that table's row of the token's position.
+``positions`` (a name, and ``n_positions``) plus that table's row of the token's position; with
+``norm_name`` (and ``eps``) divided by its root mean square, times that weight.  A model of several
+streams asks for the row once per stream.
 ``lm_head``: logits = h . W^T in float32, W a matrix of its own or, when ``tied``, the
 embedding's table (src/l5_model.c:600-605: without an output tensor the reference
 multiplies by the token-embedding matrix).
@@ -34,6 +36,11 @@ class TokenEmbedding:
         self.table: Optional[torch.Tensor] = None      # [vocab, hidden]; a tied head multiplies by it
         self.positions_name = spec.get("positions")
         self.positions: Optional[torch.Tensor] = None  # [n_positions, hidden]
+        self.norm_name = spec.get("norm_name")
+        self.eps = float(spec.get("eps") or 0.0)
+        self.norm_w: Optional[torch.Tensor] = None
+        if self.norm_name and (self.positions_name or not self.eps > 0):
+            raise ConfigError("token_embedding: a norm needs a positive eps and goes with no position table")
         self._rows = None                              # what the kernel reads: the table in the positions' type
 
     @classmethod
@@ -41,22 +48,37 @@ class TokenEmbedding:
         out = {spec["name"]: Expected((int(vocab_size), int(hidden_size)))}
         if spec.get("positions"):
             out[spec["positions"]] = Expected((int(spec["n_positions"]), int(hidden_size)))
+        if spec.get("norm_name"):
+            out[spec["norm_name"]] = Expected((int(hidden_size),), init="scale")
         return out
 
     def bind(self, tensors: dict) -> None:
         self.table = self._rows = tensors[self.name].contiguous()
+        if self.norm_name:
+            self.norm_w = tensors[self.norm_name].to(torch.float32).contiguous()
         if self.positions_name:
             self.positions = tensors[self.positions_name].contiguous()
             if self.positions.dtype != self.table.dtype:          # one of them is kept in 32-bit: read both so
                 self.positions, self._rows = self.positions.float(), self.table.float()
 
     def weights(self):
-        return tuple(t for t in (self.table, self.positions, self._rows if self._rows is not self.table else None)
+        return tuple(t for t in (self.table, self.positions, self.norm_w, self._rows if self._rows is not self.table else None)
                      if t is not None)
 
+    @property
+    def writes_copies(self) -> bool:
+        """Whether ``forward`` takes an output with room for several copies of every row."""
+        return self.norm_w is not None
+
     def forward(self, tok_ids: torch.Tensor, out32: torch.Tensor, ctx, again=None) -> None:
-        """out32[t] = table[tok_ids[t]] * scale (+ positions[its position]) as float32; out32 is [T, hidden].
+        """out32[t] = table[tok_ids[t]] * scale (+ positions[its position]) as float32, normed if the spec says so;
+        out32 is [T, hidden], or [T, copies, hidden] for as many copies of every row (``writes_copies``).
         ``again``: a second buffer that gets the same rows."""
+        if self.writes_copies:
+            kernels.embed_norm_rows(self.table, tok_ids, self.norm_w, self.eps, out32, self.scale)
+            if again is not None:
+                again.copy_(out32)
+            return
         kernels.embed_rows(self._rows, tok_ids, out32, self.scale, self.positions, ctx.tok_pos, again)
 
 

@@ -111,8 +111,8 @@ class SwiGLU:
 class ActMLP:
     """``act_mlp``: down( act(up x) ), two matrices and an elementwise activation.  Activations:
     ``xielu``, a z^2 + z/2 above zero and (1/2 + b)(exp(z) - 1 - z) + z/2 below, with a and b the
-    softplus of two learned numbers (one tensor of two), computed in 32-bit; ``relu2``, max(z, 0)^2,
-    which has no tensor of its own.
+    softplus of two learned numbers (one tensor of two), computed in 32-bit; ``relu2``, max(z, 0)^2, and
+    ``gelu_tanh``, the tanh form of GELU, which have no tensor of their own.
 
     A block may hand it one more matrix that reads the same input (``take_along``): its rows go
     under the up matrix, one product computes both, and the step leaves that matrix's output in
@@ -122,8 +122,8 @@ class ActMLP:
     def __init__(self, spec: PartSpec, hidden_size: int, dtype: torch.dtype, device):
         self.inter, self.hidden = int(spec["intermediate_size"]), int(hidden_size)
         self.activation = spec.get("activation") or "xielu"
-        if self.activation not in ("xielu", "relu2"):
-            raise ConfigError(f"act_mlp: activation {self.activation!r} is not known (known: 'xielu', 'relu2')")
+        if self.activation not in ("xielu", "relu2", "gelu_tanh"):
+            raise ConfigError(f"act_mlp: activation {self.activation!r} is not known (known: 'xielu', 'relu2', 'gelu_tanh')")
         self.dtype = dtype
         self.names = dict(spec["names"])
         self.w_up = self.w_down = self.act = None
@@ -180,6 +180,8 @@ class ActMLP:
         mid = ws.buffer("mlp.mid", (T, self.inter), self.dtype)
         if self.activation == "relu2":
             kernels.relu2(up[:, :self.inter], mid)
+        elif self.activation == "gelu_tanh":
+            kernels.act_form(up[:, :self.inter], mid, kernels.GluForm.gelu_tanh())
         else:
             kernels.xielu(up[:, :self.inter], self.act, mid)
         kernels.linear(mid, self.w_down, out32, accumulate=accumulate)

@@ -1,4 +1,5 @@
-"""``latent_attention``: causal attention over cached low-rank latents, without positions.
+"""``latent_attention``: causal attention over cached low-rank latents, without positions or with rotated entries
+beside the latent.
 
 Per token the mixer projects its input u to queries q (``n_heads`` x ``qk_dim``) and to a latent
 c = rmsnorm(W_down u) * w of ``kv_rank`` numbers, which is ALL it caches.  Keys and values are
@@ -14,7 +15,12 @@ that the schedule entry's ``cache_of`` layer stored), ``scale``, ``q_rank`` (que
 of that many numbers, c_q = rmsnorm(W_dq u) * w_q, q = W_uq c_q; names ``q_down``, ``q_down_norm``, and ``q`` for W_uq),
 ``window`` (a token sees the last ``window`` positions, its own among them), ``pad_rank`` (bfloat16: latents of a rank
 below a size that the tensor-core attention kernels take lie in rows of that size, zero-filled, as do the
-up-projections' columns; scores and sums are what they were).
+up-projections' columns; scores and sums are what they were), ``rot_dim`` with ``position`` (each head of q has
+``rot_dim`` more entries behind its ``qk_dim`` ones, the down-projection as many more rows; those entries are turned by
+the token's position, are not normed, and the key's are one part for all heads: score = q . k + q_rot . k_rot.  A
+cached row is the latent with the rotated key behind it, a query in latent coordinates its rotated part behind it, so
+that attention over the rows is still one panel for keys and values; U_v has zeros in those columns),
+``out_gate`` = "sigmoid" (an element of the gate for every element of the concatenated heads instead of one per head).
 
 Scores, softmax and the latent's norm are 32-bit; products accumulate in 32-bit.
 
@@ -34,7 +40,7 @@ from .. import kernels
 from ..cache.storage import KVNeed, KVView
 from ..config.specs import ConfigError, PartSpec
 from ..weights.loader import Expected
-from .registry import register_mixer
+from .registry import position_class, register_mixer
 
 HEAD_PRODUCT_ROWS = 64       # steps of more rows multiply per head on the tensor cores (bfloat16)
 FOLD_UP_TO = 1.5             # rank / head size up to which an up-projection is always multiplied into its neighbour
@@ -64,27 +70,41 @@ class LatentAttention:
         self.eps = float(spec["eps"])
         self.shared_kv = bool(spec.get("shared_kv") or False)
         self.has_sink = bool(spec.get("sink") or False)
-        self.has_gate = bool(spec.get("out_gate") or False)
+        gate = spec.get("out_gate")
+        if gate not in (None, False, True, "sigmoid"):
+            raise ConfigError("latent_attention: out_gate is true (a number a head), 'sigmoid' (one an element) or absent")
+        self.has_gate, self.wide_gate = bool(gate), gate == "sigmoid"
+        self.rot = int(spec.get("rot_dim") or 0)
+        self.position = None
+        if self.rot:
+            pos = spec["position"]
+            self.position = position_class(pos)(pos, self.rot, device)
+            if self.rot < 0 or not hasattr(self.position, "table_rotation") or self.position.table_rotation()[0] is None \
+                    or self.position.table_rotation()[1] != self.rot:
+                raise ConfigError("latent_attention: rot_dim goes with a position part that turns all of it by a table")
         if min(self.nh, self.dk, self.dv, self.rank) <= 0:
             raise ConfigError("latent_attention: heads, sizes and rank must be positive")
-        if self.rank > 512:
-            raise ConfigError(f"latent_attention: kv_rank {self.rank} is more than the attention kernels' 512")
+        if self.rank + self.rot > 512:
+            raise ConfigError(f"latent_attention: kv_rank {self.rank} (+ {self.rot}) is more than the attention kernels' 512")
         self.q_rank = int(spec.get("q_rank") or 0)
         self.window = int(spec.get("window") or 0)
-        if spec.get("pad_rank") and not self.q_rank:
-            raise ConfigError("latent_attention: padded ranks go with a query latent")
+        if spec.get("pad_rank") and not self.q_rank and not self.rot:
+            raise ConfigError("latent_attention: padded ranks go with a query latent or rotated entries")
+        if self.rot and self.q_rank:
+            raise ConfigError("latent_attention: rotated entries do not go with a query latent")
         if self.q_rank < 0 or self.window < 0 or (self.q_rank and (self.shared_kv or self.has_gate)):
             raise ConfigError("latent_attention: q_rank and window are positive or absent; a query latent goes with "
                               "neither shared latents nor a gate")
         self.dtype, self.device = dtype, device
         self.names = dict(spec["names"])
-        self.own_rank = self.rank                 # what the down-projection makes; ``rank``: a row of the pages
+        self.own_rank = self.rank                 # the latent's entries; ``rank``: a row of the pages
+        self.rank += self.rot
         if spec.get("pad_rank") and dtype == torch.bfloat16:
             self.rank = kernels.padded_head_size(self.rank)
         # columns of the fused input product: queries (or their latent), then the latent (unless shared), then the gates
-        self.n_q = self.q_rank or self.nh * self.dk
-        self.n_c = 0 if self.shared_kv else self.own_rank
-        self.n_g = self.nh if self.has_gate else 0
+        self.n_q = self.q_rank or self.nh * (self.dk + self.rot)
+        self.n_c = 0 if self.shared_kv else self.own_rank + self.rot
+        self.n_g = 0 if not self.has_gate else self.nh * (self.dv if self.wide_gate else 1)
         self.w_in = self.w_o = self.w_uk = self.w_uv = self.c_norm = self.sink = self.w_uq = self.q_norm = None
         self.fold_k = self.fold_v = False
 
@@ -93,19 +113,19 @@ class LatentAttention:
     def expected(cls, spec: PartSpec, hidden_size: int) -> dict:
         n = dict(spec["names"])
         nh, dk, dv, r = spec["n_heads"], spec["qk_dim"], spec["v_dim"], spec["kv_rank"]
-        qr = spec.get("q_rank")
-        out = {n["q"]: Expected((nh * dk, qr or hidden_size)), n["up_k"]: Expected((nh * dk, r)),
+        qr, rot = spec.get("q_rank"), int(spec.get("rot_dim") or 0)
+        out = {n["q"]: Expected((nh * (dk + rot), qr or hidden_size)), n["up_k"]: Expected((nh * dk, r)),
                n["up_v"]: Expected((nh * dv, r)), n["o"]: Expected((hidden_size, nh * dv))}
         if qr:
             out[n["q_down"]] = Expected((qr, hidden_size))
             out[n["q_down_norm"]] = Expected((qr,), init="scale")
         if not (spec.get("shared_kv") or False):
-            out[n["down"]] = Expected((r, hidden_size))
+            out[n["down"]] = Expected((r + rot, hidden_size))
             out[n["down_norm"]] = Expected((r,), init="scale")
         if spec.get("sink"):
             out[n["sink"]] = Expected((nh,))
         if spec.get("out_gate"):
-            out[n["gate"]] = Expected((nh, hidden_size))
+            out[n["gate"]] = Expected((nh * dv if spec["out_gate"] == "sigmoid" else nh, hidden_size))
         return out
 
     def bind(self, tensors: dict) -> None:
@@ -117,16 +137,25 @@ class LatentAttention:
         q_in = self.q_rank or self.hidden          # what the queries are a product of
         folding = self.dtype == torch.bfloat16 and w_q.dtype == torch.bfloat16 and w_o.dtype == torch.bfloat16
         self.fold_k = folding and folds(self.rank, self.dk, self.nh, q_in)
-        self.fold_v = folding and folds(self.rank, self.dv, self.nh, self.hidden)
+        # (a gate per element does not commute with U_v)
+        self.fold_v = folding and not self.wide_gate and folds(self.rank, self.dv, self.nh, self.hidden)
+        w_rot = None
+        if self.rot:                               # rows head by head [qk_dim, rot_dim]: the two kinds apart
+            w_q = w_q.view(self.nh, self.dk + self.rot, q_in)
+            w_q, w_rot = w_q[:, :self.dk].reshape(self.nh * self.dk, q_in), w_q[:, self.dk:]
         if self.fold_k:
             # W_q'[h] = U_k[h]^T W_q[h]: [rank, qk_dim] x [qk_dim, width] per head; the queries then
             # come out of the input product in latent coordinates, `rank` numbers per head
             uk = up_k.double().view(self.nh, self.dk, self.rank)
             wq = w_q.double().view(self.nh, self.dk, q_in)
-            w_q = torch.einsum("hdr,hdw->hrw", uk, wq).reshape(self.nh * self.rank, q_in) \
-                .to(torch.bfloat16).contiguous()
+            w_q = torch.einsum("hdr,hdw->hrw", uk, wq)
+            if self.rot:                           # a head's rotated entries lie behind its latent coordinates
+                w_q[:, self.own_rank:self.own_rank + self.rot] = w_rot.double()
+            w_q = w_q.reshape(self.nh * self.rank, q_in).to(torch.bfloat16).contiguous()
             if not self.q_rank:
                 self.n_q = self.nh * self.rank
+        elif self.rot:                             # all heads' unrotated rows, then all heads' rotated ones
+            w_q = torch.cat([w_q, w_rot.reshape(self.nh * self.rot, q_in)], dim=0)
         parts = [w_q]
         if self.q_rank:
             self.w_uq = w_q.contiguous()
@@ -231,6 +260,9 @@ class LatentAttention:
             kernels.latent_pair(d, self.rank, self.c_norm, view.pages, q, self.q_norm, cq, self.eps, ctx)
             q = ws.buffer("latent.uq", (T, self.w_uq.shape[0]), self.dtype)
             kernels.linear(cq, self.w_uq, q)
+        elif self.rot:
+            if ring is not None:
+                kernels.latent_keep(None, None, 0.0, None, rows, ring, taps, ctx)
         elif d is not None or ring is not None:
             kernels.latent_keep(d, self.c_norm, self.eps, view.pages if d is not None else None,
                                 rows, ring, taps, ctx)
@@ -238,7 +270,13 @@ class LatentAttention:
             qa = q                          # columns of the product's output: the attention reads them in place
         else:
             qa = ws.buffer("latent.q", (T, self.nh * self.rank), self.dtype)
-            self._per_head(q, self.w_uk, qa, False, None)
+            self._per_head(q[:, :self.nh * self.dk], self.w_uk, qa, False, None)
+        if self.rot:
+            inv_freq, _, interleaved = self.position.table_rotation()
+            at = self.own_rank                     # where a head's rotated entries begin in latent coordinates
+            src, step = (qa[:, at:], self.rank) if self.fold_k else (q[:, self.nh * self.dk:], self.rot)
+            kernels.latent_rope(d, self.own_rank, self.rank, self.c_norm, self.eps, view.pages, src, step, qa[:, at:], self.rank,
+                                self.nh, self.rot, ctx.rope_table(inv_freq), interleaved, ctx)
         mix = ws.buffer("latent.mix", (T, self.nh * self.rank), self.dtype)
         # with U_v folded into the output matrix the heads' gate is the attention's last step
         kernels.attention(qa, mix, view.pages, ctx, self.nh, 1, self.rank, view.page_size, self.window, self.scale,
@@ -247,7 +285,11 @@ class LatentAttention:
             o = mix
         else:
             o = ws.buffer("latent.o", (T, self.nh * self.dv), self.dtype)
-            self._per_head(mix, self.w_uv, o, True, gate)
+            self._per_head(mix, self.w_uv, o, True, None if self.wide_gate else gate)
+            if self.wide_gate:
+                gated = ws.buffer("latent.gated", (T, self.nh * self.dv), self.dtype)
+                kernels.gate_mul(o, self.dv, gate, self.nh, self.dv, 1.0, gated)
+                o = gated
         kernels.linear(o, self.w_o, out32, accumulate=accumulate)
 
 

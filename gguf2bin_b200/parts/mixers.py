@@ -39,6 +39,8 @@ true positions;
 inside the root, no weight);
 ``out_gate`` = "head_sigmoid": every head's output times sigmoid(W_g h)_h, one number per head (name ``gate``,
 [heads, hidden]);
+``pad_heads`` (bfloat16): pages hold heads at the next size that the tensor-core attention kernels take, zero-filled
+(scores and sums are what they were);
 ``one_pass_prologue``: norm, rotation and page writes in the one kernel below even where the narrower
 kernels would do (a rotation of neighbouring pairs then costs one launch instead of four).
 The first, second, third, sixth, the value norm, the unit norm and the gates take the prologue kernel that
@@ -136,6 +138,11 @@ class GQAAttention:
             if not hasattr(self.position, "table_rotation"):
                 raise ConfigError("gqa_attention: this position part offers no table rotation")
         self.cache_hd = max(self.hd, self.vd)
+        if spec.get("pad_heads"):
+            if not self.wide:
+                raise ConfigError("gqa_attention: padded heads need the wide prologue (one_pass_prologue)")
+            if dtype == torch.bfloat16:
+                self.cache_hd = kernels.padded_head_size(self.cache_hd)
 
     # ---- weights -------------------------------------------------------------
     @classmethod
@@ -256,7 +263,7 @@ class GQAAttention:
                                      self.k_norm_w, self.qk_eps, rope, rot, interleaved, ctx,
                                      view.pages if nkv_own else None, view.page_size, q, v_norm_eps=self.v_norm_eps,
                                      norm_per_head=self.has_qk_norm and self.norm_span == "head",
-                                     unit_eps=self.unit_eps, n_v_heads=nv_own)
+                                     unit_eps=self.unit_eps, n_v_heads=nv_own, store_dim=hd)
         if self.pool:
             kernels.pool_update(view.pages, pooled, ctx, self.nkv, hd, view.page_size, self.pool)
         gate_at = self.nh * self.hd + nkv_own * self.hd + nv_own * self.vd       # the gate's first column

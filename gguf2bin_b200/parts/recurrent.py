@@ -42,6 +42,13 @@ v = W_v h; a = sigmoid(z)^(1/tau) with z = W_a2 (W_a1 h) + b, one number per hea
 rank of the decay, come from the checkpoint); per head S_t = diag(a_t) S_{t-1} + k_t v_t^T, o_t = S_t^T q_t; each head's
 o divided by its root mean square, times a weight over v_dim shared by the heads, times silu(W_g h); output product.
 
+``wkv``: time mixing over the token before, with a decayed matrix state.  r, k, v, the gate and the decay read mixes of
+their own, h + (h' - h) mu_c, h' the row of the token before (zeros in front of the first); r = W_r(mix_r) and so on
+(heads x dim); a = exp(-exp(W_2 tanh(W_1 mix_w) + w0)) per head and key channel (W_1's rows come from the checkpoint);
+per head o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t, then S_t = diag(a_t) S_{t-1} + k_t v_t^T; each head's o divided by its
+root mean square, times a weight over all heads, times silu(W_g mix_g); output product.  The last row h of a
+sequence is part of its state, in the compute type.
+
 ``parallel``: several mixers that read the same input; the result is the sum of theirs, each times
 its ``out_scale``.  A branch is any registered mixer that takes ``out_scale``.
 
@@ -548,6 +555,87 @@ class GatedLinearAttention:
         kernels.linear(og, self.w_o, residual32, accumulate=accumulate)
 
 
+class WKVMixer:
+    graph_safe = True
+    LOW_RANK = 16             # rank of the decay's matrices where random weights are made (a checkpoint brings its own)
+    MIXES = ("r", "k", "v", "gate", "w")           # the order of the mixes, of W_in's row blocks and of the mixed rows
+
+    def __init__(self, spec: PartSpec, hidden_size: int, dtype: torch.dtype, device):
+        self.H, self.D = int(spec["n_heads"]), int(spec["head_dim"])
+        self.hidden, self.dtype, self.device = int(hidden_size), dtype, device
+        if min(self.H, self.D) <= 0 or self.D > 512:
+            raise ConfigError("wkv: heads and head_dim (at most 512) must be positive")
+        self.eps = float(spec["eps"])
+        self.names = dict(spec["names"])
+        self.mu = self.w_in = self.w_low1 = self.w_low2 = self.w0 = self.bonus = self.norm_w = self.w_o = None
+
+    @classmethod
+    def expected(cls, spec: PartSpec, hidden_size: int) -> dict:
+        n = dict(spec["names"])
+        H, D = int(spec["n_heads"]), int(spec["head_dim"])
+        rank = FreeSize(cls.LOW_RANK)
+        out = {n["mu_" + c]: Expected((hidden_size,)) for c in cls.MIXES}
+        out.update({n[c]: Expected((H * D, hidden_size)) for c in ("r", "k", "v", "gate")})
+        out.update({n["w1"]: Expected((rank, hidden_size)), n["w2"]: Expected((H * D, rank)), n["w0"]: Expected((H * D,)),
+                    n["bonus"]: Expected((H, D)), n["norm"]: Expected((H * D,), init="scale"),
+                    n["o"]: Expected((hidden_size, H * D))})
+        return out
+
+    def bind(self, tensors: dict) -> None:
+        n, f32 = self.names, torch.float32
+        w1, w2 = tensors[n["w1"]], tensors[n["w2"]]
+        rank = w1.shape[0]
+        if w2.shape[1] != rank:
+            raise WeightsError(f"{n['w1']} has {rank} rows, {n['w2']} {w2.shape[1]} columns: they must be equal")
+        if rank > 1024:
+            raise WeightsError(f"{n['w1']}: a decay rank of {rank} (at most 1024)")
+        self.mu = torch.stack([tensors[n["mu_" + c]].to(f32) for c in self.MIXES]).contiguous()
+        parts = [tensors[n[c]] for c in ("r", "k", "v", "gate")]
+        common = _common_dtype(parts)
+        self.w_in = torch.stack([p.to(common) for p in parts]).contiguous()            # [4, H * D, hidden]
+        self.w_low1 = _padded_rows([w1])                                               # a rank that is a multiple of eight
+        self.w_low2 = torch.nn.functional.pad(w2, (0, self.w_low1.shape[0] - rank)).to(self.dtype).contiguous()
+        self.w0 = tensors[n["w0"]].to(f32).contiguous()
+        self.bonus = tensors[n["bonus"]].to(f32).contiguous()
+        self.norm_w = tensors[n["norm"]].to(f32).contiguous()
+        self.w_o = tensors[n["o"]].contiguous()
+
+    def weights(self):
+        return (self.mu, self.w_in, self.w_low1, self.w_low2, self.w0, self.bonus, self.norm_w, self.w_o)
+
+    def notices(self) -> list:
+        return (kernels.product_notices("time mixing input", self.w_in[0], self.dtype)
+                + kernels.product_notices("time mixing output", self.w_o, self.dtype))
+
+    def cache_need(self):
+        return {"state": StateNeed((self.H, self.D, self.D), torch.float32), "shift": StateNeed((self.hidden,), self.dtype)}
+
+    def forward(self, h: torch.Tensor, ctx, view, residual32: torch.Tensor) -> None:
+        self._run(h, ctx, view, residual32, True)
+
+    def forward_store(self, h: torch.Tensor, ctx, view, out32: torch.Tensor) -> None:
+        """Stores the result instead of adding it."""
+        self._run(h, ctx, view, out32, False)
+
+    def _run(self, h, ctx, view, residual32, accumulate: bool) -> None:
+        T, ws, n = h.shape[0], ctx.workspace, self.H * self.D
+        mixed = ws.buffer("wkv.mixed", (len(self.MIXES), T, self.hidden), self.dtype)
+        kernels.shift_mix(h, self.mu, view["shift"].states, ctx, mixed)
+        proj = ws.buffer("wkv.in", (T, 4 * n), self.dtype)
+        for i in range(4):
+            kernels.linear(mixed[i], self.w_in[i], proj[:, i * n:(i + 1) * n])
+        low = ws.buffer("wkv.low", (T, self.w_low1.shape[0]), torch.float32)           # 32-bit: it enters the decay
+        kernels.linear(mixed[4], self.w_low1, low)
+        o32 = ws.buffer("wkv.o", (T, n), torch.float32)
+        kernels.channel_scan(proj[:, :n], proj[:, n:2 * n], proj[:, 2 * n:3 * n], low, self.w_low2, self.w0,
+                             view["state"].states, ctx, o32, self.H, self.D, self.D, 1.0, decay="double_exp", low_tanh=True,
+                             bonus=self.bonus)
+        og = ws.buffer("wkv.gated", (T, n), self.dtype)
+        kernels.state_readout(o32, self.H, self.D, og, gate=proj[:, 3 * n:], gate_act="silu", gate_first=False, group=self.D,
+                              eps=self.eps, w=self.norm_w)
+        kernels.linear(og, self.w_o, residual32, accumulate=accumulate)
+
+
 class ParallelMixer:
     """Branches side by side on one input; what each stores is kept under ``<branch>.<name>``."""
 
@@ -613,6 +701,7 @@ class ParallelMixer:
 register_mixer("retention", RetentionMixer)
 register_mixer("gated_delta", GatedDeltaMixer)
 register_mixer("gla", GatedLinearAttention)
+register_mixer("wkv", WKVMixer)
 register_mixer("parallel", ParallelMixer)
 register_mixer("ssd", SSDMixer)
 register_mixer("mlstm", MLSTMMixer)

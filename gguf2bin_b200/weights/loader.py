@@ -30,7 +30,7 @@ class FreeSize(int):
 @dataclass(frozen=True)
 class Expected:
     """A tensor the model needs.  ``init`` tells the random-weights writer how to fill
-    it: "matrix" (N(0, std)) or "scale" (1 + N(0, scale_std)).  ``optional`` tensors may
+    it: "matrix" (N(0, std)), "scale" (1 + N(0, scale_std)) or "mixing" (the identity + N(0, scale_std)).  ``optional`` tensors may
     be absent (an lm_head matrix beside tied embeddings)."""
     shape: tuple
     init: str = "matrix"

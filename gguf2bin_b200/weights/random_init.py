@@ -98,14 +98,20 @@ def normal_values(n: int, seed: int, tensor_index: int, first: int = 0) -> np.nd
     return z.reshape(-1)[:n]
 
 
+INIT_KINDS = ("matrix", "scale", "mixing")
+
+
 def random_tensor(e: Expected, seed: int, index: int, dtype: torch.dtype,
                   std: float, scale_std: float) -> torch.Tensor:
     """The tensor at position ``index`` of a model's list, made on the CPU."""
     n = 1
     for d in e.shape:
         n *= int(d)
-    if e.init not in ("matrix", "scale"):
+    if e.init not in INIT_KINDS:
         raise ValueError(f"unknown init kind {e.init!r}")
+    if e.init == "mixing":
+        z = torch.from_numpy(_f(scale_std) * normal_values(n, seed, index)).view(tuple(e.shape))
+        return (z + torch.eye(*e.shape)).to(dtype)
     out = torch.empty(n, dtype=dtype)
     for first in range(0, n, _CHUNK):
         z = normal_values(min(_CHUNK, n - first), seed, index, first)
@@ -118,8 +124,13 @@ def fill_random_on_device(out: torch.Tensor, e: Expected, seed: int, index: int,
                           scale_std: float) -> None:
     """The same tensor, made in place in device memory by the CUDA kernel."""
     from .. import kernels
-    if e.init not in ("matrix", "scale"):
+    if e.init not in INIT_KINDS:
         raise ValueError(f"unknown init kind {e.init!r}")
+    if e.init == "mixing":
+        z = torch.empty(tuple(e.shape), dtype=torch.float32, device=out.device)
+        kernels.philox_normal(z, seed, index, False, scale_std)
+        out.copy_(z + torch.eye(*e.shape, device=out.device))
+        return
     kernels.philox_normal(out, seed, index, e.init == "scale", scale_std if e.init == "scale" else std)
 
 
