@@ -2,7 +2,7 @@
 """Decode and prefill throughput of gguf2bin_b200 on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-                    [--workload decode|ragged8|b64|senotar|levolix|sominex|mopitar|kubedra] [--batch B] [--layers L] [--context C]
+                    [--workload decode|ragged8|b64|senotar|levolix|sominex|mopitar|kubedra|nekotar] [--batch B] [--layers L] [--context C]
                     [--no-points] [--sizes 0.6b|8b|14b]
 
 The default run has the layer sizes of Qwen3-0.6B (28 layers, width 1024, 16/8 heads of
@@ -57,6 +57,11 @@ vocabulary and, within a few per cent, active parameters.
 queries from a latent, gated linear attention with a decay per key channel, capped routed experts with a shared
 one) beside Levolix, the library's closest design (a matrix state per head, normed sublayer outputs, routed
 experts, a tied head), in the same way.
+
+``--workload nekotar`` sets Nekotar (two residual streams with mixing coefficients, latent attention with rotated
+entries, time mixing with a decayed matrix state, windowed attention with kept first tokens, a two-matrix GELU
+feed-forward) beside Kubedra, the library's closest design (latent attention, a matrix state with a decay per key
+channel), in the same way.
 
 Peaks come from MEASURED_PEAKS.json beside this file when present, else from the
 fallback figures 6.65 TB/s and 1.59 PFLOP/s.  Inputs are synthetic.  Between timed steps
@@ -805,6 +810,109 @@ def kubedra_comparison(a, pk) -> int:
     return 0
 
 
+# ---- Nekotar beside Kubedra at equal sizes ----------------------------------------------------------
+def nekotar_config(width, layers, vocab) -> dict:
+    """Latent attention, time mixing and windowed attention in turn; every second latent layer reads the latents of the
+    one before it."""
+    H, out, lender = width // 128, [], None
+    for i in range(layers):
+        if i % 3 == 0:
+            kind = "latent_attention"
+            mixer = dict(heads=H, dim=128, vdim=128, kv_rank=96, rot_dim=32, scale=160 ** -0.5, rot=dict(base=1e4, dims=32))
+            if lender is None:
+                lender = i
+            else:
+                mixer["kv_from"], lender = lender, None
+        elif i % 3 == 1:
+            kind, mixer = "wkv", dict(heads=width // 64, dim=64)
+        else:
+            kind = "attention"
+            mixer = dict(heads=H, kv_heads=max(H // 4, 1), dim=128, vdim=128, scale=128 ** -0.5, rot=dict(base=5e5, dims=128),
+                         mask=dict(size=512, keep_first=8))
+        out.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=9 * width // 2)))
+    return dict(architecture="Nekotar", width=width, vocab=vocab, streams=2, residual_mult=0.5, norm=dict(eps=1e-6), layers=out)
+
+
+def nekotar_bytes_and_flops(cfg: dict, T: int) -> dict:
+    """As ``mopitar_bytes_and_flops``: matrices once, states read and written, latents (once for keys and values) and
+    visible keys and values once a token."""
+    W, V = cfg["width"], cfg["vocab"]
+    params = state_bytes = 0
+    seen, pair_flops = [], 0.0     # (bytes per visible token, window, kept) of every layer that reads keys
+    for layer in cfg["layers"]:
+        m, H, D = layer["mixer"], layer["mixer"]["heads"], layer["mixer"]["dim"]
+        if layer["type"] == "wkv":
+            n = H * D
+            params += 5 * W * n + 16 * (W + n)
+            state_bytes += 2 * 4 * H * D * D
+        elif layer["type"] == "latent_attention":
+            r, rot, Vd = m["kv_rank"], m["rot_dim"], m["vdim"]
+            params += W * (H * (D + rot) + 2 * H * Vd) + H * (D + Vd) * r + (0 if "kv_from" in m else W * (r + rot))
+            seen.append((2 * (r + rot), 0, 0))
+            pair_flops += 2.0 * H * (2 * r + rot) * T * (T + 1) / 2
+        else:
+            G, Vd, w, k = m["kv_heads"], m["vdim"], m["mask"]["size"], m["mask"]["keep_first"]
+            params += W * (H * D + G * D + G * Vd + 2 * H * Vd)
+            seen.append((2 * G * (D + Vd), w, k))
+            pair_flops += 2.0 * H * (D + Vd) * sum(min(t + 1, w) + min(k, max(0, t + 1 - w)) for t in range(T))
+        params += 2 * W * layer["mlp"]["ff"]
+
+    def kv_bytes(ctx: float) -> float:
+        return sum(b * (ctx if not w else min(ctx, w) + min(k, max(0.0, ctx - w))) for b, w, k in seen)
+    return dict(layer_params=params, weight_bytes=2 * (params + V * W), state_bytes=state_bytes, kv_bytes=kv_bytes,
+                pair_flops=pair_flops)
+
+
+def nekotar_comparison(a, pk) -> int:
+    import torch
+    from gguf2bin_b200.api import LLM
+    layers, vocab, batch, T = a.layers or 6, 151936, a.batch or 8, a.prefill_tokens
+    steps, warmup = a.steps or 128, max(a.warmup, 8)
+    max_tokens = batch * (T + warmup + steps + 128)
+    rows = {}
+    clocks = ClockSampler()
+    clocks.start()
+    for name, (width, *_rest) in LEVOLIX_SIZES.items():
+        if a.sizes_only and name not in a.sizes_only.split(","):
+            continue
+        row = {}
+        for arch in ("nekotar", "kubedra"):
+            if arch == "nekotar":
+                cfg = nekotar_config(width, layers, vocab)
+                sizes = nekotar_bytes_and_flops(cfg, T)
+                pair_flops, kv_bytes = sizes["pair_flops"], sizes["kv_bytes"]
+            else:
+                cfg = kubedra_config(width, layers, vocab, T + warmup + steps + 128)
+                sizes = kubedra_bytes_and_flops(cfg)
+                seen = cfg["layers"][0]["mixer"]["mask"]["size"]
+                pair_flops = sizes["attn_flops_per_pair"] * sum(min(t + 1, seen) for t in range(T))
+                kv_bytes = lambda ctx: min(ctx, seen) * sizes["kv_bytes_per_token"]          # noqa: E731
+            flops = 2.0 * T * sizes["layer_params"] + pair_flops + 2.0 * vocab * width
+            llm = LLM.random(cfg, seed=0, dtype="bfloat16", max_tokens=max_tokens, max_seqs=batch + 1)
+            first, ms, plain = timed_prompt_step(llm, random_prompts(1, T, vocab, 1), repeats=3)
+            sec, per_step, mean_ctx = decode_device_timed(llm, random_prompts(batch, T, vocab, 100), steps, warmup,
+                                                          vocab, whole_batch_prefill=False)
+            step_bytes = sizes["weight_bytes"] + batch * (sizes["state_bytes"] + kv_bytes(mean_ctx))
+            gbs = step_bytes / (sec / steps) / 1e9
+            row[arch] = dict(
+                active_parameters_per_layer_m=round(sizes["layer_params"] / layers / 1e6, 1),
+                prefill_tokens_per_s=round(T / (ms / 1e3)), prefill_ms=round(ms, 3), prefill_plain_ms=round(plain, 3),
+                prefill_frac_of_tensor_peak=round(flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12), 3),
+                decode_tokens_per_s=round(batch * steps / sec), decode_ms_per_step=round(sec / steps * 1e3, 4),
+                decode_launches_per_step=per_step, decode_step_mb=round(step_bytes / 1e6, 1), decode_gbs=round(gbs),
+                decode_frac_of_copy_bandwidth=round(gbs / pk["hbm_gbs"], 3))
+            del llm
+            torch.cuda.empty_cache()
+        rows[name] = row
+    print(json.dumps({"metric": "prefill and decode tokens/s of Nekotar beside Kubedra at equal sizes (random weights)",
+                      "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic", "impl": "ours",
+                      "config": {"layers": layers, "vocab": vocab, "prompt_tokens": T, "decode_batch": batch,
+                                 "decode_context_from": T + warmup, "decode_steps": steps, "peaks": pk["source"],
+                                 "l2": "inputs larger than L2 (weights, states and cache read every step)"},
+                      "sizes": rows, "clocks": clocks.stop()}))
+    return 0
+
+
 WORKLOADS = {
     # name: (sizes, batch, what it is)
     "decode": ("0.6b", 8, "every sequence prefilled to half the context, then decoded"),
@@ -814,6 +922,7 @@ WORKLOADS = {
     "levolix": (None, 8, "Levolix beside Qwen3 at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
     "sominex": (None, 8, "Sominex beside Qwen3 at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
     "kubedra": (None, 8, "Kubedra beside Levolix at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
+    "nekotar": (None, 8, "Nekotar beside Kubedra at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
     "mopitar": (None, 8, "Mopitar beside Sominex at equal sizes: a 2,048-token prompt step and batch-8 decode steps each"),
 }
 
@@ -835,7 +944,7 @@ def main() -> int:
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                     help="length of the prompt of the prefill figure (decode workload; default 2048)")
     ap.add_argument("--sizes-only", default=None,
-                    help="senotar, levolix, sominex, mopitar and kubedra workloads: a comma-separated subset of " + ",".join(EQUAL_SIZES))
+                    help="senotar, levolix, sominex, mopitar, kubedra and nekotar workloads: a comma-separated subset of " + ",".join(EQUAL_SIZES))
     a = ap.parse_args()
 
     if a.impl == "reference":
@@ -859,6 +968,8 @@ def main() -> int:
         return mopitar_comparison(a, peaks())
     if a.workload == "kubedra":
         return kubedra_comparison(a, peaks())
+    if a.workload == "nekotar":
+        return nekotar_comparison(a, peaks())
 
     import numpy as np
     import torch
