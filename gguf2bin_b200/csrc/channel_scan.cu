@@ -202,14 +202,14 @@ channel_prep_kernel(const ChannelIn a, int n_tokens, float *__restrict__ qf, flo
   extern __shared__ __align__(16) float cs_sm[];      // low vectors of the block's tokens [CP_TOKENS, R]
   const int D = a.D, R = a.R, h = blockIdx.y;
   const int t0 = blockIdx.x * CP_TOKENS;
-  for (int i = threadIdx.x; i < CP_TOKENS * R; i += CP_THREADS)       // tokens behind the last one repeat it
+  for (int i = threadIdx.x; i < CP_TOKENS * R; i += blockDim.x)       // tokens behind the last one repeat it
     cs_sm[i] = low_entry<T>(a, min(t0 + i / R, n_tokens - 1), i % R);
   __syncthreads();
   const size_t row = (size_t)a.H * D;
   float sum[CP_TOKENS];
 #pragma unroll
   for (int i = 0; i < CP_TOKENS; ++i) sum[i] = 0.f;
-  for (int d = threadIdx.x; d < D; d += CP_THREADS) {
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
     const size_t ch = (size_t)h * D + d;
     const float u = a.bonus ? a.bonus[ch] : 0.f;
     float z[CP_TOKENS], qv[CP_TOKENS], kv[CP_TOKENS];
@@ -236,11 +236,17 @@ channel_prep_kernel(const ChannelIn a, int n_tokens, float *__restrict__ qf, flo
     }
   }
   if (!a.bonus) return;
-  __shared__ float scratch[32];
+  __shared__ float part[CP_THREADS / 32][CP_TOKENS];
 #pragma unroll
   for (int i = 0; i < CP_TOKENS; ++i) {
-    const float s = block_sum(sum[i], scratch);
-    if (threadIdx.x == 0 && t0 + i < n_tokens) own[(size_t)(t0 + i) * a.H + h] = s;
+    const float s = warp_sum(sum[i]);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5][i] = s;
+  }
+  __syncthreads();
+  if (threadIdx.x < CP_TOKENS && t0 + threadIdx.x < n_tokens) {
+    float s = 0.f;
+    for (int w = 0; w < (int)blockDim.x >> 5; ++w) s += part[w][threadIdx.x];
+    own[(size_t)(t0 + threadIdx.x) * a.H + h] = s;
   }
 }
 
@@ -535,14 +541,15 @@ extern "C" int g2b_channel_scan(int dtype, const void *q, int q_stride, const vo
       (bonus && !own))
     G2B_REFUSE("channel_scan: a prompt step needs its tables and scratch buffers");
   const dim3 prep_grid((n_tokens + CP_TOKENS - 1) / CP_TOKENS, H);
+  const dim3 prep_block(D > 64 ? CP_THREADS : (D > 32 ? 64 : 32));       // at most a round of idle threads
   const size_t prep_smem = (size_t)CP_TOKENS * R * sizeof(float);
   if (dtype == G2B_F32) {
     if (prep_smem > 48 * 1024) cudaFuncSetAttribute(channel_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem);
-    g2b_launch(channel_prep_kernel<float>, prep_grid, dim3(CP_THREADS), prep_smem, stream, in, n_tokens, qf, kf, af,
+    g2b_launch(channel_prep_kernel<float>, prep_grid, prep_block, prep_smem, stream, in, n_tokens, qf, kf, af,
                own);
   } else {
     if (prep_smem > 48 * 1024) cudaFuncSetAttribute(channel_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem);
-    g2b_launch(channel_prep_kernel<bf16>, prep_grid, dim3(CP_THREADS), prep_smem, stream, in, n_tokens, qf, kf, af,
+    g2b_launch(channel_prep_kernel<bf16>, prep_grid, prep_block, prep_smem, stream, in, n_tokens, qf, kf, af,
                own);
   }
   SegArgs a;

@@ -60,7 +60,7 @@ extern "C" int g2b_embed_rows(const void *table, int table_dtype, const int *ids
 }
 
 // The same rows divided by their root mean square, times w, written `copies` times side by side: out [T, copies, H].
-template <typename TW>
+template <typename TW, bool VEC>
 __global__ void __launch_bounds__(256)
 embed_norm_rows_kernel(const TW *__restrict__ table, const int *__restrict__ ids, const float *__restrict__ w, float eps,
                        float *__restrict__ out, int copies, int H, int V, float scale) {
@@ -78,9 +78,19 @@ embed_norm_rows_kernel(const TW *__restrict__ table, const int *__restrict__ ids
     ss = fmaf(v, v, ss);
   }
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
-  for (int j = threadIdx.x; j < H; j += blockDim.x) {
-    const float v = ((ok ? to_f32(row[j]) * scale : 0.f) * inv) * (w ? w[j] : 1.f);
-    for (int c = 0; c < copies; ++c) out[((size_t)t * copies + c) * H + j] = v;
+  if (VEC) {                                         // H a multiple of four: 16-byte stores
+    for (int j = 4 * threadIdx.x; j < H; j += 4 * blockDim.x) {
+      float v[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] = ((ok ? to_f32(row[j + i]) * scale : 0.f) * inv) * (w ? w[j + i] : 1.f);
+      for (int c = 0; c < copies; ++c)
+        *reinterpret_cast<float4 *>(out + ((size_t)t * copies + c) * H + j) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+  } else {
+    for (int j = threadIdx.x; j < H; j += blockDim.x) {
+      const float v = ((ok ? to_f32(row[j]) * scale : 0.f) * inv) * (w ? w[j] : 1.f);
+      for (int c = 0; c < copies; ++c) out[((size_t)t * copies + c) * H + j] = v;
+    }
   }
 }
 
@@ -88,12 +98,13 @@ extern "C" int g2b_embed_norm_rows(const void *table, int table_dtype, const int
                                    int copies, int T, int H, int V, float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || V <= 0 || copies <= 0) G2B_REFUSE("embed_norm_rows: bad sizes H=%d V=%d copies=%d", H, V, copies);
+  const bool vec = H % 4 == 0 && !((uintptr_t)out & 15);
   const int threads = H >= 256 ? 256 : 64;
   if (table_dtype == G2B_F32)
-    g2b_launch(embed_norm_rows_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float *)table, ids, w, eps, out, copies,
+    g2b_launch(vec ? embed_norm_rows_kernel<float, true> : embed_norm_rows_kernel<float, false>, dim3(T), dim3(threads), 0, stream, (const float *)table, ids, w, eps, out, copies,
                H, V, scale);
   else if (table_dtype == G2B_BF16)
-    g2b_launch(embed_norm_rows_kernel<bf16>, dim3(T), dim3(threads), 0, stream, (const bf16 *)table, ids, w, eps, out, copies,
+    g2b_launch(vec ? embed_norm_rows_kernel<bf16, true> : embed_norm_rows_kernel<bf16, false>, dim3(T), dim3(threads), 0, stream, (const bf16 *)table, ids, w, eps, out, copies,
                H, V, scale);
   else
     G2B_REFUSE("embed_norm_rows: unknown table dtype %d", table_dtype);
@@ -1065,7 +1076,7 @@ act_form_kernel(const T *__restrict__ z, int z_stride, T *__restrict__ out, long
   pdl_wait();
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
   if (i >= total) return;
-  out[i] = from_f32<T>(glu_value(to_f32(z[(size_t)(i / F) * z_stride + (i % F)]), 1.f, form));
+  out[i] = from_f32<T>(act_value(to_f32(z[(size_t)(i / F) * z_stride + (i % F)]), form));
 }
 
 extern "C" int g2b_act_form(const void *z, int z_stride, int dtype, int T_tokens, int F, void *out, float c1, float c3,

@@ -39,12 +39,25 @@ constexpr int XROW = KB + XPAD;
 constexpr int DEPTH = 4;                // K blocks of W in flight per thread
 
 // As in gemm_tc.cu: a build with -DG2B_GLU holds the gated epilogue alone, in its general form.
+// A build with -DG2B_ACT holds the bfloat16 store alone, behind the form's activation.
 #ifdef G2B_GLU
 __device__ __forceinline__ float glu_out(float gate, float up, const GluForm &f) { return glu_value(gate, up, f); }
-#define G2B_IF_UNGATED(...)
+#define G2B_IF_BF16(...)
 #else
 __device__ __forceinline__ float glu_out(float gate, float up, const GluForm &) { return (gate / (1.f + expf(-gate))) * up; }
-#define G2B_IF_UNGATED(...) __VA_ARGS__
+#define G2B_IF_BF16(...) __VA_ARGS__
+#endif
+#ifdef G2B_ACT
+__device__ __forceinline__ float bf16_out(float v, const GluForm &f) { return act_value(v, f); }
+#define G2B_IF_GATED(...)
+#else
+__device__ __forceinline__ float bf16_out(float v, const GluForm &) { return v; }
+#define G2B_IF_GATED(...) __VA_ARGS__
+#endif
+#if defined(G2B_GLU) || defined(G2B_ACT)
+#define G2B_IF_FLOAT(...)
+#else
+#define G2B_IF_FLOAT(...) __VA_ARGS__
 #endif
 enum { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ACCUM_F32 = 2, EPI_SWIGLU_BF16 = 3 };
 
@@ -164,7 +177,7 @@ gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *
       const int n = n0 + r;
       if (m < M && n < N) {
         const size_t o = (size_t)m * ldc + n;
-        if (EPI == EPI_STORE_BF16) ((bf16 *)Cv)[o] = __float2bfloat16_rn(v);
+        if (EPI == EPI_STORE_BF16) ((bf16 *)Cv)[o] = __float2bfloat16_rn(bf16_out(v, glu));
         else if (EPI == EPI_STORE_F32) ((float *)Cv)[o] = v;
         else atomicAdd((float *)Cv + o, v);   // a reduction: one add per element and launch, no load on the path
       }
@@ -346,7 +359,7 @@ gemm_small_whole_kernel(const void *__restrict__ Av, const bf16 *__restrict__ W,
       const int n = n0 + r;
       if (m < M && n < N) {
         const size_t o = (size_t)m * ldc + n;
-        if (EPI == EPI_STORE_BF16) ((bf16 *)Cv)[o] = __float2bfloat16_rn(v);
+        if (EPI == EPI_STORE_BF16) ((bf16 *)Cv)[o] = __float2bfloat16_rn(bf16_out(v, glu));
         else if (EPI == EPI_STORE_F32) ((float *)Cv)[o] = v;
         else atomicAdd((float *)Cv + o, v);   // a reduction: one add per element and launch, no load on the path
       }
@@ -529,7 +542,7 @@ gemm_small_stream_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W,
           const int n = n0 + r;
           if (m < M && n < N) {
             const size_t o = (size_t)m * ldc + n;
-            if (epi == EPI_STORE_BF16) ((bf16 *)Cv)[o] = __float2bfloat16_rn(v);
+            if (epi == EPI_STORE_BF16) ((bf16 *)Cv)[o] = __float2bfloat16_rn(bf16_out(v, glu));
             else if (epi == EPI_STORE_F32) ((float *)Cv)[o] = v;
             else atomicAdd((float *)Cv + o, v);   // a reduction: one add per element and launch
           }
@@ -587,10 +600,10 @@ static int launch_whole_depth(const void *A, const void *W, void *C, int M, int 
                        (const bf16 *)W, C, M, N, K, lda, ldw, ldc, 0.f, glu);                         \
   } while (0)
   switch (epi) {
-    G2B_IF_UNGATED(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
-    G2B_IF_UNGATED(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
-    G2B_IF_UNGATED(case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;)
-    case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;
+    G2B_IF_BF16(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
+    G2B_IF_FLOAT(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
+    G2B_IF_FLOAT(case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;)
+    G2B_IF_GATED(case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;)
     default: G2B_REFUSE("gemm_small: unknown epilogue %d", epi);
   }
 #undef G2B_LAUNCH
@@ -630,10 +643,10 @@ static int launch_mt(const void *A, const void *W, void *C, int M, int N, int K,
         (const bf16 *)A, (const bf16 *)W, C, M, N, K, lda, ldw, ldc, glu);                       \
   } while (0)
   switch (epi) {
-    G2B_IF_UNGATED(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
-    G2B_IF_UNGATED(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
-    G2B_IF_UNGATED(case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;)
-    case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;
+    G2B_IF_BF16(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
+    G2B_IF_FLOAT(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
+    G2B_IF_FLOAT(case EPI_ACCUM_F32: G2B_LAUNCH(EPI_ACCUM_F32); break;)
+    G2B_IF_GATED(case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;)
     default: G2B_REFUSE("gemm_small: unknown epilogue %d", epi);
   }
 #undef G2B_LAUNCH
@@ -662,9 +675,9 @@ static int launch_normed(const float *X, const void *W, void *C, int M, int N, i
                stream, (const void *)X, (const bf16 *)W, C, M, N, K, ldx, ldw, ldc, eps, glu);   \
   } while (0)
   switch (epi) {
-    G2B_IF_UNGATED(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
-    G2B_IF_UNGATED(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
-    case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;
+    G2B_IF_BF16(case EPI_STORE_BF16: G2B_LAUNCH(EPI_STORE_BF16); break;)
+    G2B_IF_FLOAT(case EPI_STORE_F32: G2B_LAUNCH(EPI_STORE_F32); break;)
+    G2B_IF_GATED(case EPI_SWIGLU_BF16: G2B_LAUNCH(EPI_SWIGLU_BF16); break;)
     default: G2B_REFUSE("gemm_small_normed: epilogue %d (store or SiLU gate only)", epi);
   }
 #undef G2B_LAUNCH
@@ -716,7 +729,8 @@ static int launch_stream(const void *A, const void *W, void *C, int M, int N, in
 
 // A [M,K] and W [N,K] bfloat16 with unit inner stride; rows 16-byte aligned.
 // epi: 0 store bfloat16, 1 store float, 2 add into float, 3 gate (C is [M, N/2] bfloat16; N must be a
-// multiple of 16): SiLU, or in a build with -DG2B_GLU (that epilogue alone) the form of the glu_ numbers.
+// multiple of 16): SiLU, or in a build with -DG2B_GLU (that epilogue alone) the form of the glu_ numbers; a build with
+// -DG2B_ACT has epilogue 0 alone, behind that form's activation.
 extern "C" int g2b_gemm_small(const void *A, const void *W, void *C, int M, int N, int K, int lda,
                               int ldw, int ldc, int epi, float glu_limit, float glu_offset, float glu_c1,
                               float glu_c3, cudaStream_t stream) {

@@ -38,19 +38,39 @@ constexpr int THREADS = 192;
 enum { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ACCUM_F32 = 2, EPI_SWIGLU_BF16 = 3 };
 // The gate of the gated epilogue: SiLU; in a build with -DG2B_GLU, which holds that epilogue alone, the
 // general form that the launch gives (glu.cuh).
+// A build with -DG2B_ACT holds the bfloat16 store alone, and every value passes the form's activation on its way out.
 #ifdef G2B_GLU
 __device__ __forceinline__ float glu_out(float gate, float up, const GluForm &f) { return glu_value_fast(gate, up, f); }
-#define G2B_CASE_UNGATED(...)
 #else
 __device__ __forceinline__ float glu_out(float gate, float up, const GluForm &) {
   return __fdividef(gate, 1.f + __expf(-gate)) * up;
 }
-#define G2B_CASE_UNGATED(...) G2B_CASE(__VA_ARGS__)
+#endif
+#ifdef G2B_ACT
+__device__ __forceinline__ float bf16_out(float v, const GluForm &f) { return act_value_fast(v, f); }
+#else
+__device__ __forceinline__ float bf16_out(float v, const GluForm &) { return v; }
+#endif
+#if defined(G2B_GLU) || defined(G2B_ACT)
+#define G2B_CASE_FLOAT(...)
+#else
+#define G2B_CASE_FLOAT(...) G2B_CASE(__VA_ARGS__)
+#endif
+#ifdef G2B_GLU
+#define G2B_CASE_BF16(...)
+#else
+#define G2B_CASE_BF16(...) G2B_CASE(__VA_ARGS__)
+#endif
+#ifdef G2B_ACT
+#define G2B_CASE_GATED(...)
+#else
+#define G2B_CASE_GATED(...) G2B_CASE(__VA_ARGS__)
 #endif
 enum { ST_OK = 0, ST_PRODUCER_TIMEOUT = 1, ST_MMA_TIMEOUT = 2, ST_EPILOGUE_TIMEOUT = 3 };
 
-__device__ __forceinline__ uint32_t pack2(uint32_t lo, uint32_t hi) {
-  __nv_bfloat162 v = __floats2bfloat162_rn(__uint_as_float(lo), __uint_as_float(hi));
+// two accumulators on their way into bfloat16
+__device__ __forceinline__ uint32_t pack2(uint32_t lo, uint32_t hi, const GluForm &f) {
+  __nv_bfloat162 v = __floats2bfloat162_rn(bf16_out(__uint_as_float(lo), f), bf16_out(__uint_as_float(hi), f));
   return *reinterpret_cast<uint32_t *>(&v);
 }
 
@@ -140,12 +160,12 @@ __device__ __forceinline__ void epilogue_tile(uint32_t tmem, float *scr, void *_
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
               uint4 v;
-              v.x = pack2(r[j], r[j + 1]); v.y = pack2(r[j + 2], r[j + 3]);
-              v.z = pack2(r[j + 4], r[j + 5]); v.w = pack2(r[j + 6], r[j + 7]);
+              v.x = pack2(r[j], r[j + 1], glu); v.y = pack2(r[j + 2], r[j + 3], glu);
+              v.z = pack2(r[j + 4], r[j + 5], glu); v.w = pack2(r[j + 6], r[j + 7], glu);
               *reinterpret_cast<uint4 *>(dst + j) = v;
             }
           } else {
-            for (int j = 0; j < 32 && n + j < N; ++j) dst[j] = __float2bfloat16_rn(__uint_as_float(r[j]));
+            for (int j = 0; j < 32 && n + j < N; ++j) dst[j] = __float2bfloat16_rn(bf16_out(__uint_as_float(r[j]), glu));
           }
         }
       }
@@ -379,8 +399,8 @@ __device__ __forceinline__ void epilogue_chunk(const uint32_t (&v)[32], int c, u
   } else if (EPI == EPI_STORE_BF16) {
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      put(4 * part + j, make_uint4(pack2(v[8 * j], v[8 * j + 1]), pack2(v[8 * j + 2], v[8 * j + 3]),
-                                   pack2(v[8 * j + 4], v[8 * j + 5]), pack2(v[8 * j + 6], v[8 * j + 7])));
+      put(4 * part + j, make_uint4(pack2(v[8 * j], v[8 * j + 1], glu), pack2(v[8 * j + 2], v[8 * j + 3], glu),
+                                   pack2(v[8 * j + 4], v[8 * j + 5], glu), pack2(v[8 * j + 6], v[8 * j + 7], glu)));
   } else {
     // columns 16b .. 16b+7 are gates, 16b+8 .. 16b+15 the ups of the same outputs
     float h[16];
@@ -1184,6 +1204,7 @@ gemm_tc_wstream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
         }
       } else {
         const size_t o = (size_t)m * ldc + n;
+        if (EPI == EPI_STORE_BF16) v = make_float4(bf16_out(v.x, glu), bf16_out(v.y, glu), bf16_out(v.z, glu), bf16_out(v.w, glu));
         const float f[4] = {v.x, v.y, v.z, v.w};
         if (EPI == EPI_STORE_BF16) {
           bf16 *dst = (bf16 *)Cv + o;
@@ -1478,7 +1499,8 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
 // A [M,K], W [N,K] bfloat16, inner stride 1, row strides multiples of 8 elements, base
 // addresses 16-byte aligned.  epi: 0 store bfloat16, 1 store float, 2 add into float,
 // 3 gate (C is [M, N/2] bfloat16; N a multiple of 16): SiLU, or in a build with -DG2B_GLU (which
-// has no other epilogue) the form of the four glu_ numbers (glu.cuh).  `status` is a device int the
+// has no other epilogue) the form of the four glu_ numbers (glu.cuh).  A build with -DG2B_ACT has epilogue 0
+// alone, behind that form's activation.  `status` is a device int the
 // kernel sets non-zero if one of its bounded waits gave up.  Tile shapes (bn, stages):
 // (64,4) (64,8) (128,3) (128,6) (256,4); bn = 0 picks one from the sizes: wide tiles when
 // there are plenty of them, narrow tiles with a deeper ring when the grid would not fill
@@ -1517,7 +1539,7 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
       if (M <= 64) return launch_wstream<64, 8, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, glu, stream);   \
       return launch_wstream<128, 6, E>(A, W, C, M, N, K, lda, ldw, ldc, bn, status, glu, stream);               \
     }
-    G2B_CASE_UNGATED(EPI_STORE_BF16) G2B_CASE_UNGATED(EPI_STORE_F32) G2B_CASE_UNGATED(EPI_ACCUM_F32) G2B_CASE(EPI_SWIGLU_BF16)
+    G2B_CASE_BF16(EPI_STORE_BF16) G2B_CASE_FLOAT(EPI_STORE_F32) G2B_CASE_FLOAT(EPI_ACCUM_F32) G2B_CASE_GATED(EPI_SWIGLU_BF16)
 #undef G2B_CASE
     G2B_REFUSE("gemm_tc: unknown epilogue %d", epi);
   }
@@ -1543,8 +1565,8 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
     if (bn == BN_ && stages == ST_ && epi == E)                                                      \
       return launch_pair<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, status, glu, stream);
 #define G2B_SHAPE(BN_, ST_) \
-    G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_BF16) G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_F32) G2B_CASE_UNGATED(BN_, ST_, EPI_ACCUM_F32) \
-    G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
+    G2B_CASE_BF16(BN_, ST_, EPI_STORE_BF16) G2B_CASE_FLOAT(BN_, ST_, EPI_STORE_F32) G2B_CASE_FLOAT(BN_, ST_, EPI_ACCUM_F32) \
+    G2B_CASE_GATED(BN_, ST_, EPI_SWIGLU_BF16)
     G2B_SHAPE(256, 6) G2B_SHAPE(256, 4)
 #undef G2B_SHAPE
 #undef G2B_CASE
@@ -1556,8 +1578,8 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
   if (persistent && bn == BN_ && stages == ST_ && epi == E)                                        \
     return launch_persistent<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, parts, status, glu, stream);
 #define G2B_SHAPE(BN_, ST_) \
-  G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_BF16) G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_F32) \
-  G2B_CASE_UNGATED(BN_, ST_, EPI_ACCUM_F32) G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
+  G2B_CASE_BF16(BN_, ST_, EPI_STORE_BF16) G2B_CASE_FLOAT(BN_, ST_, EPI_STORE_F32) \
+  G2B_CASE_FLOAT(BN_, ST_, EPI_ACCUM_F32) G2B_CASE_GATED(BN_, ST_, EPI_SWIGLU_BF16)
   G2B_SHAPE(128, 6) G2B_SHAPE(256, 4)
 #undef G2B_SHAPE
 #undef G2B_CASE
@@ -1566,8 +1588,8 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
 #define G2B_CASE(BN_, ST_, E) \
   if (bn == BN_ && stages == ST_ && epi == E) return launch<BN_, ST_, E>(ma, mw, C, M, N, K, ldc, status, glu, stream);
 #define G2B_SHAPE(BN_, ST_) \
-  G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_BF16) G2B_CASE_UNGATED(BN_, ST_, EPI_STORE_F32) \
-  G2B_CASE_UNGATED(BN_, ST_, EPI_ACCUM_F32) G2B_CASE(BN_, ST_, EPI_SWIGLU_BF16)
+  G2B_CASE_BF16(BN_, ST_, EPI_STORE_BF16) G2B_CASE_FLOAT(BN_, ST_, EPI_STORE_F32) \
+  G2B_CASE_FLOAT(BN_, ST_, EPI_ACCUM_F32) G2B_CASE_GATED(BN_, ST_, EPI_SWIGLU_BF16)
   G2B_SHAPE(64, 4) G2B_SHAPE(64, 8) G2B_SHAPE(128, 3) G2B_SHAPE(128, 6) G2B_SHAPE(256, 4)
 #undef G2B_SHAPE
 #undef G2B_CASE
@@ -1598,7 +1620,7 @@ static int launch_grouped(const CUtensorMap &ma, const CUtensorMap &mw, void *C,
 extern "C" int g2b_gemm_tc_grouped(const void *A, const void *W, void *C, int rows, int n_groups, int Nw, int K,
                                    int lda, int ldc, int epi, const int *plan, int max_tiles, int *status,
                                    float glu_limit, float glu_offset, float glu_c1, float glu_c3, cudaStream_t stream) {
-  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
+  [[maybe_unused]] const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
   if (rows <= 0 || Nw <= 0 || n_groups <= 0 || max_tiles <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8) G2B_REFUSE("gemm_tc: K=%d and the row stride %d must be multiples of 8", K, lda);
   if (((uintptr_t)A | (uintptr_t)W) & 15) G2B_REFUSE("gemm_tc: operands must be 16-byte aligned");
@@ -1611,9 +1633,11 @@ extern "C" int g2b_gemm_tc_grouped(const void *A, const void *W, void *C, int ro
   if (rc) return rc;
   rc = make_map(&mw, W, n_groups * Nw, K, K, 128);
   if (rc) return rc;
+#ifndef G2B_ACT
   if (epi == EPI_SWIGLU_BF16)
     return launch_grouped<128, 6, EPI_SWIGLU_BF16>(ma, mw, C, plan, n_groups, Nw, K, ldc, max_tiles, status, glu, stream);
-#ifndef G2B_GLU
+#endif
+#if !defined(G2B_GLU) && !defined(G2B_ACT)
   if (epi == EPI_STORE_F32)
     return launch_grouped<128, 6, EPI_STORE_F32>(ma, mw, C, plan, n_groups, Nw, K, ldc, max_tiles, status, glu, stream);
 #endif

@@ -21,3 +21,9 @@ __device__ __forceinline__ float glu_value_fast(float gate, float up, const GluF
   const float u = fminf(fmaxf(up, -f.limit), f.limit) + f.offset;
   return __fdividef(g, 1.f + __expf(-(g * fmaf(f.c3 * g, g, f.c1)))) * u;
 }
+
+// The activation alone: z * sigmoid(z (c1 + c3 z^2)).
+__device__ __forceinline__ float act_value(float z, const GluForm &f) { return z / (1.f + expf(-(z * fmaf(f.c3 * z, z, f.c1)))); }
+__device__ __forceinline__ float act_value_fast(float z, const GluForm &f) {
+  return __fdividef(z, 1.f + __expf(-(z * fmaf(f.c3 * z, z, f.c1))));
+}

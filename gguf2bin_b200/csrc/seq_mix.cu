@@ -985,7 +985,7 @@ extern "C" int g2b_state_scan_prompt(int mode, int dtype, const void *q, int q_s
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(128)
-head_norm_gate_kernel(const float *__restrict__ o, int T_tokens, int H, int V, const float *__restrict__ w, float eps,
+head_norm_gate_kernel(const float *__restrict__ o, int T_tokens, int H, int V, const float *__restrict__ w, int w_head, float eps,
                       const T *__restrict__ gate, int gate_stride, float out_scale, T *__restrict__ out) {
   pdl_launch();
   pdl_wait();
@@ -999,22 +999,87 @@ head_norm_gate_kernel(const float *__restrict__ o, int T_tokens, int H, int V, c
   const float inv = 1.f / sqrtf(warp_sum(ss) / (float)V + eps);
   for (int j = lane; j < V; j += 32) {
     float y = p[j] * inv;
-    if (w) y *= w[j];
+    if (w) y *= w[(size_t)h * w_head + j];
     if (gate) y *= silu_f(to_f32(gate[(size_t)t * gate_stride + (size_t)h * V + j]));
     out[(size_t)t * H * V + (size_t)h * V + j] = from_f32<T>(y * out_scale);
   }
 }
 
-extern "C" int g2b_head_norm_gate(const float *o, int T_tokens, int H, int V, const float *w, float eps,
+// The same with four neighbours a lane: L lanes (a power of two) a head, 32 / L heads a warp.  V a multiple of four,
+// everything on 16 bytes (8 for bfloat16).
+template <typename T> __device__ __forceinline__ float4 load4(const T *p);
+template <> __device__ __forceinline__ float4 load4<float>(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+template <> __device__ __forceinline__ float4 load4<bf16>(const bf16 *p) {
+  const uint2 r = *reinterpret_cast<const uint2 *>(p);
+  return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xffff0000u), __uint_as_float(r.y << 16),
+                     __uint_as_float(r.y & 0xffff0000u));
+}
+template <typename T>
+__global__ void __launch_bounds__(128)
+head_norm_gate4_kernel(const float *__restrict__ o, long long items, int H, int V, const float *__restrict__ w, int w_head,
+                       float eps, const T *__restrict__ gate, int gate_stride, float out_scale, T *__restrict__ out, int L) {
+  pdl_launch();
+  pdl_wait();
+  const int lane = threadIdx.x % L;
+  const long long item = (long long)blockIdx.x * (128 / L) + threadIdx.x / L;
+  const bool in = item < items;
+  const int t = in ? (int)(item / H) : 0, h = in ? (int)(item % H) : 0;
+  const float *p = o + ((size_t)t * H + h) * V;
+  float ss = 0.f;
+  if (in)
+    for (int j = 4 * lane; j < V; j += 4 * L) {
+      const float4 x = load4<float>(p + j);
+      ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss))));
+    }
+  for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+  if (!in) return;
+  const float inv = 1.f / sqrtf(ss / (float)V + eps);
+  for (int j = 4 * lane; j < V; j += 4 * L) {
+    float4 y = load4<float>(p + j);
+    y.x *= inv, y.y *= inv, y.z *= inv, y.w *= inv;
+    if (w) {
+      const float4 g = load4<float>(w + (size_t)h * w_head + j);
+      y.x *= g.x, y.y *= g.y, y.z *= g.z, y.w *= g.w;
+    }
+    if (gate) {
+      const float4 g = load4<T>(gate + (size_t)t * gate_stride + (size_t)h * V + j);
+      y.x *= silu_f(g.x), y.y *= silu_f(g.y), y.z *= silu_f(g.z), y.w *= silu_f(g.w);
+    }
+    y.x *= out_scale, y.y *= out_scale, y.z *= out_scale, y.w *= out_scale;
+    join_store4(out + ((size_t)t * H + h) * V + j, y);
+  }
+}
+
+// w_head 0: one weight [V] shared by the heads; V: a weight [H, V]
+extern "C" int g2b_head_norm_gate(const float *o, int T_tokens, int H, int V, const float *w, int w_head, float eps,
                                   const void *gate, int gate_stride, int dtype, float out_scale, void *out,
                                   cudaStream_t stream) {
   if (T_tokens <= 0) return 0;
+  if (w && w_head && w_head != V) G2B_REFUSE("head_norm_gate: weights of %d entries a head of %d", w_head, V);
+  const int es = dtype == G2B_F32 ? 4 : 2;
+  const bool on16 = V % 4 == 0 && !(((uintptr_t)o | (uintptr_t)w) & 15) && !((uintptr_t)out & (4 * es - 1)) &&
+                    (!gate || (!((uintptr_t)gate & (4 * es - 1)) && gate_stride % 4 == 0));
+  if (on16) {
+    int L = 1;
+    while (L < 32 && 4 * L < V) L <<= 1;
+    const long long items = (long long)T_tokens * H;
+    const unsigned blocks = (unsigned)((items + 128 / L - 1) / (128 / L));
+    if (dtype == G2B_F32)
+      g2b_launch(head_norm_gate4_kernel<float>, dim3(blocks), dim3(128), 0, stream, o, items, H, V, w, w_head, eps,
+                 (const float *)gate, gate_stride, out_scale, (float *)out, L);
+    else if (dtype == G2B_BF16)
+      g2b_launch(head_norm_gate4_kernel<bf16>, dim3(blocks), dim3(128), 0, stream, o, items, H, V, w, w_head, eps,
+                 (const bf16 *)gate, gate_stride, out_scale, (bf16 *)out, L);
+    else
+      G2B_REFUSE("head_norm_gate: unknown dtype %d", dtype);
+    return g2b_check_launch("head_norm_gate");
+  }
   const unsigned blocks = (unsigned)(((long long)T_tokens * H + 3) / 4);
   if (dtype == G2B_F32)
-    g2b_launch(head_norm_gate_kernel<float>, dim3(blocks), dim3(128), 0, stream, o, T_tokens, H, V, w, eps,
+    g2b_launch(head_norm_gate_kernel<float>, dim3(blocks), dim3(128), 0, stream, o, T_tokens, H, V, w, w_head, eps,
                (const float *)gate, gate_stride, out_scale, (float *)out);
   else if (dtype == G2B_BF16)
-    g2b_launch(head_norm_gate_kernel<bf16>, dim3(blocks), dim3(128), 0, stream, o, T_tokens, H, V, w, eps,
+    g2b_launch(head_norm_gate_kernel<bf16>, dim3(blocks), dim3(128), 0, stream, o, T_tokens, H, V, w, w_head, eps,
                (const bf16 *)gate, gate_stride, out_scale, (bf16 *)out);
   else
     G2B_REFUSE("head_norm_gate: unknown dtype %d", dtype);
@@ -1039,9 +1104,41 @@ gate_mul_kernel(const T *__restrict__ o, int hd, const T *__restrict__ gate, int
   out[i] = from_f32<T>(y * out_scale);
 }
 
+// bfloat16, eight neighbours a thread (V, hd and the gate's stride multiples of eight)
+__global__ void __launch_bounds__(256)
+gate_mul8_kernel(const bf16 *__restrict__ o, int hd, const bf16 *__restrict__ gate, int gate_stride, long long total8, int H, int V,
+                 float out_scale, bf16 *__restrict__ out) {
+  pdl_launch();
+  pdl_wait();
+  const long long i8 = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i8 >= total8) return;
+  const int n8 = H * V / 8;
+  const int t = (int)(i8 / n8), r = (int)(i8 % n8) * 8, h = r / V, j = r - h * V;
+  const uint4 x = *reinterpret_cast<const uint4 *>(o + ((size_t)t * H + h) * hd + j);
+  uint4 g = make_uint4(0u, 0u, 0u, 0u), y;
+  if (gate) g = *reinterpret_cast<const uint4 *>(gate + (size_t)t * gate_stride + r);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const unsigned xw = (&x.x)[k], gw = (&g.x)[k];
+    float a = __uint_as_float(xw << 16), b = __uint_as_float(xw & 0xffff0000u);
+    if (gate) {
+      a *= sigmoid_f(__uint_as_float(gw << 16));
+      b *= sigmoid_f(__uint_as_float(gw & 0xffff0000u));
+    }
+    *reinterpret_cast<__nv_bfloat162 *>(&(&y.x)[k]) = __floats2bfloat162_rn(a * out_scale, b * out_scale);
+  }
+  *reinterpret_cast<uint4 *>(out + i8 * 8) = y;
+}
+
 extern "C" int g2b_gate_mul(const void *o, int hd, const void *gate, int gate_stride, int dtype, int T_tokens, int H,
                             int V, float out_scale, void *out, cudaStream_t stream) {
   if (T_tokens <= 0) return 0;
+  if (dtype == G2B_BF16 && V % 8 == 0 && hd % 8 == 0 && gate_stride % 8 == 0 && !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)out) & 15)) {
+    const long long total8 = (long long)T_tokens * H * V / 8;
+    g2b_launch(gate_mul8_kernel, dim3((unsigned)((total8 + 255) / 256)), dim3(256), 0, stream, (const bf16 *)o, hd,
+               (const bf16 *)gate, gate_stride, total8, H, V, out_scale, (bf16 *)out);
+    return g2b_check_launch("gate_mul");
+  }
   const unsigned blocks = (unsigned)(((long long)T_tokens * H * V + 255) / 256);
   if (dtype == G2B_F32)
     g2b_launch(gate_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float *)o, hd, (const float *)gate,

@@ -22,6 +22,7 @@
 // Rings are indexed by position, never by step: a decode step that is taken back and run again
 // at the same position reads what the step before it read.
 #include "common.cuh"
+#include "mma.cuh"
 
 G2B_DEFINE_LAST_ERROR
 
@@ -507,7 +508,7 @@ extern "C" int g2b_latent_rope(const void *d, int d_stride, int rank, int rot, i
 // ---------------------------------------------------------------------------
 // products with one small matrix per head.  W [heads * n, r] (rows of head h: h*n .. h*n+n-1).
 //   absorb: out[t, h, 0..r)  = sum_i W[h*n + i, :] * in[t, h, i]        (W_h^T applied; in has n per head)
-//   expand: out[t, h, 0..n)  = W[h*n + i, :] . in[t, h, :], times sigmoid(gate[t, h]) when gate
+//   expand: out[t, h, 0..n)  = W[h*n + i, :] . in[t, h, :], times sigmoid(gate[t, h]) (or gate[t, h * n + i], `gate_each`) when gate
 // One block per (head, tile of HP_ROWS tokens); the sum over the inner index always runs in
 // the same order, so a token's result does not depend on its tile.
 // ---------------------------------------------------------------------------
@@ -566,7 +567,7 @@ head_absorb_kernel(const TA *__restrict__ in, int in_stride, const TA *__restric
 template <typename TA>
 __global__ void __launch_bounds__(HP_THREADS)
 head_expand_kernel(const TA *__restrict__ in, int in_stride, const TA *__restrict__ W,
-                   const TA *__restrict__ gate, int gate_stride, TA *__restrict__ out,
+                   const TA *__restrict__ gate, int gate_stride, int gate_each, TA *__restrict__ out,
                    int out_stride, int T, int heads, int n, int r) {
   pdl_launch();
   pdl_wait();
@@ -596,13 +597,13 @@ head_expand_kernel(const TA *__restrict__ in, int in_stride, const TA *__restric
     float v = acc[0];
 #pragma unroll
     for (int m = 1; m < HP_ROWS; ++m) v = lane == m ? acc[m] : v;
-    if (gate) v *= sigmoid_f(to_f32(gate[(size_t)(t0 + lane) * gate_stride + h]));
+    if (gate) v *= sigmoid_f(to_f32(gate[(size_t)(t0 + lane) * gate_stride + (gate_each ? h * n + i : h)]));
     out[(size_t)(t0 + lane) * out_stride + (size_t)h * n + i] = from_f32<TA>(v);
   }
 }
 
 extern "C" int g2b_head_product(const void *in, int in_stride, const void *W, const void *gate,
-                                int gate_stride, void *out, int out_stride, int T, int heads, int n,
+                                int gate_stride, int gate_each, void *out, int out_stride, int T, int heads, int n,
                                 int r, int expand, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (heads <= 0 || n <= 0 || r <= 0) G2B_REFUSE("head_product: bad sizes heads=%d n=%d r=%d", heads, n, r);
@@ -614,14 +615,14 @@ extern "C" int g2b_head_product(const void *in, int in_stride, const void *W, co
   if (dtype == G2B_F32) {
     if (expand)
       g2b_launch(head_expand_kernel<float>, grid, dim3(HP_THREADS), smem, stream, (const float *)in, in_stride,
-                 (const float *)W, (const float *)gate, gate_stride, (float *)out, out_stride, T, heads, n, r);
+                 (const float *)W, (const float *)gate, gate_stride, gate_each, (float *)out, out_stride, T, heads, n, r);
     else
       g2b_launch(head_absorb_kernel<float>, grid, dim3(HP_THREADS), smem, stream, (const float *)in, in_stride,
                  (const float *)W, (float *)out, out_stride, T, heads, n, r);
   } else if (dtype == G2B_BF16) {
     if (expand)
       g2b_launch(head_expand_kernel<bf16>, grid, dim3(HP_THREADS), smem, stream, (const bf16 *)in, in_stride,
-                 (const bf16 *)W, (const bf16 *)gate, gate_stride, (bf16 *)out, out_stride, T, heads, n, r);
+                 (const bf16 *)W, (const bf16 *)gate, gate_stride, gate_each, (bf16 *)out, out_stride, T, heads, n, r);
     else
       g2b_launch(head_absorb_kernel<bf16>, grid, dim3(HP_THREADS), smem, stream, (const bf16 *)in, in_stride,
                  (const bf16 *)W, (bf16 *)out, out_stride, T, heads, n, r);
@@ -629,6 +630,102 @@ extern "C" int g2b_head_product(const void *in, int in_stride, const void *W, co
     G2B_REFUSE("head_product: unknown dtype %d", dtype);
   }
   return g2b_check_launch("head_product");
+}
+
+// Many rows in bfloat16: the expanding product on the tensor cores (mma.sync), all heads in one launch.  A block takes
+// 64 tokens x 64 outputs of a head, four warps of 16 tokens; both operands' whole rows (r entries, a multiple of 16 once
+// filled with zeros) lie in shared memory.  The gate (one a head, or one an output) is applied to the accumulators.
+#define HT_TILE 64
+__global__ void __launch_bounds__(128)
+head_expand_tile_kernel(const bf16 *__restrict__ in, int in_stride, const bf16 *__restrict__ W, const bf16 *__restrict__ gate,
+                        int gate_stride, int gate_each, bf16 *__restrict__ out, int out_stride, int T, int n, int r, int rp) {
+  pdl_launch();
+  extern __shared__ __align__(128) unsigned char ht_smem[];
+  const int row = rp + 8;                              // 16 bytes of padding: rows of eight start in different banks
+  bf16 *xs = reinterpret_cast<bf16 *>(ht_smem), *ws = xs + HT_TILE * row;
+  const int h = blockIdx.z, t0 = blockIdx.y * HT_TILE, n0 = blockIdx.x * HT_TILE;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int per = rp / 8;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  for (int i = threadIdx.x; i < HT_TILE * per; i += 128) {             // the weights do not wait for an earlier kernel
+    const int m = i / per, k = (i - m * per) * 8;
+    bf16 *d = ws + m * row + k;
+    if (n0 + m < n && k < r) cp_async_16(smem_u32(d), W + ((size_t)h * n + n0 + m) * r + k);
+    else *reinterpret_cast<uint4 *>(d) = zero;
+  }
+  pdl_wait();
+  for (int i = threadIdx.x; i < HT_TILE * per; i += 128) {
+    const int m = i / per, k = (i - m * per) * 8;
+    bf16 *d = xs + m * row + k;
+    if (t0 + m < T && k < r) cp_async_16(smem_u32(d), in + (size_t)(t0 + m) * in_stride + (size_t)h * r + k);
+    else *reinterpret_cast<uint4 *>(d) = zero;
+  }
+  cp_async_commit();
+  cp_async_wait<0>();
+  __syncthreads();
+  float acc[8][4];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  const uint32_t xa = smem_u32(xs + (16 * warp + (lane & 15)) * row + 8 * (lane >> 4));
+  const uint32_t wa = smem_u32(ws + ((lane & 7) + 8 * (lane >> 4)) * row + 8 * ((lane >> 3) & 1));
+  for (int k = 0; k < rp; k += 16) {
+    uint32_t a[4];
+    ldmatrix_x4(a, xa + 2 * k);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {                      // 16 outputs at a time
+      uint32_t b[4];
+      ldmatrix_x4(b, wa + 2 * (16 * j * row + k));
+      mma_bf16_16816(acc[2 * j], a, b[0], b[1]);
+      mma_bf16_16816(acc[2 * j + 1], a, b[2], b[3]);
+    }
+  }
+  const int g = lane >> 2, c = lane & 3;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int t = t0 + 16 * warp + g + 8 * half;
+    if (t >= T) continue;
+    const bf16 *gr = gate ? gate + (size_t)t * gate_stride + (gate_each ? h * n : h) : nullptr;
+    const float one = gate && !gate_each ? sigmoid_f(to_f32(*gr)) : 1.f;
+    bf16 *dst = out + (size_t)t * out_stride + (size_t)h * n;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int col = n0 + 8 * j + 2 * c;              // n is a multiple of eight
+      if (col >= n) continue;
+      float u = acc[j][2 * half], v = acc[j][2 * half + 1];
+      if (gate && gate_each) {
+        const uint32_t z = *reinterpret_cast<const uint32_t *>(gr + col);
+        u *= sigmoid_f(__uint_as_float(z << 16)), v *= sigmoid_f(__uint_as_float(z & 0xffff0000u));
+      } else {
+        u *= one, v *= one;
+      }
+      *reinterpret_cast<uint32_t *>(dst + col) = pack_bf16(u, v);
+    }
+  }
+}
+
+// in [T, heads * r], W [heads * n, r], out [T, heads * n], all bfloat16; n and r multiples of eight, rows of the three on
+// 16, 16 and 4 bytes (a gate per output: on 4).  Returns -1 where the case is not taken.
+extern "C" int g2b_head_expand_tile(const void *in, int in_stride, const void *W, const void *gate, int gate_stride,
+                                    int gate_each, void *out, int out_stride, int T, int heads, int n, int r,
+                                    cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const int rp = (r + 15) / 16 * 16;
+  const size_t smem = (size_t)2 * HT_TILE * (rp + 8) * sizeof(bf16);
+  if (heads <= 0 || n <= 0 || r <= 0 || n % 8 || r % 8 || in_stride % 8 || out_stride % 2 || smem > 200 * 1024 || heads > 65535 ||
+      (T + HT_TILE - 1) / HT_TILE > 65535 || (((uintptr_t)in | (uintptr_t)W) & 15) || ((uintptr_t)out & 3) ||
+      (gate && gate_each && (((uintptr_t)gate & 3) || gate_stride % 2)))
+    return -1;
+  static G2bPerDevice configured;
+  const int dev = g2b_current_device();
+  if (smem > 48 * 1024 && (dev < 0 || configured.value[dev] < (int)smem)) {
+    cudaError_t e = cudaFuncSetAttribute(head_expand_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) G2B_REFUSE("head_expand_tile: shared memory of %zu bytes refused: %s", smem, cudaGetErrorString(e));
+    if (dev >= 0) configured.value[dev] = (int)smem;
+  }
+  const dim3 grid((n + HT_TILE - 1) / HT_TILE, (T + HT_TILE - 1) / HT_TILE, heads);
+  g2b_launch(head_expand_tile_kernel, grid, dim3(128), smem, stream, (const bf16 *)in, in_stride, (const bf16 *)W,
+             (const bf16 *)gate, gate_stride, gate_each, (bf16 *)out, out_stride, T, n, r, rp);
+  return g2b_check_launch("head_expand_tile");
 }
 
 // o[t, h, :] *= sigmoid(gate[t, h]); o [T, heads * n] contiguous.  A block per token.

@@ -22,7 +22,7 @@ __all__ = ["KernelError", "KernelBuildError", "embed_rows", "rmsnorm", "qknorm_r
            "canon_conv", "norm_canon_single", "latent_keep", "head_product", "head_gate", "gated_add", "xielu",
            "proj_norm_rope_cache", "rotate_heads", "short_conv", "state_scan", "head_norm_gate", "gate_mul",
            "norm_add", "norm_shift", "scan_gates_step", "scan_gates_max", "state_readout", "pool_update", "moe_route", "moe_plan", "moe_gemm", "moe_gemv", "moe_gather", "moe_gemm_tc", "moe_combine", "moe_combine_norm_add", "moe_tile_rows", "tanh_norm", "scaled_join", "relu2", "selective_scan", "diff_combine", "GluForm", "norm_join", "moe_combine_join", "latent_pair",
-           "channel_scan", "stream_add", "embed_norm_rows", "streams_read", "streams_join", "shift_mix", "latent_rope", "act_form"]
+           "channel_scan", "stream_add", "embed_norm_rows", "streams_read", "streams_join", "shift_mix", "latent_rope", "act_form", "linear_act", "head_expand_tiles"]
 
 F32, BF16 = 0, 1
 EPI_STORE_F32, EPI_STORE_BF16, EPI_ACCUM_F32 = 0, 1, 2
@@ -504,20 +504,43 @@ def latent_rope(d, rank: int, width: int, norm_w, eps: float, pages, q_in, in_he
           _code(q_in.dtype), _stream())
 
 
+def head_expand_tiles(x, w, out, heads: int, gate=None) -> bool:
+    """``head_product(expand=True)`` for many rows of bfloat16, all heads in one launch on the tensor cores; False where
+    the sizes or alignments do not fit (nothing done)."""
+    n, r = w.shape[0] // heads, w.shape[1]
+    if any(t.dtype != torch.bfloat16 for t in (x, w, out)) or not w.is_contiguous() or x.stride(1) != 1 or out.stride(1) != 1 \
+            or (gate is not None and (gate.stride(1) != 1 or gate.dtype != x.dtype)):
+        return False
+    f = _fn("stream_ops.cu", "g2b_head_expand_tile",
+            [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    global _launches
+    rc = f(_ptr(x), x.stride(0), _ptr(w), _ptr(gate), gate.stride(0) if gate is not None else 0,
+           1 if gate is not None and gate.shape[1] != heads else 0, _ptr(out), out.stride(0), x.shape[0], heads, n, r, _stream())
+    if rc == -1:
+        return False
+    if rc:
+        raise KernelError(f._lib.g2b_last_error().decode("utf-8", "replace"))
+    _launches += 1
+    return True
+
+
 def head_product(x, w, out, heads: int, expand: bool, gate=None) -> None:
     """One small matrix per head, w [heads * n, r].  ``expand`` False: out[t, h] = w_h^T x[t, h]
     (x has n values per head, out r); True: out[t, h] = w_h x[t, h] (x has r per head, out n),
-    times sigmoid(gate[t, h]) when ``gate`` [T, heads] is given.  Views with row strides are taken."""
+    times sigmoid(gate[t, h]) when ``gate`` [T, heads] is given, or times sigmoid(gate[t, h n + i]) with a gate
+    of [T, heads * n].  Views with row strides are taken."""
     n, r = w.shape[0] // heads, w.shape[1]
+    if gate is not None and gate.shape[1] not in (heads, heads * n):
+        raise KernelError("head_product: a gate per head or per output")
     if x.dtype != w.dtype or out.dtype != w.dtype or not w.is_contiguous():
         raise KernelError("head_product: x, w and out must have one dtype, w contiguous")
     if x.stride(1) != 1 or out.stride(1) != 1 or (gate is not None and (gate.stride(1) != 1 or gate.dtype != x.dtype)):
         raise KernelError("head_product: innermost strides must be 1")
     f = _fn("stream_ops.cu", "g2b_head_product",
-            [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
+            [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
              c_int, c_int, c_void_p])
     _call(f, _ptr(x), x.stride(0), _ptr(w), _ptr(gate), gate.stride(0) if gate is not None else 0,
-          _ptr(out), out.stride(0), x.shape[0], heads, n, r, 1 if expand else 0, _code(x.dtype), _stream())
+          1 if gate is not None and gate.shape[1] != heads else 0, _ptr(out), out.stride(0), x.shape[0], heads, n, r, 1 if expand else 0, _code(x.dtype), _stream())
 
 
 def head_gate(o, gate, heads: int) -> None:
@@ -604,6 +627,14 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool
         if (_bf16 or _bf16_mod()).linear_bf16(a, w, out, accumulate):
             return
     gemm_simt(a, w, out, accumulate)
+
+
+def linear_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, form: GluForm) -> bool:
+    """out = act(a @ w.T) with an activation of ``GluForm``'s kind in the product's epilogue; False when no kernel
+    takes the case (the caller then runs the product and ``act_form``)."""
+    if a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and out.dtype == torch.bfloat16:
+        return (_bf16 or _bf16_mod()).linear_act_bf16(a, w, out, form)
+    return False
 
 
 def product_notices(what: str, w: Optional[torch.Tensor], compute_dtype: torch.dtype) -> list:
@@ -990,16 +1021,18 @@ def pool_update(cache_pages, pooled_pages, ctx, n_kv_heads, head_dim, page_size,
 
 
 def head_norm_gate(o32, heads, v_dim, w, eps, gate, out_scale, out) -> None:
-    """out = o / sqrt(mean(o^2) + eps) per head (times ``w`` [v_dim], float32, if given), times
+    """out = o / sqrt(mean(o^2) + eps) per head (times ``w``, float32, if given: [v_dim] or [heads * v_dim]), times
     silu(gate) (if given; [T, heads*v_dim], rows may lie apart), times ``out_scale``."""
     _need(o32, torch.float32, "scan output")
     if w is not None:
         _need(w, torch.float32, "head norm weight")
     f = _fn("seq_mix.cu", "g2b_head_norm_gate",
-            [c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p])
+            [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p])
     if gate is not None and gate.dtype != out.dtype:
         raise KernelError("head_norm_gate: gate and output must have one dtype")
-    _call(f, _ptr(o32), o32.shape[0], heads, v_dim, _ptr(w), eps, _ptr(gate),
+    if w is not None and w.numel() not in (v_dim, heads * v_dim):
+        raise KernelError("head_norm_gate: a weight of one head or of all heads")
+    _call(f, _ptr(o32), o32.shape[0], heads, v_dim, _ptr(w), v_dim if w is not None and w.numel() != v_dim else 0, eps, _ptr(gate),
           _dense_rows(gate, "gate") if gate is not None else 0, _code(out.dtype), out_scale, _ptr(out), _stream())
 
 

@@ -20,7 +20,9 @@ units.SPECIALISED_SOURCES[:] = [("attn_decode.cu", ()), ("attn_decode.cu", ("ATT
                                 ("attn_prefill_tc_split.cu", ()), ("attn_pool_decode.cu", ())]
 # a build with G2B_GLU holds the gated epilogue alone, in the form that a launch gives (other gates than SiLU)
 GLU_DEFINES = ("G2B_GLU",)
-units.BF16_UNITS[:] = [("gemm_small.cu", ()), ("gemm_tc.cu", ()), ("gemm_small.cu", GLU_DEFINES), ("gemm_tc.cu", GLU_DEFINES)]
+# a build with G2B_ACT holds the bfloat16 store alone, behind an activation in the form that a launch gives
+ACT_DEFINES = ("G2B_ACT",)
+units.BF16_UNITS[:] = [(src, d) for d in ((), GLU_DEFINES, ACT_DEFINES) for src in ("gemm_small.cu", "gemm_tc.cu")]
 
 
 SMALL_M = 64                         # rows the weight-streaming product takes
@@ -34,10 +36,17 @@ def _small_ok(a: torch.Tensor, w: torch.Tensor) -> bool:
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
+def _form_defines(epi: int, form) -> tuple:
+    """Which build of the products' sources has the epilogue with that form."""
+    if form == SILU:
+        return ()
+    return GLU_DEFINES if epi == EPI_SWIGLU_BF16 else ACT_DEFINES
+
+
 def _gemm_small(a, w, out, epi, form=SILU) -> None:
     f = _fn("gemm_small.cu", "g2b_gemm_small",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, *_GLU_TYPES, c_void_p],
-            defines=GLU_DEFINES if form != SILU else ())
+            defines=_form_defines(epi, form))
     _call(f, _ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
           w.stride(0), out.stride(0), epi, *form, _stream())
 
@@ -124,7 +133,7 @@ def _gemm_tc(a, w, out, epi, bn: int = 0, stages: int = 0, persistent=False, def
     f = _fn("gemm_tc.cu", "g2b_gemm_tc",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
              c_int, c_int, c_void_p, *_GLU_TYPES, c_void_p],
-            defines=tuple(defines) + (GLU_DEFINES if form != SILU else ()))
+            defines=tuple(defines) + _form_defines(epi, form))
     _call(f, _ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
           w.stride(0), out.stride(0), epi, bn, stages, int(persistent),
           _ptr(_status_word(a.device)), *form, _stream())
@@ -189,6 +198,20 @@ def linear_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate:
         _gemm_tc(a, w, out, epi, bn, stages, persistent)
         return True
     return False
+
+
+def linear_act_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, form) -> bool:
+    """out = act(a @ w.T), bfloat16, the activation on the accumulators."""
+    if out.stride(1) != 1 or form == SILU:       # (the plain builds have no activation)
+        return False
+    choice, bn, stages, persistent = _route(a, w, out)
+    if choice == "small":
+        _gemm_small(a, w, out, EPI_STORE_BF16, form)
+    elif choice == "tc":
+        _gemm_tc(a, w, out, EPI_STORE_BF16, bn, stages, persistent, form=form)
+    else:
+        return False
+    return True
 
 
 def _pick_product(a: torch.Tensor, w: torch.Tensor):

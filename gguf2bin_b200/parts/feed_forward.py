@@ -174,6 +174,11 @@ class ActMLP:
     def _run(self, h, ctx, out32, accumulate: bool) -> None:
         T = h.shape[0]
         ws = ctx.workspace
+        if self.activation == "gelu_tanh" and not self.n_side:
+            mid = ws.buffer("mlp.mid", (T, self.inter), self.dtype)
+            if kernels.linear_act(h, self.w_up, mid, kernels.GluForm.gelu_tanh()):
+                kernels.linear(mid, self.w_down, out32, accumulate=accumulate)
+                return
         up = ws.buffer("mlp.up", (T, self.w_up.shape[0]), self.dtype)
         kernels.linear(h, self.w_up, up)
         self.side_out = up[:, self.inter:self.inter + self.n_side] if self.n_side else None

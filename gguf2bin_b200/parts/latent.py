@@ -224,6 +224,8 @@ class LatentAttention:
         if not fast:
             kernels.head_product(x, w, out, self.nh, expand, gate)
             return
+        if kernels.head_expand_tiles(x, w if expand else self._uk_t.view(self.nh * r, n), out, self.nh, gate):
+            return
         for h in range(self.nh):
             wh = w[h * n:(h + 1) * n]
             if expand:
@@ -231,7 +233,10 @@ class LatentAttention:
             else:
                 kernels.linear(x[:, h * n:(h + 1) * n], self._uk_t[h], out[:, h * r:(h + 1) * r])
         if expand and gate is not None:
-            kernels.head_gate(out, gate, self.nh)
+            if self.wide_gate:
+                kernels.gate_mul(out, n, gate, self.nh, n, 1.0, out)       # in place: an element is read and written by one thread
+            else:
+                kernels.head_gate(out, gate, self.nh)
 
     @property
     def _uk_t(self):
@@ -285,11 +290,7 @@ class LatentAttention:
             o = mix
         else:
             o = ws.buffer("latent.o", (T, self.nh * self.dv), self.dtype)
-            self._per_head(mix, self.w_uv, o, True, None if self.wide_gate else gate)
-            if self.wide_gate:
-                gated = ws.buffer("latent.gated", (T, self.nh * self.dv), self.dtype)
-                kernels.gate_mul(o, self.dv, gate, self.nh, self.dv, 1.0, gated)
-                o = gated
+            self._per_head(mix, self.w_uv, o, True, gate)
         kernels.linear(o, self.w_o, out32, accumulate=accumulate)
 
 

@@ -631,8 +631,7 @@ class WKVMixer:
                              view["state"].states, ctx, o32, self.H, self.D, self.D, 1.0, decay="double_exp", low_tanh=True,
                              bonus=self.bonus)
         og = ws.buffer("wkv.gated", (T, n), self.dtype)
-        kernels.state_readout(o32, self.H, self.D, og, gate=proj[:, 3 * n:], gate_act="silu", gate_first=False, group=self.D,
-                              eps=self.eps, w=self.norm_w)
+        kernels.head_norm_gate(o32, self.H, self.D, self.norm_w, self.eps, proj[:, 3 * n:], 1.0, og)
         kernels.linear(og, self.w_o, residual32, accumulate=accumulate)
 
 

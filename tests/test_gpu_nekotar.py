@@ -101,6 +101,48 @@ def test_gelu_feed_forward(ff, width, dtype):
         close(y.cpu().numpy(), ref, dtype, "gelu feed-forward, stored")
 
 
+@pytest.mark.parametrize("M,N,K", [(1, 96, 64), (7, 40, 256), (12, 512, 1024), (40, 1024, 1024), (50, 128, 96), (100, 2304, 1024),
+                                   (130, 264, 128), (300, 520, 256), (700, 2048, 512), (4100, 1280, 256), (3, 4096, 2048),
+                                   (33, 48, 4096), (16, 4096, 4096), (2048, 1024, 4096)])
+def test_an_activation_in_the_products_epilogues(M, N, K):
+    """Every product kernel (few rows whole and streamed, rows over a cluster, tiles, persistent tiles, parts of K,
+    pairs of CTAs) with the activation on its way out, against that of the 32-bit product; columns of a wider output."""
+    from gguf2bin_b200 import kernels
+    g = torch.Generator(device=DEV).manual_seed(M + N)
+    a = torch.randn((M, K), device=DEV, generator=g).to(torch.bfloat16)
+    w = (torch.randn((N, K), device=DEV, generator=g) * 2.0 / K ** 0.5).to(torch.bfloat16)
+    wide = torch.full((M, N + 16), 7.0, dtype=torch.bfloat16, device=DEV)
+    for out in (torch.full((M, N), 7.0, dtype=torch.bfloat16, device=DEV), wide[:, 8:8 + N]):
+        assert kernels.linear_act(a, w, out, kernels.GluForm.gelu_tanh())
+        ref = NP.gelu_tanh((a.double() @ w.double().t()).cpu().numpy())
+        err = np.abs(out.float().cpu().numpy() - ref)
+        assert err.max() <= 0.006 * np.abs(ref).max() and (err <= 0.01 * np.abs(ref) + 2e-3).all()
+    assert (wide[:, :8] == 7.0).all() and (wide[:, 8 + N:] == 7.0).all()
+
+
+@pytest.mark.parametrize("T,heads,n,r", [(65, 3, 16, 48), (200, 2, 128, 128), (70, 5, 72, 64), (300, 1, 8, 8), (129, 4, 64, 512),
+                                         (66, 16, 136, 40)])
+def test_products_of_small_matrices_per_head(T, heads, n, r):
+    """One launch for all heads, with no gate, a gate per head and a gate per output; rows of wider buffers."""
+    from gguf2bin_b200 import kernels
+    rng = np.random.default_rng(n + r)
+    x, w, g1, g2 = (bf(rng.standard_normal(s)) for s in ((T, heads * r), (heads, n, r), (T, heads), (T, heads * n)))
+    w = bf(w / np.sqrt(r))
+    ref = np.einsum("thr,hnr->thn", x.reshape(T, heads, r), w)
+    wide = torch.zeros((T, heads * r + 24), dtype=torch.bfloat16, device=DEV)
+    wide[:, 16:16 + heads * r] = dev(x, torch.bfloat16)
+    for gate, factor in ((None, 1.0), (g1, NP.sigmoid(g1)[:, :, None]), (g2, NP.sigmoid(g2).reshape(T, heads, n))):
+        gd = dev(gate, torch.bfloat16) if gate is not None else None
+        for xs in (dev(x, torch.bfloat16), wide[:, 16:16 + heads * r]):
+            out = torch.full((T, heads * n), 5.0, dtype=torch.bfloat16, device=DEV)
+            assert kernels.head_expand_tiles(xs, dev(w.reshape(heads * n, r), torch.bfloat16), out, heads, gd)
+            close(out.float().cpu().numpy(), (ref * factor).reshape(T, -1), "bfloat16", "per-head product", loose=0.3)
+        few = torch.full((9, heads * n), 5.0, dtype=torch.bfloat16, device=DEV)
+        kernels.head_product(dev(x[:9], torch.bfloat16), dev(w.reshape(heads * n, r), torch.bfloat16), few, heads, True,
+                             gd[:9] if gd is not None else None)
+        close(few.float().cpu().numpy(), (ref * factor).reshape(T, -1)[:9], "bfloat16", "per-head product of few rows", loose=0.3)
+
+
 # ----------------------------------------------------------------------------
 # latent attention with rotated entries and a gate per element
 # ----------------------------------------------------------------------------
