@@ -988,6 +988,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 // shared memory it is turned, so that C is written in rows, four outputs per lane.
 // Every wait on an mbarrier is bounded as above and no role leaves before the two cluster
 // barriers, whatever it has recorded in `status`.
+constexpr int WS_MAX_SPLITS = 8;            // parts of K, CTAs of a cluster
 template <int BNB, int STAGES> struct SmemWS {
   static constexpr int W_BYTES = BM * BK * 2;
   static constexpr int A_BYTES = BNB * BK * 2;
@@ -1177,7 +1178,7 @@ gemm_tc_wstream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
     for (int m = m_lo + warp; m < m_hi; m += 4) {
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int p = 0; p < 4; ++p) {
+      for (int p = 0; p < WS_MAX_SPLITS; ++p) {
         if (p < splits) {
           const float *src = p == rank ? tile + (size_t)m * BM : recv + ((size_t)p * mq + (m - m_lo)) * BM;
           const float4 t = *reinterpret_cast<const float4 *>(src + 4 * lane);
@@ -1461,10 +1462,11 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
   if (rc) return rc;
   const int tiles = (N + BM - 1) / BM, nkb = (K + BK - 1) / BK;
   // parts of K: as many (up to 4) as keep every CTA on the GPU at once and give a part 4 blocks
-  // or more; three where four would not fit (40 tiles: 120 CTAs instead of 80).  How many
+  // or more; three where four would not fit (40 tiles: 120 CTAs instead of 80); up to 8 for few
+  // tiles with a K so long that a part still has 8 blocks.  How many
   // clusters of a size the GPU holds at once is asked of the runtime: clusters do not straddle
   // the GPU's processing clusters, so it can be fewer than SMs / size.
-  static G2bPerDevice fit[5];                     // fit[s].value[device] = clusters of s CTAs at once (+1; 0 = not asked yet)
+  static G2bPerDevice fit[WS_MAX_SPLITS + 1];     // fit[s].value[device] = clusters of s CTAs at once (+1; 0 = not asked yet)
   auto clusters_at_once = [&](int s) -> int {
     if (cfg_dev >= 0 && fit[s].value[cfg_dev]) return fit[s].value[cfg_dev] - 1;
     cudaLaunchConfig_t cfg = {};
@@ -1486,11 +1488,11 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
     return n;
   };
   int splits = 1;
-  for (int s = 2; s <= 4; ++s)
-    if (nkb / s >= 4 && tiles <= clusters_at_once(s)) splits = s;
-  if (want_splits >= 1 && want_splits <= 4) splits = want_splits;                           // the caller's choice
+  for (int s = 2; s <= WS_MAX_SPLITS; ++s)
+    if (nkb / s >= (s <= 4 ? 4 : 8) && tiles <= clusters_at_once(s)) splits = s;
+  if (want_splits >= 1 && want_splits <= WS_MAX_SPLITS) splits = want_splits;                           // the caller's choice
   while (splits > 1 && (splits - 1) * ((nkb + splits - 1) / splits) >= nkb) --splits;      // no empty part
-  static_assert((2 * BNB + 8) * BM * 4 <= S::RING_BYTES, "the tile and the received ranges must fit the ring");
+  static_assert((2 * BNB + WS_MAX_SPLITS) * BM * 4 <= S::RING_BYTES, "the tile and the received ranges must fit the ring");
   g2b_launch_cluster(gemm_tc_wstream_kernel<BNB, STAGES, EPI>, dim3((unsigned)(tiles * splits)), dim3(THREADS),
                      S::TOTAL, stream, (unsigned)splits, mw, ma, C, M, N, K, ldc, splits, status, glu);
   return g2b_check_launch("gemm_tc (weight streaming)");
@@ -1509,7 +1511,7 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
 // the launcher choose between them; with fewer tiles than half the SMs it takes K in parts over
 // a cluster (persistent = 11 to 14 asks for 1 to 4 parts).  persistent
 // = 2: pairs of CTAs on 256 x 256 tiles, shapes (256,6) and (256,4).  persistent = 3 (at most
-// 128 rows; stages is ignored, bn = 1 to 4 asks for that many parts of K, anything else lets
+// 128 rows; stages is ignored, bn = 1 to 8 asks for that many parts of K, anything else lets
 // the launcher choose): the weight-streaming kernel with K split over a cluster.
 extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, int K, int lda,
                            int ldw, int ldc, int epi, int bn, int stages, int persistent, int *status,
@@ -1528,7 +1530,7 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
   }
   if (persistent == 3) {                           // 17 to 128 rows: the weights stream, K split over a cluster
     if (M > 128) G2B_REFUSE("gemm_tc: the weight-streaming kernel takes at most 128 rows, got %d", M);
-    const bool crowded = (N + BM - 1) / BM > sm_count() && (bn < 1 || bn > 4);
+    const bool crowded = (N + BM - 1) / BM > sm_count() && (bn < 1 || bn > WS_MAX_SPLITS);
 #define G2B_CASE(E) \
     if (epi == E) {                                                                                        \
       /* more tiles than SMs (K is not split then): half the ring, so that two CTAs share an SM and */ \
