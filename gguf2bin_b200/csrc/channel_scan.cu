@@ -484,11 +484,21 @@ channel_carry_kernel(const float *__restrict__ state, float *__restrict__ seg_st
   float S = state[(size_t)slot * per + i];
   float *e = seg_state + (size_t)id0 * per + i;
   const float *p = seg_decay + ((size_t)id0 * H + h) * D + d;
-#pragma unroll 4
-  for (int s = 0; s < segs; ++s) {
-    const float end = s + 1 < segs ? e[(size_t)s * per] : 0.f, dec = s + 1 < segs ? p[(size_t)s * H * D] : 0.f;
-    e[(size_t)s * per] = S;
-    S = fmaf(dec, S, end);
+  // a batch of loads at a time: behind the stores of the places in front, one by one, each would wait for the last
+  constexpr int BATCH = 8;
+  for (int s0 = 0; s0 < segs; s0 += BATCH) {
+    float end[BATCH], dec[BATCH];
+#pragma unroll
+    for (int j = 0; j < BATCH; ++j) {
+      const bool in = s0 + j + 1 < segs;
+      end[j] = in ? e[(size_t)(s0 + j) * per] : 0.f;
+      dec[j] = in ? p[(size_t)(s0 + j) * H * D] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < BATCH; ++j) {
+      if (s0 + j < segs) e[(size_t)(s0 + j) * per] = S;
+      S = fmaf(dec[j], S, end[j]);
+    }
   }
 }
 

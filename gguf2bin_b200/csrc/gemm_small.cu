@@ -72,7 +72,7 @@ __device__ __forceinline__ uint4 ld_stream(const void *p) {
 template <int MT, int EPI>
 __global__ void __launch_bounds__(WARPS * 32)
 gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *__restrict__ Cv,
-                  int M, int N, int K, int lda, int ldw, int ldc, GluForm glu) {
+                  int M, int N, int K, int lda, int ldw, int ldc, ProductTail glu) {
   pdl_launch();
   constexpr int MROWS = MT * 8;
   extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -80,6 +80,7 @@ gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, c = lane & 3;
   const int n0 = blockIdx.x * 16;
+  const int a_row = glu.a_row(n0, M);
   const int nkb = (K + KB - 1) / KB;
 
   const bf16 *w0 = W + (size_t)min(n0 + g, N - 1) * ldw;
@@ -101,7 +102,7 @@ gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *
       const int r = i / (KB / 8), piece = i % (KB / 8);
       const int k = kb * KB + piece * 8;
       bf16 *d = dst + r * XROW + piece * 8;
-      if (r < M && k < K) cp_async_16(smem_u32(d), A + (size_t)r * lda + k);
+      if (r < M && k < K) cp_async_16(smem_u32(d), A + (size_t)(a_row + r) * lda + k);
       else *reinterpret_cast<uint4 *>(d) = make_uint4(0, 0, 0, 0);
     }
   };
@@ -206,7 +207,7 @@ gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *
 template <int MT, int EPI, int DEPTH_WHOLE, int SPLIT, bool NORMED = false>
 __global__ void __launch_bounds__(WARPS * 32, DEPTH_WHOLE == 4 ? 3 : 2)
 gemm_small_whole_kernel(const void *__restrict__ Av, const bf16 *__restrict__ W,
-                        void *__restrict__ Cv, int M, int N, int K, int lda, int ldw, int ldc, float eps, GluForm glu) {
+                        void *__restrict__ Cv, int M, int N, int K, int lda, int ldw, int ldc, float eps, ProductTail glu) {
   static_assert(!NORMED || SPLIT == 1, "the normalised product is not split over a cluster");
   pdl_launch();
   const bf16 *A = reinterpret_cast<const bf16 *>(Av);
@@ -272,7 +273,7 @@ gemm_small_whole_kernel(const void *__restrict__ Av, const bf16 *__restrict__ W,
       if (lane == 0) row_scale[r] = 1.f / sqrtf(ss / (float)K + eps);
       continue;
     }
-    const bf16 *x = A + (size_t)r * lda + k_lo;
+    const bf16 *x = A + (size_t)(glu.a_row(n0, M) + r) * lda + k_lo;
     for (int k = lane * 8; k < k_hi - k_lo; k += 256) cp_async_16(smem_u32(dst + k), x + k);
     for (int k = max(0, k_hi - k_lo) + lane * 4; k < xrow; k += 128) *reinterpret_cast<uint2 *>(dst + k) = make_uint2(0, 0);
   }
@@ -396,7 +397,7 @@ template <int MT>
 __global__ void __launch_bounds__(WARPS * 32, 1)
 gemm_small_stream_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *__restrict__ Cv,
                          int M, int N, int K, int lda, int ldw, int ldc, int epi, int n_chunks, int kbc,
-                         int tiles_per_cta, GluForm glu) {
+                         int tiles_per_cta, ProductTail glu) {
   pdl_launch();
   using C = StreamCfg<MT>;
   constexpr int MROWS = C::MROWS, XROWS = C::XROWS, RING = C::RING, G = STREAM_BATCH;
@@ -409,6 +410,7 @@ gemm_small_stream_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W,
   const int kw = 32 * warp + 8 * c;
   const int n_tiles = (N + 15) / 16;
   const int t_begin = blockIdx.x * tiles_per_cta, t_end = min(n_tiles, t_begin + tiles_per_cta);
+  const int a_row = glu.a_row(t_begin * 16, M);            // a CTA's tiles lie in one group
 
   // ---- the weight stream: blocks in the order (batch of 8 tiles, chunk, tile, block of the chunk)
   int p_tile0 = t_begin, p_chunk = 0, p_j = 0, p_d = 0;    // the block that is copied next
@@ -452,7 +454,7 @@ gemm_small_stream_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W,
     const int k = chunk * kbc * KB + threadIdx.x * 8;
 #pragma unroll
     for (int r = 0; r < MROWS; ++r)
-      areg[r] = (stager && r < M && k < K) ? *reinterpret_cast<const uint4 *>(A + (size_t)r * lda + k)
+      areg[r] = (stager && r < M && k < K) ? *reinterpret_cast<const uint4 *>(A + (size_t)(a_row + r) * lda + k)
                                            : make_uint4(0, 0, 0, 0);
   };
   auto store_a = [&](int buf) {
@@ -581,7 +583,7 @@ static int final_split(int N, int K) {
 
 template <int MT, int DEPTH_WHOLE, int SPLIT>
 static int launch_whole_depth(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw,
-                              int ldc, int epi, GluForm glu, cudaStream_t stream) {
+                              int ldc, int epi, ProductTail glu, cudaStream_t stream) {
   const int smem = (int)whole_smem(MT * 8, K, SPLIT);
   const int n_tiles = (N + 15) / 16;
   const unsigned grid = (unsigned)(n_tiles * SPLIT);
@@ -612,7 +614,7 @@ static int launch_whole_depth(const void *A, const void *W, void *C, int M, int 
 
 template <int MT>
 static int launch_whole(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw, int ldc,
-                        int epi, GluForm glu, cudaStream_t stream) {
+                        int epi, ProductTail glu, cudaStream_t stream) {
   const int nkb = (K + KB - 1) / KB;
   const int split = final_split(N, K);
   if (split == 4) return launch_whole_depth<MT, 4, 4>(A, W, C, M, N, K, lda, ldw, ldc, epi, glu, stream);
@@ -623,7 +625,7 @@ static int launch_whole(const void *A, const void *W, void *C, int M, int N, int
 
 template <int MT>
 static int launch_mt(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw,
-                     int ldc, int epi, GluForm glu, cudaStream_t stream) {
+                     int ldc, int epi, ProductTail glu, cudaStream_t stream) {
   constexpr int MROWS = MT * 8;
   const size_t stage = (size_t)2 * MROWS * XROW * sizeof(bf16);
   const size_t red = (size_t)WARPS * 16 * MROWS * sizeof(float);
@@ -658,7 +660,8 @@ static int launch_mt(const void *A, const void *W, void *C, int M, int N, int K,
 template <int MT, int DEPTH_WHOLE>
 static int launch_normed(const float *X, const void *W, void *C, int M, int N, int K, int ldx, int ldw,
                          int ldc, int epi, float eps, cudaStream_t stream) {
-  const GluForm glu = {INFINITY, 0.f, 1.f, 0.f};             // SiLU
+  ProductTail glu;
+  glu.limit = INFINITY, glu.offset = 0.f, glu.c1 = 1.f, glu.c3 = 0.f, glu.a_group = 0;             // SiLU
   const int smem = (int)whole_smem(MT * 8, K, 1);
   const unsigned grid = (unsigned)((N + 15) / 16);
 #define G2B_LAUNCH(E)                                                                            \
@@ -706,7 +709,7 @@ static bool stream_case(int M, int N, int K) {
 
 template <int MT>
 static int launch_stream(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw, int ldc,
-                         int epi, GluForm glu, cudaStream_t stream) {
+                         int epi, ProductTail glu, cudaStream_t stream) {
   if (epi < EPI_STORE_BF16 || epi > EPI_SWIGLU_BF16) G2B_REFUSE("gemm_small: unknown epilogue %d", epi);
   constexpr int CB = StreamCfg<MT>::CB;
   const int smem = (int)StreamCfg<MT>::TOTAL;
@@ -720,7 +723,8 @@ static int launch_stream(const void *A, const void *W, void *C, int M, int N, in
   }
   const int n_tiles = (N + 15) / 16, nkb = (K + KB - 1) / KB;
   const int n_chunks = (nkb + CB - 1) / CB, kbc = (nkb + n_chunks - 1) / n_chunks;
-  const int per = (n_tiles + sm_count() - 1) / sm_count();          // tiles per CTA: the same for (almost) all
+  int per = (n_tiles + sm_count() - 1) / sm_count();                // tiles per CTA: the same for (almost) all
+  while (glu.a_group && glu.a_group / 16 % per) ++per;              // none across a border of groups
   const unsigned grid = (unsigned)((n_tiles + per - 1) / per);
   g2b_launch(gemm_small_stream_kernel<MT>, dim3(grid), dim3(WARPS * 32), smem, stream, (const bf16 *)A,
              (const bf16 *)W, C, M, N, K, lda, ldw, ldc, epi, n_chunks, kbc, per, glu);
@@ -730,11 +734,13 @@ static int launch_stream(const void *A, const void *W, void *C, int M, int N, in
 // A [M,K] and W [N,K] bfloat16 with unit inner stride; rows 16-byte aligned.
 // epi: 0 store bfloat16, 1 store float, 2 add into float, 3 gate (C is [M, N/2] bfloat16; N must be a
 // multiple of 16): SiLU, or in a build with -DG2B_GLU (that epilogue alone) the form of the glu_ numbers; a build with
-// -DG2B_ACT has epilogue 0 alone, behind that form's activation.
+// -DG2B_ACT has epilogue 0 alone, behind that form's activation.  a_group > 0 (a multiple of 16): as in gemm_tc.cu.
 extern "C" int g2b_gemm_small(const void *A, const void *W, void *C, int M, int N, int K, int lda,
                               int ldw, int ldc, int epi, float glu_limit, float glu_offset, float glu_c1,
-                              float glu_c3, cudaStream_t stream) {
-  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
+                              float glu_c3, int a_group, cudaStream_t stream) {
+  ProductTail glu;
+  glu.limit = glu_limit, glu.offset = glu_offset, glu.c1 = glu_c1, glu.c3 = glu_c3, glu.a_group = a_group;
+  if (a_group < 0 || (a_group && (N % a_group || a_group % 16))) G2B_REFUSE("gemm_small: %d columns in groups of %d", N, a_group);
   if (M <= 0 || N <= 0) return 0;
   if (M > 64) G2B_REFUSE("gemm_small: M=%d (at most 64 rows)", M);
   if (K <= 0 || K % 8 || lda % 8 || ldw % 8)

@@ -174,7 +174,7 @@ __device__ __forceinline__ void epilogue_tile(uint32_t tmem, float *scr, void *_
 template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-               void *__restrict__ Cv, int M, int N, int K, int ldc, int *__restrict__ status, GluForm glu) {
+               void *__restrict__ Cv, int M, int N, int K, int ldc, int *__restrict__ status, ProductTail glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = Smem<BN, STAGES>;
@@ -219,7 +219,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         }
         const uint32_t a_dst = smem_addr(smem + s * S::STAGE_BYTES);
         mbar_expect_tx(full0 + 8 * s, S::STAGE_BYTES);
-        tma_load_2d(a_dst, &map_a, kb * BK, m0, full0 + 8 * s);
+        tma_load_2d(a_dst, &map_a, kb * BK, m0 + glu.a_row(n0, M), full0 + 8 * s);
         tma_load_2d(a_dst + S::A_BYTES, &map_w, kb * BK, n0, full0 + 8 * s);
       }
     }
@@ -275,7 +275,7 @@ template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                        void *__restrict__ Cv, const int *__restrict__ plan, int n_groups, int Nw, int K, int ldc,
-                       int *__restrict__ status, GluForm glu) {
+                       int *__restrict__ status, ProductTail glu) {
   pdl_launch();
   pdl_wait();                  // the plan is an earlier kernel's output
   const int tile = blockIdx.y;
@@ -608,7 +608,7 @@ template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                           const __grid_constant__ CUtensorMap map_c, int M, int N, int K, int group_m,
-                          int k_parts, int *__restrict__ status, GluForm glu) {
+                          int k_parts, int *__restrict__ status, ProductTail glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = SmemP<BN, STAGES>;
@@ -694,7 +694,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
             mbar_expect_tx(full0 + 8 * s, S::STAGE_BYTES);
             tma_load_2d(a_dst + S::A_BYTES, &map_w, kb * BK, n0, full0 + 8 * s);
           }
-          tma_load_2d(a_dst, &map_a, kb * BK, m0, full0 + 8 * s);
+          tma_load_2d(a_dst, &map_a, kb * BK, m0 + glu.a_row(n0, M), full0 + 8 * s);
         }
       }
       TOCK(0, t_prod);
@@ -842,7 +842,7 @@ template <int BN, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     const __grid_constant__ CUtensorMap map_c, int M, int N, int K, int group_m,
-                    int *__restrict__ status, GluForm glu) {
+                    int *__restrict__ status, ProductTail glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = SmemPair<BN, STAGES>;
@@ -900,7 +900,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           }
           const uint32_t a_dst = smem_addr(smem + s * S::STAGE_BYTES);
           if (leader) mbar_expect_tx(full0 + 8 * s, 2 * S::STAGE_BYTES);
-          tma_load_2d_pair(a_dst, &map_a, kb * BK, m0, leader_full0 + 8 * s);
+          tma_load_2d_pair(a_dst, &map_a, kb * BK, m0 + glu.a_row(n0, M), leader_full0 + 8 * s);
           tma_load_2d_pair(a_dst + S::A_BYTES, &map_w, kb * BK, n0, leader_full0 + 8 * s);
         }
       }
@@ -1002,7 +1002,7 @@ template <int BNB, int STAGES, int EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_tc_wstream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
                        void *__restrict__ Cv, int M, int N, int K, int ldc, int splits,
-                       int *__restrict__ status, GluForm glu) {
+                       int *__restrict__ status, ProductTail glu) {
   pdl_launch();
   extern __shared__ unsigned char smem_raw[];
   using S = SmemWS<BNB, STAGES>;
@@ -1073,7 +1073,7 @@ gemm_tc_wstream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
           mbar_expect_tx(full0 + 8 * s, S::STAGE_BYTES);
           tma_load_2d(w_dst, &map_w, kb * BK, n0, full0 + 8 * s);
         }
-        tma_load_2d(w_dst + S::W_BYTES, &map_a, kb * BK, 0, full0 + 8 * s);
+        tma_load_2d(w_dst + S::W_BYTES, &map_a, kb * BK, glu.a_row(n0, M), full0 + 8 * s);
       }
     }
   } else if (warp == 5) {
@@ -1263,7 +1263,7 @@ static int make_map_c(CUtensorMap *map, const void *base, int rows, int cols, in
 
 template <int BN, int STAGES, int EPI>
 static int launch(const CUtensorMap &ma, const CUtensorMap &mw, void *C, int M, int N, int K, int ldc,
-                  int *status, GluForm glu, cudaStream_t stream) {
+                  int *status, ProductTail glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = Smem<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1376,7 +1376,7 @@ static_assert(SmemP<128, 6>::RING_BYTES == 196608 && SmemP<256, 4>::RING_BYTES =
 // want_parts: 1 to 4 parts of K
 template <int BN, int STAGES, int EPI>
 static int launch_persistent(const CUtensorMap &ma, const CUtensorMap &mw, void *C, int M, int N, int K, int ldc,
-                             int want_parts, int *status, GluForm glu, cudaStream_t stream) {
+                             int want_parts, int *status, ProductTail glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = SmemP<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1415,7 +1415,7 @@ static int launch_persistent(const CUtensorMap &ma, const CUtensorMap &mw, void 
 
 template <int BN, int STAGES, int EPI>
 static int launch_pair(const CUtensorMap &ma, const CUtensorMap &mw, void *C, int M, int N, int K, int ldc,
-                       int *status, GluForm glu, cudaStream_t stream) {
+                       int *status, ProductTail glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = SmemPair<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1445,7 +1445,7 @@ static int launch_pair(const CUtensorMap &ma, const CUtensorMap &mw, void *C, in
 
 template <int BNB, int STAGES, int EPI>
 static int launch_wstream(const void *A, const void *W, void *C, int M, int N, int K, int lda, int ldw, int ldc,
-                          int want_splits, int *status, GluForm glu, cudaStream_t stream) {
+                          int want_splits, int *status, ProductTail glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   using S = SmemWS<BNB, STAGES>;
   const int cfg_dev = g2b_current_device();
@@ -1458,7 +1458,7 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
   CUtensorMap mw, ma;
   int rc = make_map(&mw, W, N, K, ldw, BM);
   if (rc) return rc;
-  rc = make_map(&ma, A, M, K, lda, BNB);
+  rc = make_map(&ma, A, glu.a_group ? N / glu.a_group * M : M, K, lda, BNB);
   if (rc) return rc;
   const int tiles = (N + BM - 1) / BM, nkb = (K + BK - 1) / BK;
   // parts of K: as many (up to 4) as keep every CTA on the GPU at once and give a part 4 blocks
@@ -1510,14 +1510,18 @@ static int launch_wstream(const void *A, const void *W, void *C, int M, int N, i
 // the variant with one CTA per SM and two accumulators, shapes (128,6) and (256,4), bn = 0 lets
 // the launcher choose between them; with fewer tiles than half the SMs it takes K in parts over
 // a cluster (persistent = 11 to 14 asks for 1 to 4 parts).  persistent
-// = 2: pairs of CTAs on 256 x 256 tiles, shapes (256,6) and (256,4).  persistent = 3 (at most
+// = 2: pairs of CTAs on 256 x 256 tiles, shapes (256,6) and (256,4).  a_group > 0: columns [i a_group, (i + 1) a_group)
+// of C come from rows [i M, (i + 1) M) of A, which has N / a_group times M rows; a group is a multiple of the tile width.  persistent = 3 (at most
 // 128 rows; stages is ignored, bn = 1 to 8 asks for that many parts of K, anything else lets
 // the launcher choose): the weight-streaming kernel with K split over a cluster.
 extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, int K, int lda,
                            int ldw, int ldc, int epi, int bn, int stages, int persistent, int *status,
-                           float glu_limit, float glu_offset, float glu_c1, float glu_c3, cudaStream_t stream) {
-  const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
+                           float glu_limit, float glu_offset, float glu_c1, float glu_c3, int a_group, cudaStream_t stream) {
+  ProductTail glu;
+  glu.limit = glu_limit, glu.offset = glu_offset, glu.c1 = glu_c1, glu.c3 = glu_c3, glu.a_group = a_group;
   if (M <= 0 || N <= 0) return 0;
+  if (a_group < 0 || (a_group && (N % a_group || (long long)N / a_group * M > 0x7fffffffLL)))
+    G2B_REFUSE("gemm_tc: %d columns in groups of %d", N, a_group);
   if (K <= 0 || K % 8 || lda % 8 || ldw % 8)
     G2B_REFUSE("gemm_tc: K=%d and the row strides (%d, %d) must be multiples of 8", K, lda, ldw);
   if (((uintptr_t)A | (uintptr_t)W) & 15) G2B_REFUSE("gemm_tc: operands must be 16-byte aligned");
@@ -1528,6 +1532,7 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
     if (tiles128 >= 2 * 148) { bn = 128; stages = 3; }
     else { bn = 64; stages = 4; }
   }
+  if (persistent == 3 && a_group && a_group % BM) G2B_REFUSE("gemm_tc: groups of %d columns on tiles %d wide", a_group, BM);
   if (persistent == 3) {                           // 17 to 128 rows: the weights stream, K split over a cluster
     if (M > 128) G2B_REFUSE("gemm_tc: the weight-streaming kernel takes at most 128 rows, got %d", M);
     const bool crowded = (N + BM - 1) / BM > sm_count() && (bn < 1 || bn > WS_MAX_SPLITS);
@@ -1556,8 +1561,9 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
     if (bn == 0) { bn = w; stages = w == 256 ? 4 : 6; }
     parts = p;
   }
+  if (a_group && a_group % bn) G2B_REFUSE("gemm_tc: groups of %d columns on tiles %d wide", a_group, bn);
   CUtensorMap ma, mw;
-  int rc = make_map(&ma, A, M, K, lda, BM);
+  int rc = make_map(&ma, A, a_group ? N / a_group * M : M, K, lda, BM);
   if (rc) return rc;
   if (persistent == 2) {                           // pairs of CTAs: 256 x bn tiles, bn / 2 rows of W per CTA
     if (bn != 256) G2B_REFUSE("gemm_tc: the paired kernel has tiles 256 wide, not %d", bn);
@@ -1600,7 +1606,7 @@ extern "C" int g2b_gemm_tc(const void *A, const void *W, void *C, int M, int N, 
 
 template <int BN, int STAGES, int EPI>
 static int launch_grouped(const CUtensorMap &ma, const CUtensorMap &mw, void *C, const int *plan, int n_groups, int Nw,
-                          int K, int ldc, int max_tiles, int *status, GluForm glu, cudaStream_t stream) {
+                          int K, int ldc, int max_tiles, int *status, ProductTail glu, cudaStream_t stream) {
   static G2bPerDevice configured;
   const int smem = Smem<BN, STAGES>::TOTAL;
   const int cfg_dev = g2b_current_device();
@@ -1622,7 +1628,8 @@ static int launch_grouped(const CUtensorMap &ma, const CUtensorMap &mw, void *C,
 extern "C" int g2b_gemm_tc_grouped(const void *A, const void *W, void *C, int rows, int n_groups, int Nw, int K,
                                    int lda, int ldc, int epi, const int *plan, int max_tiles, int *status,
                                    float glu_limit, float glu_offset, float glu_c1, float glu_c3, cudaStream_t stream) {
-  [[maybe_unused]] const GluForm glu = {glu_limit, glu_offset, glu_c1, glu_c3};
+  [[maybe_unused]] ProductTail glu;
+  glu.limit = glu_limit, glu.offset = glu_offset, glu.c1 = glu_c1, glu.c3 = glu_c3, glu.a_group = 0;
   if (rows <= 0 || Nw <= 0 || n_groups <= 0 || max_tiles <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8) G2B_REFUSE("gemm_tc: K=%d and the row stride %d must be multiples of 8", K, lda);
   if (((uintptr_t)A | (uintptr_t)W) & 15) G2B_REFUSE("gemm_tc: operands must be 16-byte aligned");

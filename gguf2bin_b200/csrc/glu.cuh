@@ -27,3 +27,11 @@ __device__ __forceinline__ float act_value(float z, const GluForm &f) { return z
 __device__ __forceinline__ float act_value_fast(float z, const GluForm &f) {
   return __fdividef(z, 1.f + __expf(-(z * fmaf(f.c3 * z, z, f.c1))));
 }
+
+// What a product's kernel gets beside its operands: the form of its epilogue, and, where the columns of C come from
+// several inputs (W's rows in groups of `a_group`, A a stack of as many [M, K] matrices), the size of a group; 0: one A.
+struct ProductTail : GluForm {
+  int a_group;
+  // the first row of the A that the columns from n0 on are a product of
+  __device__ __forceinline__ int a_row(int n0, int M) const { return a_group ? n0 / a_group * M : 0; }
+};

@@ -226,6 +226,80 @@ proj_rope_cache_headwise_kernel(const T *__restrict__ qkv, int row_stride, const
   for (int d = lane; d < hd; d += 32) dst[d] = from_f32<T>(d < n ? x[d] : 0.f);
 }
 
+// The same where nothing is normed either, in bfloat16: eight neighbours of a head a thread, the other half of their
+// pairs loaded beside them.  D, V, hd multiples of eight; rotated halves a multiple of eight (or neighbouring pairs).
+__global__ void __launch_bounds__(256)
+proj_rope_cache_vec_kernel(const bf16 *__restrict__ qkv, int row_stride, const float *__restrict__ bias, int nh, int nkv, int D,
+                           int V, const float2 *__restrict__ rope, int rot, int interleaved, const int *__restrict__ tok_pos,
+                           const int *__restrict__ tok_seq, const int *__restrict__ page_table, int P, bf16 *__restrict__ cache,
+                           int page_size, bf16 *__restrict__ q_out, int nvh, int hd, int n_tokens) {
+  pdl_launch();
+  pdl_wait();
+  const int heads = nh + nkv + nvh, per_head = hd >> 3, per_token = heads * per_head;
+  const long long item = (long long)blockIdx.x * 256 + threadIdx.x;
+  const int t = (int)(item / per_token);
+  if (t >= n_tokens) return;
+  const int r = (int)(item - (long long)t * per_token), h = r / per_head, d = (r - h * per_head) * 8;
+  const bool is_v = h >= nh + nkv;
+  const int n = is_v ? V : D;
+  const int col = is_v ? (nh + nkv) * D + (h - nh - nkv) * V : h * D;
+  const bf16 *src = qkv + (size_t)t * row_stride + col;
+  float x[8];
+  auto fetch = [&](int at, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4 *>(src + at);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const unsigned u = (&raw.x)[i];
+      v[2 * i] = __uint_as_float(u << 16), v[2 * i + 1] = __uint_as_float(u & 0xffff0000u);
+    }
+    if (bias) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[i] += bias[col + at + i];
+    }
+  };
+  if (d < n) {
+    fetch(d, x);
+    if (!is_v && rope && d < rot) {
+      const int half = rot >> 1;
+      const float2 *cs = rope + (size_t)t * half;
+      if (interleaved) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 c = cs[(d >> 1) + i];
+          const float u = x[2 * i], v = x[2 * i + 1];
+          x[2 * i] = u * c.x - v * c.y;
+          x[2 * i + 1] = v * c.x + u * c.y;
+        }
+      } else {
+        const bool upper = d >= half;
+        float o[8];
+        fetch(upper ? d - half : d + half, o);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float2 c = cs[(upper ? d - half : d) + i];
+          x[i] = upper ? x[i] * c.x + o[i] * c.y : x[i] * c.x - o[i] * c.y;
+        }
+      }
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] = 0.f;
+  }
+  bf16 *dst;
+  if (h < nh) {
+    dst = q_out + ((size_t)t * nh + h) * hd + d;
+  } else {
+    const int pos = tok_pos[t];
+    const size_t page = (size_t)page_table[(size_t)tok_seq[t] * P + pos / page_size];
+    const int kh = is_v ? h - nh - nkv : h - nh;
+    dst = cache + (((page * 2 + (is_v ? 1 : 0)) * nkv + kh) * page_size + pos % page_size) * hd + d;
+  }
+  uint4 y;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) *reinterpret_cast<__nv_bfloat162 *>(&(&y.x)[i]) = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+  *reinterpret_cast<uint4 *>(dst) = y;
+}
+
 extern "C" int g2b_proj_norm_rope_cache(const void *qkv, int dtype, int row_stride, int T_tokens,
                                         const float *bias, int nh, int nkv, int D, int V, const float *q_w,
                                         const float *k_w, float eps, const float *rope, int rot, int interleaved,
@@ -237,6 +311,17 @@ extern "C" int g2b_proj_norm_rope_cache(const void *qkv, int dtype, int row_stri
   if (nkv < 0 || nvh < 0 || nvh > nkv) G2B_REFUSE("proj_norm_rope_cache: %d value heads beside %d key heads", nvh, nkv);
   if (hd < D || hd < V) G2B_REFUSE("proj_norm_rope_cache: heads of %d and %d in rows of %d", D, V, hd);
   if (nkv > 0 && !cache) G2B_REFUSE("proj_norm_rope_cache: keys without pages to write them to");
+  if (dtype == G2B_BF16 && !q_w && !k_w && unit_eps <= 0.f && v_norm_eps <= 0.f && D % 8 == 0 && V % 8 == 0 && hd % 8 == 0 &&
+      row_stride % 8 == 0 && (!rope || interleaved ? rot % 8 == 0 : rot % 16 == 0) &&
+      !(((uintptr_t)qkv | (uintptr_t)cache | (uintptr_t)q_out) & 15)) {
+    const long long items = (long long)T_tokens * (nh + nkv + nvh) * (hd / 8);
+    if ((items + 255) / 256 <= 0x7fffffffLL) {
+      g2b_launch(proj_rope_cache_vec_kernel, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, stream, (const bf16 *)qkv,
+                 row_stride, bias, nh, nkv, D, V, (const float2 *)rope, rot, interleaved, tok_pos, tok_seq, page_table, P,
+                 (bf16 *)cache, page_size, (bf16 *)q_out, nvh, hd, T_tokens);
+      return g2b_check_launch("proj_norm_rope_cache");
+    }
+  }
   if (norm_per_head || (!q_w && !k_w)) {                // nothing spans the heads: a warp a (token, head)
     const long long n_items = (long long)T_tokens * (nh + nkv + nvh);
     const long long blocks = (n_items + HEADWISE_WARPS - 1) / HEADWISE_WARPS;
@@ -1026,23 +1111,29 @@ head_norm_gate4_kernel(const float *__restrict__ o, long long items, int H, int 
   const int t = in ? (int)(item / H) : 0, h = in ? (int)(item % H) : 0;
   const float *p = o + ((size_t)t * H + h) * V;
   float ss = 0.f;
+  // the lane's first four of everything, asked for at once
+  const int j0 = min(4 * lane, V - 4);
+  const float4 x0 = load4<float>(p + j0);
+  const float4 w0 = w ? load4<float>(w + (size_t)h * w_head + j0) : make_float4(1.f, 1.f, 1.f, 1.f);
+  const float4 g0 = gate ? load4<T>(gate + (size_t)t * gate_stride + (size_t)h * V + j0) : make_float4(0.f, 0.f, 0.f, 0.f);
   if (in)
     for (int j = 4 * lane; j < V; j += 4 * L) {
-      const float4 x = load4<float>(p + j);
+      const float4 x = j == 4 * lane ? x0 : load4<float>(p + j);
       ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss))));
     }
   for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
   if (!in) return;
   const float inv = 1.f / sqrtf(ss / (float)V + eps);
   for (int j = 4 * lane; j < V; j += 4 * L) {
-    float4 y = load4<float>(p + j);
+    const bool again = j != 4 * lane;
+    float4 y = again ? load4<float>(p + j) : x0;
     y.x *= inv, y.y *= inv, y.z *= inv, y.w *= inv;
     if (w) {
-      const float4 g = load4<float>(w + (size_t)h * w_head + j);
+      const float4 g = again ? load4<float>(w + (size_t)h * w_head + j) : w0;
       y.x *= g.x, y.y *= g.y, y.z *= g.z, y.w *= g.w;
     }
     if (gate) {
-      const float4 g = load4<T>(gate + (size_t)t * gate_stride + (size_t)h * V + j);
+      const float4 g = again ? load4<T>(gate + (size_t)t * gate_stride + (size_t)h * V + j) : g0;
       y.x *= silu_f(g.x), y.y *= silu_f(g.y), y.z *= silu_f(g.z), y.w *= silu_f(g.w);
     }
     y.x *= out_scale, y.y *= out_scale, y.z *= out_scale, y.w *= out_scale;

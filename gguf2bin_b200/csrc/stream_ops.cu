@@ -661,6 +661,18 @@ head_expand_tile_kernel(const bf16 *__restrict__ in, int in_stride, const bf16 *
     else *reinterpret_cast<uint4 *>(d) = zero;
   }
   cp_async_commit();
+  // the gate's words of this thread's outputs, on their way while the products run
+  const int g = lane >> 2, c = lane & 3;
+  uint32_t z[2][8];
+  if (gate && gate_each) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int t = t0 + 16 * warp + g + 8 * half, col = n0 + 8 * j + 2 * c;
+        z[half][j] = t < T && col < n ? *reinterpret_cast<const uint32_t *>(gate + (size_t)t * gate_stride + h * n + col) : 0u;
+      }
+  }
   cp_async_wait<0>();
   __syncthreads();
   float acc[8][4];
@@ -679,13 +691,11 @@ head_expand_tile_kernel(const bf16 *__restrict__ in, int in_stride, const bf16 *
       mma_bf16_16816(acc[2 * j + 1], a, b[2], b[3]);
     }
   }
-  const int g = lane >> 2, c = lane & 3;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int t = t0 + 16 * warp + g + 8 * half;
     if (t >= T) continue;
-    const bf16 *gr = gate ? gate + (size_t)t * gate_stride + (gate_each ? h * n : h) : nullptr;
-    const float one = gate && !gate_each ? sigmoid_f(to_f32(*gr)) : 1.f;
+    const float one = gate && !gate_each ? sigmoid_f(to_f32(gate[(size_t)t * gate_stride + h])) : 1.f;
     bf16 *dst = out + (size_t)t * out_stride + (size_t)h * n;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -693,8 +703,7 @@ head_expand_tile_kernel(const bf16 *__restrict__ in, int in_stride, const bf16 *
       if (col >= n) continue;
       float u = acc[j][2 * half], v = acc[j][2 * half + 1];
       if (gate && gate_each) {
-        const uint32_t z = *reinterpret_cast<const uint32_t *>(gr + col);
-        u *= sigmoid_f(__uint_as_float(z << 16)), v *= sigmoid_f(__uint_as_float(z & 0xffff0000u));
+        u *= sigmoid_f(__uint_as_float(z[half][j] << 16)), v *= sigmoid_f(__uint_as_float(z[half][j] & 0xffff0000u));
       } else {
         u *= one, v *= one;
       }

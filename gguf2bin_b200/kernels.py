@@ -22,7 +22,7 @@ __all__ = ["KernelError", "KernelBuildError", "embed_rows", "rmsnorm", "qknorm_r
            "canon_conv", "norm_canon_single", "latent_keep", "head_product", "head_gate", "gated_add", "xielu",
            "proj_norm_rope_cache", "rotate_heads", "short_conv", "state_scan", "head_norm_gate", "gate_mul",
            "norm_add", "norm_shift", "scan_gates_step", "scan_gates_max", "state_readout", "pool_update", "moe_route", "moe_plan", "moe_gemm", "moe_gemv", "moe_gather", "moe_gemm_tc", "moe_combine", "moe_combine_norm_add", "moe_tile_rows", "tanh_norm", "scaled_join", "relu2", "selective_scan", "diff_combine", "GluForm", "norm_join", "moe_combine_join", "latent_pair",
-           "channel_scan", "stream_add", "embed_norm_rows", "streams_read", "streams_join", "shift_mix", "latent_rope", "act_form", "linear_act", "head_expand_tiles"]
+           "channel_scan", "stream_add", "embed_norm_rows", "streams_read", "streams_join", "shift_mix", "latent_rope", "act_form", "linear_act", "linear_stacked", "head_expand_tiles"]
 
 F32, BF16 = 0, 1
 EPI_STORE_F32, EPI_STORE_BF16, EPI_ACCUM_F32 = 0, 1, 2
@@ -627,6 +627,18 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool
         if (_bf16 or _bf16_mod()).linear_bf16(a, w, out, accumulate):
             return
     gemm_simt(a, w, out, accumulate)
+
+
+def linear_stacked(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """Several products of inputs of their own side by side: out[:, i N:(i + 1) N] = a[i] @ w[i].T; a [G, M, K] and
+    w [G, N, K] contiguous, out [M, G N].  One launch where a kernel takes the case."""
+    G, N = w.shape[0], w.shape[1]
+    if a.shape[0] != G or out.shape[1] != G * N or not a.is_contiguous() or not w.is_contiguous():
+        raise KernelError("linear_stacked: contiguous stacks of matrices, and an output with a range of columns for each")
+    if a.dtype == w.dtype == out.dtype == torch.bfloat16 and (_bf16 or _bf16_mod()).linear_stacked_bf16(a, w, out):
+        return
+    for i in range(G):
+        linear(a[i], w[i], out[:, i * N:(i + 1) * N])
 
 
 def linear_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, form: GluForm) -> bool:

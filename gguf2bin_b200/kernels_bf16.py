@@ -43,12 +43,13 @@ def _form_defines(epi: int, form) -> tuple:
     return GLU_DEFINES if epi == EPI_SWIGLU_BF16 else ACT_DEFINES
 
 
-def _gemm_small(a, w, out, epi, form=SILU) -> None:
+def _gemm_small(a, w, out, epi, form=SILU, a_group: int = 0) -> None:
+    """``a_group`` > 0: ``a`` is a stack of matrices [G * M, K]; that many columns of ``out`` come from each."""
     f = _fn("gemm_small.cu", "g2b_gemm_small",
-            [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, *_GLU_TYPES, c_void_p],
+            [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, *_GLU_TYPES, c_int, c_void_p],
             defines=_form_defines(epi, form))
-    _call(f, _ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
-          w.stride(0), out.stride(0), epi, *form, _stream())
+    _call(f, _ptr(a), _ptr(w), _ptr(out), out.shape[0], w.shape[0], a.shape[1], a.stride(0),
+          w.stride(0), out.stride(0), epi, *form, a_group, _stream())
 
 
 def normed_product(x32: torch.Tensor, eps: float, w: torch.Tensor, out: torch.Tensor, gated: bool) -> bool:
@@ -124,7 +125,7 @@ def _tc_ok(a: torch.Tensor, w: torch.Tensor) -> bool:
             and w.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def _gemm_tc(a, w, out, epi, bn: int = 0, stages: int = 0, persistent=False, defines=(), form=SILU) -> None:
+def _gemm_tc(a, w, out, epi, bn: int = 0, stages: int = 0, persistent=False, defines=(), form=SILU, a_group: int = 0) -> None:
     """bn = 0 lets the launcher pick the tile shape from the sizes.  persistent: one CTA per SM
     walks over the tiles with two accumulators (shapes (128, 6) and (256, 4)); persistent = 2:
     pairs of CTAs on 256 x 256 tiles (shapes (256, 6) and (256, 4)); persistent = 3: at most 128
@@ -132,11 +133,11 @@ def _gemm_tc(a, w, out, epi, bn: int = 0, stages: int = 0, persistent=False, def
     ``defines``: another build of the source (the tests' build whose waits run out)."""
     f = _fn("gemm_tc.cu", "g2b_gemm_tc",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_int, c_int, c_void_p, *_GLU_TYPES, c_void_p],
+             c_int, c_int, c_void_p, *_GLU_TYPES, c_int, c_void_p],
             defines=tuple(defines) + _form_defines(epi, form))
-    _call(f, _ptr(a), _ptr(w), _ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
+    _call(f, _ptr(a), _ptr(w), _ptr(out), out.shape[0], w.shape[0], a.shape[1], a.stride(0),
           w.stride(0), out.stride(0), epi, bn, stages, int(persistent),
-          _ptr(_status_word(a.device)), *form, _stream())
+          _ptr(_status_word(a.device)), *form, a_group, _stream())
 
 
 def gemm_tc_grouped(a_rows, w, n_out: int, plan, n_groups: int, max_tiles: int, swiglu: bool, out, form=SILU) -> bool:
@@ -200,6 +201,22 @@ def linear_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate:
     return False
 
 
+def linear_stacked_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
+    """out[:, i N:(i + 1) N] = a[i] @ w[i].T for a [G, M, K], w [G, N, K], out [M, G N], all bfloat16 and a, w contiguous, in
+    one launch; False where a tile would lie across two of the products (or the sizes do not fit)."""
+    G, M, K = a.shape
+    N = w.shape[1]
+    flat_a, flat_w = a.view(G * M, K), w.view(G * N, K)
+    choice, bn, stages, persistent = _route(a[0], flat_w, out)
+    if choice == "small" and N % 16 == 0:
+        _gemm_small(flat_a, flat_w, out, EPI_STORE_BF16, a_group=N)
+    elif choice == "tc" and N % 256 == 0:            # whatever the tiles' width
+        _gemm_tc(flat_a, flat_w, out, EPI_STORE_BF16, bn, stages, persistent, a_group=N)
+    else:
+        return False
+    return True
+
+
 def linear_act_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, form) -> bool:
     """out = act(a @ w.T), bfloat16, the activation on the accumulators."""
     if out.stride(1) != 1 or form == SILU:       # (the plain builds have no activation)
@@ -260,6 +277,8 @@ def _wstream_case(M: int, N: int, K: int) -> bool:
         if M <= 64:
             return True
         return N < 8192 and M <= 96
+    if 1024 <= N < 2048 and K >= 4096 and M <= 32:
+        return True                    # 1024 x 4608: 5.7 to 6.4 us in eight parts of K against 9.6 to 11.0 by the mma.sync kernel
     if N > 65536:                      # a vocabulary with a short K
         return 8 < M <= 64 and K >= 1024
     if M <= 16 or N < 1024 or K < 1024 or N > 16384:

@@ -622,8 +622,7 @@ class WKVMixer:
         mixed = ws.buffer("wkv.mixed", (len(self.MIXES), T, self.hidden), self.dtype)
         kernels.shift_mix(h, self.mu, view["shift"].states, ctx, mixed)
         proj = ws.buffer("wkv.in", (T, 4 * n), self.dtype)
-        for i in range(4):
-            kernels.linear(mixed[i], self.w_in[i], proj[:, i * n:(i + 1) * n])
+        kernels.linear_stacked(mixed[:4], self.w_in, proj)
         low = ws.buffer("wkv.low", (T, self.w_low1.shape[0]), torch.float32)           # 32-bit: it enters the decay
         kernels.linear(mixed[4], self.w_low1, low)
         o32 = ws.buffer("wkv.o", (T, n), torch.float32)

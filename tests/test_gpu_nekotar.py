@@ -120,6 +120,25 @@ def test_an_activation_in_the_products_epilogues(M, N, K):
     assert (wide[:, :8] == 7.0).all() and (wide[:, 8 + N:] == 7.0).all()
 
 
+@pytest.mark.parametrize("G,M,N,K", [(4, 1, 64, 72), (3, 8, 48, 1024), (4, 8, 2048, 2048), (2, 13, 128, 256), (5, 40, 272, 512),
+                                     (4, 3, 1024, 2048), (3, 100, 256, 512), (4, 300, 512, 256), (2, 2048, 768, 512),
+                                     (3, 4200, 256, 256), (4, 130, 96, 64), (2, 7, 20, 64), (4, 16, 4096, 4096)])
+def test_products_of_several_inputs_side_by_side(G, M, N, K):
+    """A stack of inputs, each for a range of the output's columns, in one launch where a kernel takes the case (few rows
+    whole and streamed, rows over a cluster, tiles, persistent tiles, pairs of CTAs) and one by one where none does."""
+    from gguf2bin_b200 import kernels
+    gen = torch.Generator(device=DEV).manual_seed(M + N)
+    a = torch.randn((G, M, K), device=DEV, generator=gen).to(torch.bfloat16)
+    w = (torch.randn((G, N, K), device=DEV, generator=gen) / K ** 0.5).to(torch.bfloat16)
+    out = torch.full((M, G * N), 7.0, dtype=torch.bfloat16, device=DEV)
+    kernels.linear_stacked(a, w, out)
+    ref = torch.einsum("gmk,gnk->mgn", a.double(), w.double()).reshape(M, G * N).cpu().numpy()
+    assert np.abs(out.float().cpu().numpy() - ref).max() <= 0.006 * np.abs(ref).max()
+    out32 = torch.empty((M, G * N), dtype=torch.float32, device=DEV)
+    kernels.linear_stacked(a.float(), w.float(), out32)
+    assert np.abs(out32.cpu().numpy() - ref).max() <= 1e-4 * np.abs(ref).max()
+
+
 @pytest.mark.parametrize("T,heads,n,r", [(65, 3, 16, 48), (200, 2, 128, 128), (70, 5, 72, 64), (300, 1, 8, 8), (129, 4, 64, 512),
                                          (66, 16, 136, 40)])
 def test_products_of_small_matrices_per_head(T, heads, n, r):
