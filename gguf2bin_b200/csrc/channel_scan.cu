@@ -191,7 +191,7 @@ static int launch_channel_step(const ChannelIn &a, float *state, const int *seq_
 // ---------------------------------------------------------------------------
 // prompts: what every column of a head needs of a token, once
 // ---------------------------------------------------------------------------
-#define CP_TOKENS 4
+#define CP_TOKENS 8
 #define CP_THREADS 128
 template <typename T>
 __global__ void __launch_bounds__(CP_THREADS)

@@ -13,6 +13,8 @@
 //  * The 8 partial sums of an output are added in warp order through shared memory: the
 //    order of the sum depends on K only, not on M or on the batch's contents.
 //
+// The kernels read weights above pdl_wait(); A carries no __restrict__, so that no load of it can be moved there.
+//
 // Two ways of staging the activations.  `gemm_small_kernel` stages one 256-wide block of K
 // at a time (any K, M up to 64).  `gemm_small_whole_kernel` stages all of A once, when
 // M x K fits shared memory: its K loop then has no barrier at all and up to 8 blocks of W are
@@ -71,7 +73,7 @@ __device__ __forceinline__ uint4 ld_stream(const void *p) {
 
 template <int MT, int EPI>
 __global__ void __launch_bounds__(WARPS * 32)
-gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *__restrict__ Cv,
+gemm_small_kernel(const bf16 *A, const bf16 *__restrict__ W, void *__restrict__ Cv,
                   int M, int N, int K, int lda, int ldw, int ldc, ProductTail glu) {
   pdl_launch();
   constexpr int MROWS = MT * 8;
@@ -206,7 +208,7 @@ gemm_small_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *
 // normalises nor stores anything twice, and the step has one dependent launch less.
 template <int MT, int EPI, int DEPTH_WHOLE, int SPLIT, bool NORMED = false>
 __global__ void __launch_bounds__(WARPS * 32, DEPTH_WHOLE == 4 ? 3 : 2)
-gemm_small_whole_kernel(const void *__restrict__ Av, const bf16 *__restrict__ W,
+gemm_small_whole_kernel(const void *Av, const bf16 *__restrict__ W,
                         void *__restrict__ Cv, int M, int N, int K, int lda, int ldw, int ldc, float eps, ProductTail glu) {
   static_assert(!NORMED || SPLIT == 1, "the normalised product is not split over a cluster");
   pdl_launch();
@@ -395,7 +397,7 @@ constexpr int STREAM_BATCH = 8;                     // tiles whose accumulators 
 
 template <int MT>
 __global__ void __launch_bounds__(WARPS * 32, 1)
-gemm_small_stream_kernel(const bf16 *__restrict__ A, const bf16 *__restrict__ W, void *__restrict__ Cv,
+gemm_small_stream_kernel(const bf16 *A, const bf16 *__restrict__ W, void *__restrict__ Cv,
                          int M, int N, int K, int lda, int ldw, int ldc, int epi, int n_chunks, int kbc,
                          int tiles_per_cta, ProductTail glu) {
   pdl_launch();

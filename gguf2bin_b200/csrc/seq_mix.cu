@@ -236,10 +236,10 @@ proj_rope_cache_vec_kernel(const bf16 *__restrict__ qkv, int row_stride, const f
   pdl_launch();
   pdl_wait();
   const int heads = nh + nkv + nvh, per_head = hd >> 3, per_token = heads * per_head;
-  const long long item = (long long)blockIdx.x * 256 + threadIdx.x;
-  const int t = (int)(item / per_token);
+  const unsigned item = blockIdx.x * 256 + threadIdx.x;
+  const int t = (int)(item / (unsigned)per_token);
   if (t >= n_tokens) return;
-  const int r = (int)(item - (long long)t * per_token), h = r / per_head, d = (r - h * per_head) * 8;
+  const int r = (int)(item - (unsigned)t * per_token), h = r / per_head, d = (r - h * per_head) * 8;
   const bool is_v = h >= nh + nkv;
   const int n = is_v ? V : D;
   const int col = is_v ? (nh + nkv) * D + (h - nh - nkv) * V : h * D;
@@ -315,7 +315,7 @@ extern "C" int g2b_proj_norm_rope_cache(const void *qkv, int dtype, int row_stri
       row_stride % 8 == 0 && (!rope || interleaved ? rot % 8 == 0 : rot % 16 == 0) &&
       !(((uintptr_t)qkv | (uintptr_t)cache | (uintptr_t)q_out) & 15)) {
     const long long items = (long long)T_tokens * (nh + nkv + nvh) * (hd / 8);
-    if ((items + 255) / 256 <= 0x7fffffffLL) {
+    if (items < 0x7fffff00LL) {
       g2b_launch(proj_rope_cache_vec_kernel, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, stream, (const bf16 *)qkv,
                  row_stride, bias, nh, nkv, D, V, (const float2 *)rope, rot, interleaved, tok_pos, tok_seq, page_table, P,
                  (bf16 *)cache, page_size, (bf16 *)q_out, nvh, hd, T_tokens);
@@ -1101,14 +1101,14 @@ template <> __device__ __forceinline__ float4 load4<bf16>(const bf16 *p) {
 }
 template <typename T>
 __global__ void __launch_bounds__(128)
-head_norm_gate4_kernel(const float *__restrict__ o, long long items, int H, int V, const float *__restrict__ w, int w_head,
+head_norm_gate4_kernel(const float *__restrict__ o, unsigned items, int H, int V, const float *__restrict__ w, int w_head,
                        float eps, const T *__restrict__ gate, int gate_stride, float out_scale, T *__restrict__ out, int L) {
   pdl_launch();
   pdl_wait();
   const int lane = threadIdx.x % L;
-  const long long item = (long long)blockIdx.x * (128 / L) + threadIdx.x / L;
+  const unsigned item = blockIdx.x * (128 / L) + threadIdx.x / L;          // 32-bit: a 64-bit division costs more than the rest
   const bool in = item < items;
-  const int t = in ? (int)(item / H) : 0, h = in ? (int)(item % H) : 0;
+  const int t = in ? (int)(item / (unsigned)H) : 0, h = in ? (int)(item - (unsigned)t * H) : 0;
   const float *p = o + ((size_t)t * H + h) * V;
   float ss = 0.f;
   // the lane's first four of everything, asked for at once
@@ -1150,10 +1150,10 @@ extern "C" int g2b_head_norm_gate(const float *o, int T_tokens, int H, int V, co
   const int es = dtype == G2B_F32 ? 4 : 2;
   const bool on16 = V % 4 == 0 && !(((uintptr_t)o | (uintptr_t)w) & 15) && !((uintptr_t)out & (4 * es - 1)) &&
                     (!gate || (!((uintptr_t)gate & (4 * es - 1)) && gate_stride % 4 == 0));
-  if (on16) {
+  if (on16 && (long long)T_tokens * H < 0x7fffff00LL) {
     int L = 1;
     while (L < 32 && 4 * L < V) L <<= 1;
-    const long long items = (long long)T_tokens * H;
+    const unsigned items = (unsigned)T_tokens * (unsigned)H;
     const unsigned blocks = (unsigned)((items + 128 / L - 1) / (128 / L));
     if (dtype == G2B_F32)
       g2b_launch(head_norm_gate4_kernel<float>, dim3(blocks), dim3(128), 0, stream, o, items, H, V, w, w_head, eps,
@@ -1197,14 +1197,14 @@ gate_mul_kernel(const T *__restrict__ o, int hd, const T *__restrict__ gate, int
 
 // bfloat16, eight neighbours a thread (V, hd and the gate's stride multiples of eight)
 __global__ void __launch_bounds__(256)
-gate_mul8_kernel(const bf16 *__restrict__ o, int hd, const bf16 *__restrict__ gate, int gate_stride, long long total8, int H, int V,
+gate_mul8_kernel(const bf16 *__restrict__ o, int hd, const bf16 *__restrict__ gate, int gate_stride, unsigned total8, int H, int V,
                  float out_scale, bf16 *__restrict__ out) {
   pdl_launch();
   pdl_wait();
-  const long long i8 = (long long)blockIdx.x * 256 + threadIdx.x;
+  const unsigned i8 = blockIdx.x * 256 + threadIdx.x;
   if (i8 >= total8) return;
-  const int n8 = H * V / 8;
-  const int t = (int)(i8 / n8), r = (int)(i8 % n8) * 8, h = r / V, j = r - h * V;
+  const unsigned n8 = H * V / 8;
+  const int t = (int)(i8 / n8), r = (int)(i8 - t * n8) * 8, h = r / V, j = r - h * V;
   const uint4 x = *reinterpret_cast<const uint4 *>(o + ((size_t)t * H + h) * hd + j);
   uint4 g = make_uint4(0u, 0u, 0u, 0u), y;
   if (gate) g = *reinterpret_cast<const uint4 *>(gate + (size_t)t * gate_stride + r);
@@ -1218,14 +1218,14 @@ gate_mul8_kernel(const bf16 *__restrict__ o, int hd, const bf16 *__restrict__ ga
     }
     *reinterpret_cast<__nv_bfloat162 *>(&(&y.x)[k]) = __floats2bfloat162_rn(a * out_scale, b * out_scale);
   }
-  *reinterpret_cast<uint4 *>(out + i8 * 8) = y;
+  *reinterpret_cast<uint4 *>(out + (size_t)i8 * 8) = y;
 }
 
 extern "C" int g2b_gate_mul(const void *o, int hd, const void *gate, int gate_stride, int dtype, int T_tokens, int H,
                             int V, float out_scale, void *out, cudaStream_t stream) {
   if (T_tokens <= 0) return 0;
-  if (dtype == G2B_BF16 && V % 8 == 0 && hd % 8 == 0 && gate_stride % 8 == 0 && !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)out) & 15)) {
-    const long long total8 = (long long)T_tokens * H * V / 8;
+  if (dtype == G2B_BF16 && V % 8 == 0 && hd % 8 == 0 && gate_stride % 8 == 0 && !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)out) & 15) && (long long)T_tokens * H * V / 8 < 0x7fffff00LL) {
+    const unsigned total8 = (unsigned)((long long)T_tokens * H * V / 8);
     g2b_launch(gate_mul8_kernel, dim3((unsigned)((total8 + 255) / 256)), dim3(256), 0, stream, (const bf16 *)o, hd,
                (const bf16 *)gate, gate_stride, total8, H, V, out_scale, (bf16 *)out);
     return g2b_check_launch("gate_mul");

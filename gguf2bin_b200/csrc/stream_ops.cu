@@ -634,11 +634,12 @@ extern "C" int g2b_head_product(const void *in, int in_stride, const void *W, co
 
 // Many rows in bfloat16: the expanding product on the tensor cores (mma.sync), all heads in one launch.  A block takes
 // 64 tokens x 64 outputs of a head, four warps of 16 tokens; both operands' whole rows (r entries, a multiple of 16 once
-// filled with zeros) lie in shared memory.  The gate (one a head, or one an output) is applied to the accumulators.
+// filled with zeros) lie in shared memory.  (No __restrict__ on what earlier kernels write: the weights are read above
+// pdl_wait(), and loads through such pointers could be moved there, too.)  The gate (one a head, or one an output) is applied to the accumulators.
 #define HT_TILE 64
 __global__ void __launch_bounds__(128)
-head_expand_tile_kernel(const bf16 *__restrict__ in, int in_stride, const bf16 *__restrict__ W, const bf16 *__restrict__ gate,
-                        int gate_stride, int gate_each, bf16 *__restrict__ out, int out_stride, int T, int n, int r, int rp) {
+head_expand_tile_kernel(const bf16 *in, int in_stride, const bf16 *__restrict__ W, const bf16 *gate, int gate_stride,
+                        int gate_each, bf16 *out, int out_stride, int T, int n, int r, int rp) {
   pdl_launch();
   extern __shared__ __align__(128) unsigned char ht_smem[];
   const int row = rp + 8;                              // 16 bytes of padding: rows of eight start in different banks

@@ -33,13 +33,14 @@ __device__ __forceinline__ float dot4(const float4 &x, float c) {
 
 // A block a row; a thread keeps PER groups of four neighbours of every stream in registers.  JOIN false: nothing is
 // written back, `rows` may gather rows.
+// (No __restrict__ on what earlier kernels write: the compiler may move loads through such pointers above pdl_wait().)
 template <typename T, int S, int PER, bool JOIN>
 __global__ void __launch_bounds__(256)
-streams_kernel(float *__restrict__ X, const float *__restrict__ y, const float *__restrict__ mix,
-               const float *__restrict__ out, float m, const int *__restrict__ rows, const StreamsNext next, int H) {
+streams_kernel(float *X, const float *y, const float *__restrict__ mix, const float *__restrict__ out, float m, const int *rows,
+               const StreamsNext next, int H) {
   __shared__ float scratch[32];
   pdl_launch();
-  // coefficients are weights: no earlier kernel wrote them
+  // coefficients and norm weights are no earlier kernel's output
   float A[S], M[JOIN ? S * S : 1], O[S];
 #pragma unroll
   for (int s = 0; s < S; ++s) A[s] = next.in ? __ldg(next.in + s) : 1.f;
@@ -49,8 +50,15 @@ streams_kernel(float *__restrict__ X, const float *__restrict__ y, const float *
 #pragma unroll
     for (int s = 0; s < S; ++s) O[s] = m * __ldg(out + s);
   }
+  const int r = blockIdx.x, H4 = H >> 2;
+  float4 w[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int j = threadIdx.x + blockDim.x * i;
+    w[i] = next.w && j < H4 ? *reinterpret_cast<const float4 *>(next.w + 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
+  }
   pdl_wait();
-  const int r = blockIdx.x, t = rows ? rows[r] : r, H4 = H >> 2;
+  const int t = rows ? rows[r] : r;
   float *xr = X + (size_t)t * S * H;
   float4 u[PER];
   float ss = 0.f;
@@ -84,9 +92,8 @@ streams_kernel(float *__restrict__ X, const float *__restrict__ y, const float *
   for (int i = 0; i < PER; ++i) {
     const int j = threadIdx.x + blockDim.x * i;
     if (j >= H4) continue;
-    const float4 w = next.w ? *reinterpret_cast<const float4 *>(next.w + 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
     store4((T *)next.h + (size_t)r * H + 4 * j,
-           make_float4((w.x * u[i].x) * inv, (w.y * u[i].y) * inv, (w.z * u[i].z) * inv, (w.w * u[i].w) * inv));
+           make_float4((w[i].x * u[i].x) * inv, (w[i].y * u[i].y) * inv, (w[i].z * u[i].z) * inv, (w[i].w * u[i].w) * inv));
   }
 }
 
