@@ -30,12 +30,12 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + lo
 __device__ __forceinline__ float decay_of(float z, float inv_tau) { return expf(-softplus_f(-z) * inv_tau); }
 enum { DECAY_SIGMOID_ROOT = 0, DECAY_DOUBLE_EXP = 1 };
 
-// sum over r of w[r] * low[r], R a multiple of eight, ascending r
+// sum over r of w[r] * low[r], R a multiple of eight, ascending r; low on 16 bytes
 __device__ __forceinline__ float low_dot(const float *w, const float *low, int R, float acc) {
   for (int r = 0; r < R; r += 4) {
-    const float4 a = __ldg(reinterpret_cast<const float4 *>(w + r));
-    acc = fmaf(a.x, low[r], acc), acc = fmaf(a.y, low[r + 1], acc);
-    acc = fmaf(a.z, low[r + 2], acc), acc = fmaf(a.w, low[r + 3], acc);
+    const float4 a = __ldg(reinterpret_cast<const float4 *>(w + r)), l = *reinterpret_cast<const float4 *>(low + r);
+    acc = fmaf(a.x, l.x, acc), acc = fmaf(a.y, l.y, acc);
+    acc = fmaf(a.z, l.z, acc), acc = fmaf(a.w, l.w, acc);
   }
   return acc;
 }
@@ -44,9 +44,12 @@ __device__ __forceinline__ float low_dot(const bf16 *w, const float *low, int R,
     const uint4 a = __ldg(reinterpret_cast<const uint4 *>(w + r));
     const unsigned int u[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      acc = fmaf(__uint_as_float(u[i] << 16), low[r + 2 * i], acc);
-      acc = fmaf(__uint_as_float(u[i] & 0xffff0000u), low[r + 2 * i + 1], acc);
+    for (int i = 0; i < 4; i += 2) {
+      const float4 l = *reinterpret_cast<const float4 *>(low + r + 2 * i);
+      acc = fmaf(__uint_as_float(u[i] << 16), l.x, acc);
+      acc = fmaf(__uint_as_float(u[i] & 0xffff0000u), l.y, acc);
+      acc = fmaf(__uint_as_float(u[i + 1] << 16), l.z, acc);
+      acc = fmaf(__uint_as_float(u[i + 1] & 0xffff0000u), l.w, acc);
     }
   }
   return acc;

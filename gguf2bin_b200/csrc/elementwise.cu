@@ -14,6 +14,45 @@
 
 G2B_DEFINE_LAST_ERROR
 
+// E neighbours (4 or 8, a multiple of 4 in float) in accesses of 8 or 16 bytes
+template <int E> __device__ __forceinline__ void ldE(const bf16 *p, float (&v)[E]) {
+  if constexpr (E == 8) {
+    const uint4 raw = *reinterpret_cast<const uint4 *>(p);
+    const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&w[i]));
+      v[2 * i] = f.x; v[2 * i + 1] = f.y;
+    }
+  } else {
+    const uint2 raw = *reinterpret_cast<const uint2 *>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&raw.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&raw.y));
+    v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+  }
+}
+template <int E> __device__ __forceinline__ void ldE(const float *p, float (&v)[E]) {
+#pragma unroll
+  for (int i = 0; i < E; i += 4) {
+    const float4 raw = *reinterpret_cast<const float4 *>(p + i);
+    v[i] = raw.x; v[i + 1] = raw.y; v[i + 2] = raw.z; v[i + 3] = raw.w;
+  }
+}
+template <int E> __device__ __forceinline__ void stE(bf16 *p, const float (&v)[E]) {
+  uint32_t w[E / 2];
+#pragma unroll
+  for (int i = 0; i < E / 2; ++i) {
+    __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    w[i] = *reinterpret_cast<uint32_t *>(&h);
+  }
+  if constexpr (E == 8) *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+  else *reinterpret_cast<uint2 *>(p) = make_uint2(w[0], w[1]);
+}
+template <int E> __device__ __forceinline__ void stE(float *p, const float (&v)[E]) {
+#pragma unroll
+  for (int i = 0; i < E; i += 4) *reinterpret_cast<float4 *>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+}
+
 // ---------------------------------------------------------------------------
 // embedding: out[t, :] = table[ids[t], :] * scale   (out is the 32-bit residual stream); with a position
 // table also + positions[tok_pos[t], :], and a second copy of the rows into `again` when it is given
@@ -73,16 +112,28 @@ embed_norm_rows_kernel(const TW *__restrict__ table, const int *__restrict__ ids
   if (!ok) id = 0;                                   // host validates ids; never read outside
   const TW *row = table + (size_t)id * H;
   float ss = 0.f;
-  for (int j = threadIdx.x; j < H; j += blockDim.x) {
-    const float v = ok ? to_f32(row[j]) * scale : 0.f;
-    ss = fmaf(v, v, ss);
-  }
-  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
-  if (VEC) {                                         // H a multiple of four: 16-byte stores
+  if (VEC) {                                         // H a multiple of four, everything on four entries: 16-byte stores
     for (int j = 4 * threadIdx.x; j < H; j += 4 * blockDim.x) {
       float v[4];
+      ldE<4>(row + j, v);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) v[i] = ((ok ? to_f32(row[j + i]) * scale : 0.f) * inv) * (w ? w[j + i] : 1.f);
+      for (int i = 0; i < 4; ++i) ss = fmaf(v[i] * scale, v[i] * scale, ss);
+    }
+    if (!ok) ss = 0.f;
+  } else {
+    for (int j = threadIdx.x; j < H; j += blockDim.x) {
+      const float v = ok ? to_f32(row[j]) * scale : 0.f;
+      ss = fmaf(v, v, ss);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
+  if (VEC) {
+    for (int j = 4 * threadIdx.x; j < H; j += 4 * blockDim.x) {
+      float v[4], g[4] = {1.f, 1.f, 1.f, 1.f};
+      ldE<4>(row + j, v);
+      if (w) ldE<4>(w + j, g);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] = ((ok ? v[i] * scale : 0.f) * inv) * g[i];
       for (int c = 0; c < copies; ++c)
         *reinterpret_cast<float4 *>(out + ((size_t)t * copies + c) * H + j) = make_float4(v[0], v[1], v[2], v[3]);
     }
@@ -98,7 +149,7 @@ extern "C" int g2b_embed_norm_rows(const void *table, int table_dtype, const int
                                    int copies, int T, int H, int V, float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || V <= 0 || copies <= 0) G2B_REFUSE("embed_norm_rows: bad sizes H=%d V=%d copies=%d", H, V, copies);
-  const bool vec = H % 4 == 0 && !((uintptr_t)out & 15);
+  const bool vec = H % 4 == 0 && !(((uintptr_t)out | (uintptr_t)w) & 15) && !((uintptr_t)table & (table_dtype == G2B_F32 ? 15 : 7));
   const int threads = H >= 256 ? 256 : 64;
   if (table_dtype == G2B_F32)
     g2b_launch(vec ? embed_norm_rows_kernel<float, true> : embed_norm_rows_kernel<float, false>, dim3(T), dim3(threads), 0, stream, (const float *)table, ids, w, eps, out, copies,
@@ -338,44 +389,6 @@ extern "C" int g2b_rope_table(const int *tok_pos, const float *inv_freq, float *
 // second half, loaded and stored as vectors; everything stays in registers.  E = 4 gives a
 // decode step more lanes per head (shorter chains); E = 8 moves 16 bytes per load for prompts.
 #define QKN_FAST_WARPS 8
-
-template <int E> __device__ __forceinline__ void ldE(const bf16 *p, float (&v)[E]) {
-  if constexpr (E == 8) {
-    const uint4 raw = *reinterpret_cast<const uint4 *>(p);
-    const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&w[i]));
-      v[2 * i] = f.x; v[2 * i + 1] = f.y;
-    }
-  } else {
-    const uint2 raw = *reinterpret_cast<const uint2 *>(p);
-    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&raw.x));
-    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&raw.y));
-    v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
-  }
-}
-template <int E> __device__ __forceinline__ void ldE(const float *p, float (&v)[E]) {
-#pragma unroll
-  for (int i = 0; i < E; i += 4) {
-    const float4 raw = *reinterpret_cast<const float4 *>(p + i);
-    v[i] = raw.x; v[i + 1] = raw.y; v[i + 2] = raw.z; v[i + 3] = raw.w;
-  }
-}
-template <int E> __device__ __forceinline__ void stE(bf16 *p, const float (&v)[E]) {
-  uint32_t w[E / 2];
-#pragma unroll
-  for (int i = 0; i < E / 2; ++i) {
-    __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-    w[i] = *reinterpret_cast<uint32_t *>(&h);
-  }
-  if constexpr (E == 8) *reinterpret_cast<uint4 *>(p) = make_uint4(w[0], w[1], w[2], w[3]);
-  else *reinterpret_cast<uint2 *>(p) = make_uint2(w[0], w[1]);
-}
-template <int E> __device__ __forceinline__ void stE(float *p, const float (&v)[E]) {
-#pragma unroll
-  for (int i = 0; i < E; i += 4) *reinterpret_cast<float4 *>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
-}
 
 template <typename T, int LPH, int E>
 __global__ void __launch_bounds__(QKN_FAST_WARPS * 32)
@@ -739,14 +752,15 @@ shift_mix_kernel(const T *__restrict__ h, int h_stride, const float *__restrict_
   if (first) *keep = h[(size_t)(first_row + rows - 1) * h_stride + j];       // this thread alone reads and writes that entry
 }
 
-// four bfloat16 neighbours a thread, 8-byte accesses
+// N (4 or 8) bfloat16 neighbours a thread
+template <int N>
 __global__ void __launch_bounds__(256)
-shift_mix4_kernel(const bf16 *__restrict__ h, int h_stride, const float *__restrict__ mu, int n, bf16 *__restrict__ kept,
+shift_mix_vec_kernel(const bf16 *__restrict__ h, int h_stride, const float *__restrict__ mu, int n, bf16 *__restrict__ kept,
                   const int *__restrict__ tok_seq, const int *__restrict__ tok_pos, const int *__restrict__ seq_slots,
                   const int *__restrict__ seq_meta, int n_tokens, int H, bf16 *__restrict__ out) {
   pdl_launch();
   pdl_wait();
-  const int t = blockIdx.x, j = (blockIdx.y * 256 + threadIdx.x) * 4;
+  const int t = blockIdx.x, j = (blockIdx.y * blockDim.x + threadIdx.x) * N;
   if (j >= H) return;
   const int b = tok_seq[t];
   const int first_row = seq_meta ? seq_meta[4 * b + 0] : t, rows = seq_meta ? seq_meta[4 * b + 1] : 1;
@@ -755,22 +769,32 @@ shift_mix4_kernel(const bf16 *__restrict__ h, int h_stride, const float *__restr
   const bool first = t == first_row;
   bf16 *keep = kept + (size_t)slot * H + j;
   const bf16 *own = h + (size_t)t * h_stride + j;
-  const uint2 xr = *reinterpret_cast<const uint2 *>(own);
-  uint2 pr = make_uint2(0u, 0u);
-  if (!first) pr = *reinterpret_cast<const uint2 *>(own - h_stride);
-  else if (past > 0) pr = *reinterpret_cast<const uint2 *>(keep);
-  const float x[4] = {__uint_as_float(xr.x << 16), __uint_as_float(xr.x & 0xffff0000u), __uint_as_float(xr.y << 16),
-                      __uint_as_float(xr.y & 0xffff0000u)};
-  const float d[4] = {__uint_as_float(pr.x << 16) - x[0], __uint_as_float(pr.x & 0xffff0000u) - x[1],
-                      __uint_as_float(pr.y << 16) - x[2], __uint_as_float(pr.y & 0xffff0000u) - x[3]};
-  for (int m = 0; m < n; ++m) {
-    const float4 w = *reinterpret_cast<const float4 *>(mu + (size_t)m * H + j);
-    uint2 r;
-    *reinterpret_cast<__nv_bfloat162 *>(&r.x) = __floats2bfloat162_rn(fmaf(d[0], w.x, x[0]), fmaf(d[1], w.y, x[1]));
-    *reinterpret_cast<__nv_bfloat162 *>(&r.y) = __floats2bfloat162_rn(fmaf(d[2], w.z, x[2]), fmaf(d[3], w.w, x[3]));
-    *reinterpret_cast<uint2 *>(out + ((size_t)m * n_tokens + t) * H + j) = r;
+  float x[N], d[N];
+  ldE<N>(own, x);
+  if (!first) {
+    ldE<N>(own - h_stride, d);
+  } else if (past > 0) {
+    ldE<N>(keep, d);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) d[i] = 0.f;
   }
-  if (first) *reinterpret_cast<uint2 *>(keep) = *reinterpret_cast<const uint2 *>(h + (size_t)(first_row + rows - 1) * h_stride + j);
+#pragma unroll
+  for (int i = 0; i < N; ++i) d[i] -= x[i];
+  for (int m = 0; m < n; ++m) {
+    float r[N];
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      const float4 w = *reinterpret_cast<const float4 *>(mu + (size_t)m * H + j + i);
+      r[i] = fmaf(d[i], w.x, x[i]), r[i + 1] = fmaf(d[i + 1], w.y, x[i + 1]);
+      r[i + 2] = fmaf(d[i + 2], w.z, x[i + 2]), r[i + 3] = fmaf(d[i + 3], w.w, x[i + 3]);
+    }
+    stE<N>(out + ((size_t)m * n_tokens + t) * H + j, r);
+  }
+  if (first) {                                       // this thread alone reads and writes these entries of the slot
+    ldE<N>(h + (size_t)(first_row + rows - 1) * h_stride + j, x);
+    stE<N>(keep, x);
+  }
 }
 
 extern "C" int g2b_shift_mix(const void *h, int h_stride, const float *mu, int n, void *kept, const int *tok_seq,
@@ -779,9 +803,14 @@ extern "C" int g2b_shift_mix(const void *h, int h_stride, const float *mu, int n
   if (T_tokens <= 0) return 0;
   if (!mu || n <= 0 || !kept || !tok_seq || (!seq_meta && (!tok_pos || !seq_slots)))
     G2B_REFUSE("shift_mix: mixing weights, kept rows and the step's tables are needed");
-  if (dtype == G2B_BF16 && H % 4 == 0 && h_stride % 4 == 0 && !(((uintptr_t)h | (uintptr_t)kept | (uintptr_t)out) & 7) && !((uintptr_t)mu & 15)) {
-    g2b_launch(shift_mix4_kernel, dim3(T_tokens, (H / 4 + 255) / 256), dim3(256), 0, stream, (const bf16 *)h, h_stride, mu, n,
-               (bf16 *)kept, tok_seq, tok_pos, seq_slots, seq_meta, T_tokens, H, (bf16 *)out);
+  const uintptr_t at = (uintptr_t)h | (uintptr_t)kept | (uintptr_t)out;
+  if (dtype == G2B_BF16 && H % 4 == 0 && h_stride % 4 == 0 && !(at & 7) && !((uintptr_t)mu & 15)) {
+    const bool wide = H % 8 == 0 && h_stride % 8 == 0 && !(at & 15) && T_tokens >= 64;
+    const int pieces = H / (wide ? 8 : 4), threads = pieces >= 256 ? 256 : (pieces + 31) / 32 * 32;
+    const dim3 grid(T_tokens, (pieces + threads - 1) / threads);
+    if (grid.y > 65535) G2B_REFUSE("shift_mix: rows of %d", H);
+    g2b_launch(wide ? shift_mix_vec_kernel<8> : shift_mix_vec_kernel<4>, grid, dim3(threads), 0, stream, (const bf16 *)h, h_stride, mu,
+               n, (bf16 *)kept, tok_seq, tok_pos, seq_slots, seq_meta, T_tokens, H, (bf16 *)out);
     return g2b_check_launch("shift_mix");
   }
   const dim3 grid(T_tokens, (H + 255) / 256);

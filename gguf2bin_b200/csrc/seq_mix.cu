@@ -254,7 +254,10 @@ proj_rope_cache_vec_kernel(const bf16 *__restrict__ qkv, int row_stride, const f
     }
     if (bias) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) v[i] += bias[col + at + i];
+      for (int i = 0; i < 8; i += 4) {
+        const float4 b = *reinterpret_cast<const float4 *>(bias + col + at + i);
+        v[i] += b.x, v[i + 1] += b.y, v[i + 2] += b.z, v[i + 3] += b.w;
+      }
     }
   };
   if (d < n) {
@@ -264,20 +267,21 @@ proj_rope_cache_vec_kernel(const bf16 *__restrict__ qkv, int row_stride, const f
       const float2 *cs = rope + (size_t)t * half;
       if (interleaved) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float2 c = cs[(d >> 1) + i];
-          const float u = x[2 * i], v = x[2 * i + 1];
-          x[2 * i] = u * c.x - v * c.y;
-          x[2 * i + 1] = v * c.x + u * c.y;
+        for (int i = 0; i < 4; i += 2) {                 // two pairs' cosines and sines at a time
+          const float4 c = *reinterpret_cast<const float4 *>(cs + (d >> 1) + i);
+          const float u = x[2 * i], v = x[2 * i + 1], y = x[2 * i + 2], z = x[2 * i + 3];
+          x[2 * i] = u * c.x - v * c.y, x[2 * i + 1] = v * c.x + u * c.y;
+          x[2 * i + 2] = y * c.z - z * c.w, x[2 * i + 3] = z * c.z + y * c.w;
         }
       } else {
         const bool upper = d >= half;
         float o[8];
         fetch(upper ? d - half : d + half, o);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const float2 c = cs[(upper ? d - half : d) + i];
+        for (int i = 0; i < 8; i += 2) {
+          const float4 c = *reinterpret_cast<const float4 *>(cs + (upper ? d - half : d) + i);
           x[i] = upper ? x[i] * c.x + o[i] * c.y : x[i] * c.x - o[i] * c.y;
+          x[i + 1] = upper ? x[i + 1] * c.z + o[i + 1] * c.w : x[i + 1] * c.z - o[i + 1] * c.w;
         }
       }
     }
@@ -313,7 +317,7 @@ extern "C" int g2b_proj_norm_rope_cache(const void *qkv, int dtype, int row_stri
   if (nkv > 0 && !cache) G2B_REFUSE("proj_norm_rope_cache: keys without pages to write them to");
   if (dtype == G2B_BF16 && !q_w && !k_w && unit_eps <= 0.f && v_norm_eps <= 0.f && D % 8 == 0 && V % 8 == 0 && hd % 8 == 0 &&
       row_stride % 8 == 0 && (!rope || interleaved ? rot % 8 == 0 : rot % 16 == 0) &&
-      !(((uintptr_t)qkv | (uintptr_t)cache | (uintptr_t)q_out) & 15)) {
+      !(((uintptr_t)qkv | (uintptr_t)cache | (uintptr_t)q_out | (uintptr_t)bias | (uintptr_t)rope) & 15)) {
     const long long items = (long long)T_tokens * (nh + nkv + nvh) * (hd / 8);
     if (items < 0x7fffff00LL) {
       g2b_launch(proj_rope_cache_vec_kernel, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, stream, (const bf16 *)qkv,
@@ -1099,45 +1103,52 @@ template <> __device__ __forceinline__ float4 load4<bf16>(const bf16 *p) {
   return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xffff0000u), __uint_as_float(r.y << 16),
                      __uint_as_float(r.y & 0xffff0000u));
 }
-template <typename T>
+// ITEMS heads a group of lanes, one behind the other, their loads all under way first (prompts).
+template <typename T, int ITEMS>
 __global__ void __launch_bounds__(128)
 head_norm_gate4_kernel(const float *__restrict__ o, unsigned items, int H, int V, const float *__restrict__ w, int w_head,
                        float eps, const T *__restrict__ gate, int gate_stride, float out_scale, T *__restrict__ out, int L) {
   pdl_launch();
   pdl_wait();
   const int lane = threadIdx.x % L;
-  const unsigned item = blockIdx.x * (128 / L) + threadIdx.x / L;          // 32-bit: a 64-bit division costs more than the rest
-  const bool in = item < items;
-  const int t = in ? (int)(item / (unsigned)H) : 0, h = in ? (int)(item - (unsigned)t * H) : 0;
-  const float *p = o + ((size_t)t * H + h) * V;
-  float ss = 0.f;
-  // the lane's first four of everything, asked for at once
+  const unsigned first = (blockIdx.x * (128 / L) + threadIdx.x / L) * ITEMS;      // 32-bit: a 64-bit division costs more than the rest
   const int j0 = min(4 * lane, V - 4);
-  const float4 x0 = load4<float>(p + j0);
-  const float4 w0 = w ? load4<float>(w + (size_t)h * w_head + j0) : make_float4(1.f, 1.f, 1.f, 1.f);
-  const float4 g0 = gate ? load4<T>(gate + (size_t)t * gate_stride + (size_t)h * V + j0) : make_float4(0.f, 0.f, 0.f, 0.f);
-  if (in)
+  float4 x0[ITEMS], w0[ITEMS], g0[ITEMS];
+  int t[ITEMS], h[ITEMS];
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const unsigned item = min(first + i, items - 1);
+    t[i] = (int)(item / (unsigned)H), h[i] = (int)(item - (unsigned)t[i] * H);
+    x0[i] = load4<float>(o + ((size_t)t[i] * H + h[i]) * V + j0);
+    w0[i] = w ? load4<float>(w + (size_t)h[i] * w_head + j0) : make_float4(1.f, 1.f, 1.f, 1.f);
+    g0[i] = gate ? load4<T>(gate + (size_t)t[i] * gate_stride + (size_t)h[i] * V + j0) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    const float *p = o + ((size_t)t[i] * H + h[i]) * V;
+    float ss = 0.f;
     for (int j = 4 * lane; j < V; j += 4 * L) {
-      const float4 x = j == 4 * lane ? x0 : load4<float>(p + j);
+      const float4 x = j == 4 * lane ? x0[i] : load4<float>(p + j);
       ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss))));
     }
-  for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
-  if (!in) return;
-  const float inv = 1.f / sqrtf(ss / (float)V + eps);
-  for (int j = 4 * lane; j < V; j += 4 * L) {
-    const bool again = j != 4 * lane;
-    float4 y = again ? load4<float>(p + j) : x0;
-    y.x *= inv, y.y *= inv, y.z *= inv, y.w *= inv;
-    if (w) {
-      const float4 g = again ? load4<float>(w + (size_t)h * w_head + j) : w0;
-      y.x *= g.x, y.y *= g.y, y.z *= g.z, y.w *= g.w;
+    for (int m = L >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    if (first + i >= items) continue;                  // (its lanes only took part in the sums)
+    const float inv = 1.f / sqrtf(ss / (float)V + eps);
+    for (int j = 4 * lane; j < V; j += 4 * L) {
+      const bool again = j != 4 * lane;
+      float4 y = again ? load4<float>(p + j) : x0[i];
+      y.x *= inv, y.y *= inv, y.z *= inv, y.w *= inv;
+      if (w) {
+        const float4 g = again ? load4<float>(w + (size_t)h[i] * w_head + j) : w0[i];
+        y.x *= g.x, y.y *= g.y, y.z *= g.z, y.w *= g.w;
+      }
+      if (gate) {
+        const float4 g = again ? load4<T>(gate + (size_t)t[i] * gate_stride + (size_t)h[i] * V + j) : g0[i];
+        y.x *= silu_f(g.x), y.y *= silu_f(g.y), y.z *= silu_f(g.z), y.w *= silu_f(g.w);
+      }
+      y.x *= out_scale, y.y *= out_scale, y.z *= out_scale, y.w *= out_scale;
+      join_store4(out + ((size_t)t[i] * H + h[i]) * V + j, y);
     }
-    if (gate) {
-      const float4 g = again ? load4<T>(gate + (size_t)t * gate_stride + (size_t)h * V + j) : g0;
-      y.x *= silu_f(g.x), y.y *= silu_f(g.y), y.z *= silu_f(g.z), y.w *= silu_f(g.w);
-    }
-    y.x *= out_scale, y.y *= out_scale, y.z *= out_scale, y.w *= out_scale;
-    join_store4(out + ((size_t)t * H + h) * V + j, y);
   }
 }
 
@@ -1154,12 +1165,13 @@ extern "C" int g2b_head_norm_gate(const float *o, int T_tokens, int H, int V, co
     int L = 1;
     while (L < 32 && 4 * L < V) L <<= 1;
     const unsigned items = (unsigned)T_tokens * (unsigned)H;
-    const unsigned blocks = (unsigned)((items + 128 / L - 1) / (128 / L));
+    const bool many = items >= 16384;
+    const unsigned per = 128 / L * (many ? 4 : 1), blocks = (items + per - 1) / per;
     if (dtype == G2B_F32)
-      g2b_launch(head_norm_gate4_kernel<float>, dim3(blocks), dim3(128), 0, stream, o, items, H, V, w, w_head, eps,
+      g2b_launch(many ? head_norm_gate4_kernel<float, 4> : head_norm_gate4_kernel<float, 1>, dim3(blocks), dim3(128), 0, stream, o, items, H, V, w, w_head, eps,
                  (const float *)gate, gate_stride, out_scale, (float *)out, L);
     else if (dtype == G2B_BF16)
-      g2b_launch(head_norm_gate4_kernel<bf16>, dim3(blocks), dim3(128), 0, stream, o, items, H, V, w, w_head, eps,
+      g2b_launch(many ? head_norm_gate4_kernel<bf16, 4> : head_norm_gate4_kernel<bf16, 1>, dim3(blocks), dim3(128), 0, stream, o, items, H, V, w, w_head, eps,
                  (const bf16 *)gate, gate_stride, out_scale, (bf16 *)out, L);
     else
       G2B_REFUSE("head_norm_gate: unknown dtype %d", dtype);
