@@ -7,6 +7,7 @@ bandwidth or FLOP/s.
     python -m gguf2bin_b200.kernel_bench prefill [--tokens 2048] [--only NAME] [--layers 4]
     python -m gguf2bin_b200.kernel_bench latent-decode | latent-prefill  [--rank 128] ...
     python -m gguf2bin_b200.kernel_bench state-decode | state-prefill  [--experts 16] [--top 4] [--chunk 512] ...
+    python -m gguf2bin_b200.kernel_bench streams-decode | streams-prefill  [--streams 2] [--rank 96] [--rot 32] [--window 512] ...
 
 The ``latent-*`` modes time the kernels of a gated layer with latent attention (``--heads`` heads of
 ``--head-dim`` key and value numbers, ``--rank`` cached numbers per token) at the same geometry.
@@ -14,6 +15,10 @@ The ``latent-*`` modes time the kernels of a gated layer with latent attention (
 The ``state-*`` modes time the kernels of layers that keep a matrix state per head (``--heads`` / 2 heads with
 keys of ``--head-dim`` and values of twice that), of attention in chunks of ``--chunk`` keys with the wide
 prologue, and of a routed feed-forward (``--experts`` experts of ``--inter`` / 4 each, ``--top`` choices).
+
+The ``streams-*`` modes time the kernels of a model of several residual streams (``--streams``) with time mixing
+(``--hidden`` / 64 heads of 64), latent attention with rotated entries (``--rank`` + ``--rot`` numbers a token) and
+attention behind ``--window`` tokens, beside the like kernels of a model of one stream.
 
 Sizes default to Qwen3-0.6B (width 1024, 16/8 heads of 128, feed-forward 3072, vocabulary
 151936); --hidden/--inter/--heads/--kv-heads/--vocab change them.  Decode kernels run
@@ -390,13 +395,121 @@ def state(a, single: bool) -> None:
     kernels_bf16.check_status()
 
 
+def streams(a, single: bool) -> None:
+    """The kernels around several residual streams, time mixing, rotated latents and windowed attention: ``single``: a
+    decode step of ``--batch`` sequences behind ``--ctx`` tokens; else one prompt of ``--tokens`` tokens.  Every kernel
+    walks over ``--layers`` copies of what it reads and writes."""
+    from .parts.base import StepContext
+    L, W, S, nh, nkv, hd = a.layers, a.hidden, a.streams, a.heads, a.kv_heads, a.head_dim
+    r, rot, I = a.rank, a.rot, a.inter
+    B = a.batch if single else 1
+    n = 1 if single else a.tokens
+    T, past, ps = B * n, (a.ctx if single else 0), 64
+    b = Bench(a)
+    per = -(-(past + n) // ps)
+    table = torch.arange(B * per, dtype=torch.int32, device=DEV).view(B, per)
+    pos = (torch.arange(n, dtype=torch.int32, device=DEV) + past).repeat(B)
+    seq = torch.arange(B, dtype=torch.int32, device=DEV).repeat_interleave(n)
+    tiles = {rows: torch.tensor(sorted([(s, s * n + r0, min(rows, n - r0), past + r0) for s in range(B) for r0 in range(0, n, rows)],
+                                       key=lambda t: -(t[3] + t[2])), dtype=torch.int32, device=DEV) for rows in (64, 128)}
+    meta = torch.tensor([[s * n, n, past, s] for s in range(B)], dtype=torch.int32, device=DEV)
+    ctx = StepContext(n_tokens=T, n_seqs=B, tok_ids=pos, tok_pos=pos, tok_seq=seq, page_table=table, page_size=ps,
+                      workspace=Workspace(DEV), dtype=torch.bfloat16, q_lens=[n] * B, past_lens=[past] * B, slots=list(range(B)),
+                      max_kv_len=per * ps, kv_len_hint=past + n, seq_meta=None if single else meta,
+                      seq_slots=torch.arange(B, dtype=torch.int32, device=DEV), attn_tiles=tiles[64], n_attn_tiles=len(tiles[64]),
+                      attn_tiles_wide=tiles[128], n_attn_tiles_wide=len(tiles[128]))
+    f32 = lambda *shape: torch.randn(*shape, device=DEV)                      # noqa: E731
+    each = lambda make: [make() for _ in range(L)]                            # noqa: E731
+    mm = (lambda N, K, G=1: dict(nbytes=G * N * K * 2)) if single else (lambda N, K, G=1: dict(flops=2 * G * T * N * K))
+    # ---- the streams, beside one stream between two norms ---------------------------------------------
+    mix, out, coef, nw = torch.eye(S, device=DEV) + 0.1 * f32(S, S), f32(S), f32(S), torch.ones(W, device=DEV)
+    if b.want("streams_join") or b.want("streams_read"):
+        X, y, h = each(lambda: f32(T, S, W)), each(lambda: f32(T, W)), each(lambda: bf(T, W))
+        b.run("streams_join", lambda: [kernels.streams_join(X[i], y[i], mix, out, 0.5, (coef, nw, 1e-6), h[i]) for i in range(L)], L,
+              nbytes=T * W * (8 * S + 6))
+        b.run("streams_read", lambda: [kernels.streams_read(X[i], coef, nw, 1e-6, h[i]) for i in range(L)], L, nbytes=T * W * (4 * S + 2))
+        del X, y, h
+    if b.want("norm_join"):
+        X, y, h = each(lambda: f32(T, W)), each(lambda: f32(T, W)), each(lambda: bf(T, W))
+        b.run("norm_join", lambda: [kernels.norm_join(X[i], y[i], nw, 1e-6, (nw, 1e-6), h[i]) for i in range(L)], L, nbytes=T * W * 14)
+        del X, y, h
+    # ---- time mixing, beside the scan without a bonus ---------------------------------------------------
+    D, H = 64, W // 64
+    h, mixed = each(lambda: bf(T, W)), each(lambda: bf(5, T, W))
+    mu, kept = f32(5, W), torch.zeros(B + 1, W, dtype=torch.bfloat16, device=DEV)
+    b.run("shift_mix", lambda: [kernels.shift_mix(h[i], mu, kept, ctx, mixed[i]) for i in range(L)], L, nbytes=T * W * 12)
+    proj = each(lambda: bf(T, 4 * W) * 50)
+    if b.want("four products"):
+        w4 = each(lambda: bf(4, W, W))
+        b.run("four products", lambda: [kernels.linear_stacked(mixed[i][:4], w4[i], proj[i]) for i in range(L)], L, **mm(W, W, 4))
+        del w4
+    low, w2, w0, bonus = each(lambda: f32(T, 16)), bf(W, 16), f32(W) - 2, f32(H, D)
+    o32 = each(lambda: f32(T, W))
+    for name, Hs, Ds, Vs in (("scan with a bonus", H, D, D), ("scan", W // 256, 128, 256)):
+        if not b.want(name):
+            continue
+        st = each(lambda: torch.zeros(B + 1, Hs, Vs, Ds, device=DEV))
+        nq, nv = Hs * Ds, Hs * Vs
+        kw = dict(decay="double_exp", low_tanh=True, bonus=bonus) if Vs == D else dict(tau=16.0)
+        lows = low if Vs == D else each(lambda: bf(T, 16))
+        b.run(name, lambda: [kernels.channel_scan(proj[i][:, :nq], proj[i][:, nq:2 * nq], proj[i][:, 2 * nq:2 * nq + nv], lows[i],
+                                                  w2[:nq], w0[:nq], st[i], ctx, o32[i], Hs, Ds, Vs, 1.0, **kw) for i in range(L)], L,
+              nbytes=2 * 4 * B * Hs * Vs * Ds + T * (2 * nq + nv) * 2 + T * nv * 4, flops=6.0 * T * Hs * Ds * Vs)
+    nrm, og = f32(W), each(lambda: bf(T, W))
+    b.run("head_norm_gate", lambda: [kernels.head_norm_gate(o32[i], H, D, nrm, 1e-6, proj[i][:, 3 * W:], 1.0, og[i]) for i in range(L)],
+          L, nbytes=T * W * 8)
+    # ---- latent attention with rotated entries ------------------------------------------------------------
+    R = kernels.padded_head_size(r + rot)
+    inv = torch.tensor([1e4 ** (-2.0 * j / rot) for j in range(rot // 2)], device=DEV)
+    rope, cn = ctx.rope_table(inv), torch.ones(r, device=DEV)
+    lat = each(lambda: torch.randn(B * per + 1, 1, 1, ps, R, device=DEV).to(torch.bfloat16))
+    lp = each(lambda: bf(T, nh * R + r + rot + (-(r + rot) % 8)))
+    b.run("latent_rope", lambda: [kernels.latent_rope(lp[i][:, nh * R:nh * R + r + rot], r, R, cn, 1e-6, lat[i], lp[i][:, r:], R, lp[i][:, r:],
+                                                      R, nh, rot, rope, True, ctx) for i in range(L)], L,
+          nbytes=T * 2 * (2 * nh * rot + r + rot + R))
+    mixo, gate, o = each(lambda: bf(T, nh * R)), each(lambda: bf(T, nh * hd)), each(lambda: bf(T, nh * hd))
+    at = dict(nbytes=B * (past + 1) * R * 2) if single else dict(flops=2.0 * nh * (2 * r + rot) * n * (n + 1) / 2)
+    b.run("latent attention", lambda: [kernels.attention(lp[i][:, :nh * R], mixo[i], lat[i], ctx, nh, 1, R, ps, 0, 0.08, planes=1)
+                                       for i in range(L)], L, **at)
+    uv = each(lambda: bf(nh * hd, R))
+    expand = (lambda i: kernels.head_product(mixo[i], uv[i], o[i], nh, True, gate[i])) if single else \
+        (lambda i: kernels.head_expand_tiles(mixo[i], uv[i], o[i], nh, gate[i]))
+    b.run("values and gate", lambda: [expand(i) for i in range(L)], L, nbytes=T * nh * (R + 2 * hd) * 2 + nh * hd * R * 2)
+    # ---- attention behind a window that keeps the first tokens ---------------------------------------------
+    nq, nk = nh * hd, nkv * hd
+    inv2 = torch.tensor([5e5 ** (-2.0 * j / hd) for j in range(hd // 2)], device=DEV)
+    rope2, bias = ctx.rope_table(inv2), f32(nq + 2 * nk)
+    qkv, qo = each(lambda: bf(T, 2 * nq + 2 * nk)), each(lambda: bf(T, nq))
+    kv = each(lambda: torch.randn(B * per + 1, 2, nkv, ps, hd, device=DEV).to(torch.bfloat16))
+    b.run("bias, rotation, pages", lambda: [kernels.proj_norm_rope_cache(qkv[i], bias, nh, nkv, hd, hd, None, None, 0.0, rope2, hd, False, ctx,
+                                                                         kv[i], ps, qo[i]) for i in range(L)], L, nbytes=T * (nq + 2 * nk) * 4)
+    win, keep = a.window, 8
+    seen = min(past + 1, win + keep)
+    at = dict(nbytes=B * seen * 2 * nk * 2) if single else dict(flops=4.0 * nq * sum(min(t + 1, win) + min(keep, max(0, t + 1 - win)) for t in range(n)))
+    b.run("windowed attention", lambda: [kernels.attention(qo[i], o[i], kv[i], ctx, nh, nkv, hd, ps, win, hd ** -0.5, keep_first=keep)
+                                         for i in range(L)], L, **at)
+    b.run("gate_mul", lambda: [kernels.gate_mul(o[i], hd, gate[i], nh, hd, 1.0, qo[i]) for i in range(L)], L, nbytes=T * nq * 6)
+    # ---- the feed-forward's first product with its activation ----------------------------------------------
+    if b.want("up and GELU"):
+        wu, mid = each(lambda: bf(I, W)), each(lambda: bf(T, I))
+        b.run("up and GELU", lambda: [kernels.linear_act(h[i], wu[i], mid[i], kernels.GluForm.gelu_tanh()) for i in range(L)], L, **mm(I, W))
+    if b.want("down"):
+        wd, mid, y = each(lambda: bf(W, I)), each(lambda: bf(T, I)), each(lambda: f32(T, W))
+        b.run("down", lambda: [kernels.linear(mid[i], wd[i], y[i]) for i in range(L)], L, **mm(W, I))
+    kernels_bf16.check_status()
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("mode", choices=["decode", "prefill", "latent-decode", "latent-prefill", "state-decode", "state-prefill"])
+    ap.add_argument("mode", choices=["decode", "prefill", "latent-decode", "latent-prefill", "state-decode", "state-prefill",
+                                     "streams-decode", "streams-prefill"])
     ap.add_argument("--experts", type=int, default=16, help="state modes: experts of the routed feed-forward")
     ap.add_argument("--top", type=int, default=4, help="state modes: experts a token uses")
     ap.add_argument("--chunk", type=int, default=512, help="state modes: keys a chunk of the attention holds")
     ap.add_argument("--rank", type=int, default=128, help="latent modes: cached numbers per token")
+    ap.add_argument("--streams", type=int, default=2, help="streams modes: residual streams")
+    ap.add_argument("--rot", type=int, default=32, help="streams modes: rotated numbers behind a latent")
+    ap.add_argument("--window", type=int, default=512, help="streams modes: tokens an attention layer sees")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--ctx", type=int, default=3072)
     ap.add_argument("--tokens", type=int, default=2048)
@@ -412,7 +525,9 @@ def main(argv=None) -> int:
     a = ap.parse_args(argv)
     if a.layers is None:
         a.layers = 28 if a.mode.endswith("decode") else 4
-    if a.mode.startswith("state"):
+    if a.mode.startswith("streams"):
+        streams(a, a.mode == "streams-decode")
+    elif a.mode.startswith("state"):
         state(a, a.mode == "state-decode")
     elif a.mode.startswith("latent"):
         latent(a, a.mode == "latent-decode")
