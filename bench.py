@@ -827,10 +827,10 @@ def nekotar_config(width, layers, vocab) -> dict:
             kind, mixer = "wkv", dict(heads=width // 64, dim=64)
         else:
             kind = "attention"
-            mixer = dict(heads=H, kv_heads=max(H // 4, 1), dim=128, vdim=128, scale=128 ** -0.5, rot=dict(base=5e5, dims=128),
+            mixer = dict(heads=H, kv_heads=max(H // 4, 1), dim=128, vdim=128, scale=128 ** -0.5, rot=dict(base=1e6, dims=128),
                          mask=dict(size=512, keep_first=8))
         out.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=9 * width // 2)))
-    return dict(architecture="Nekotar", width=width, vocab=vocab, streams=2, residual_mult=0.5, norm=dict(eps=1e-6), layers=out)
+    return dict(architecture="Nekotar", width=width, vocab=vocab, streams=2, residual_mult=0.7, norm=dict(eps=1e-5), layers=out)
 
 
 def nekotar_bytes_and_flops(cfg: dict, T: int) -> dict:

@@ -425,7 +425,7 @@ def streams(a, single: bool) -> None:
     mix, out, coef, nw = torch.eye(S, device=DEV) + 0.1 * f32(S, S), f32(S), f32(S), torch.ones(W, device=DEV)
     if b.want("streams_join") or b.want("streams_read"):
         X, y, h = each(lambda: f32(T, S, W)), each(lambda: f32(T, W)), each(lambda: bf(T, W))
-        b.run("streams_join", lambda: [kernels.streams_join(X[i], y[i], mix, out, 0.5, (coef, nw, 1e-6), h[i]) for i in range(L)], L,
+        b.run("streams_join", lambda: [kernels.streams_join(X[i], y[i], mix, out, 0.7, (coef, nw, 1e-6), h[i]) for i in range(L)], L,
               nbytes=T * W * (8 * S + 6))
         b.run("streams_read", lambda: [kernels.streams_read(X[i], coef, nw, 1e-6, h[i]) for i in range(L)], L, nbytes=T * W * (4 * S + 2))
         del X, y, h
@@ -477,7 +477,7 @@ def streams(a, single: bool) -> None:
     b.run("values and gate", lambda: [expand(i) for i in range(L)], L, nbytes=T * nh * (R + 2 * hd) * 2 + nh * hd * R * 2)
     # ---- attention behind a window that keeps the first tokens ---------------------------------------------
     nq, nk = nh * hd, nkv * hd
-    inv2 = torch.tensor([5e5 ** (-2.0 * j / hd) for j in range(hd // 2)], device=DEV)
+    inv2 = torch.tensor([1e6 ** (-2.0 * j / hd) for j in range(hd // 2)], device=DEV)
     rope2, bias = ctx.rope_table(inv2), f32(nq + 2 * nk)
     qkv, qo = each(lambda: bf(T, 2 * nq + 2 * nk)), each(lambda: bf(T, nq))
     kv = each(lambda: torch.randn(B * per + 1, 2, nkv, ps, hd, device=DEV).to(torch.bfloat16))
